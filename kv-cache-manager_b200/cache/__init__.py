@@ -16,8 +16,9 @@ Sequence = core.Sequence
 make_kv_manager = core.make_kv_manager
 
 
-def manager_from_config(kv_cfg, windows=(0,)):
-    """A ``KVManager`` from the Python-side ``KVManagerConfig`` dataclass and the groups' windows."""
+def manager_from_config(kv_cfg, windows=(0,), chunks=None):
+    """A ``KVManager`` from the Python-side ``KVManagerConfig`` dataclass and the groups' windows and chunk
+    sizes (None: no group is chunked)."""
     c = core.KVManagerConfig()
     c.policy = kv_cfg.policy
     c.num_blocks = int(kv_cfg.num_blocks)
@@ -26,7 +27,7 @@ def manager_from_config(kv_cfg, windows=(0,)):
     c.prefix_caching = bool(kv_cfg.prefix_caching) and kv_cfg.policy != "contiguous"
     c.watermark_blocks = int(kv_cfg.watermark_blocks)
     c.watermark_frac = float(kv_cfg.watermark_frac)
-    c.groups = [core.LayerGroupSpec(int(w)) for w in windows]
+    c.groups = [core.LayerGroupSpec(int(w), int(n)) for w, n in zip(windows, chunks or [0] * len(windows))]
     return core.make_kv_manager(c)
 
 

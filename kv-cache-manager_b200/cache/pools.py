@@ -6,7 +6,8 @@ values with the same geometry and window form a *layer group*: one pool
 same page in every site of its group, as in the reference's per-layer pools,
 ``src/cuda/kv_cache.h:1-2``), and one page table per request.  Pools are zero-filled so that a
 stray read is deterministic (``src/cuda/kv_cache.cu:12-14``).  Sites whose mixers ask for
-fixed-size state get a slab ``[slots, *shape]`` indexed by the request's state slot.
+fixed-size state get a slab ``[slots, *shape]`` indexed by the request's state slot, and so do sites
+whose block (the arrangement around the mixer) keeps state of its own.
 """
 from __future__ import annotations
 
@@ -32,14 +33,19 @@ class CachePlan:
     site_layer: List[int]            # per call site: index inside the group's pool
     site_writes: List[bool]
     site_state: List[Optional[StateSpec]]
+    site_block_state: List[Optional[StateSpec]]     # what the layer's block itself keeps per request
 
     @property
     def windows(self) -> List[int]:
         return [g.spec.window for g in self.groups]
 
     @property
+    def chunks(self) -> List[int]:
+        return [g.spec.chunk for g in self.groups]
+
+    @property
     def has_state(self) -> bool:
-        return any(s is not None for s in self.site_state)
+        return any(s is not None for s in self.site_state + self.site_block_state)
 
 
 def plan_cache(spec) -> CachePlan:
@@ -48,6 +54,7 @@ def plan_cache(spec) -> CachePlan:
     n = len(spec.order)
     site_group, site_layer, site_writes = [-1] * n, [-1] * n, [True] * n
     site_state: List[Optional[StateSpec]] = [None] * n
+    site_block_state: List[Optional[StateSpec]] = [None] * n
     for k, call in enumerate(spec.order):
         mixer = spec.blocks[call.layer].mixer
         cs, ss = mixer.cache_spec(), mixer.state_spec()
@@ -68,7 +75,8 @@ def plan_cache(spec) -> CachePlan:
             site_group[k], site_layer[k] = g, len(groups[g].sites)
             groups[g].sites.append(k)
         site_state[k] = ss
-    return CachePlan(groups, site_group, site_layer, site_writes, site_state)
+        site_block_state[k] = spec.blocks[call.layer].state_spec()
+    return CachePlan(groups, site_group, site_layer, site_writes, site_state, site_block_state)
 
 
 class CachePools:
@@ -82,20 +90,20 @@ class CachePools:
             shape = (len(g.sites), num_blocks, g.spec.num_kv_heads, block_size, g.spec.head_dim)
             self.k.append(torch.zeros(shape, dtype=dtype, device=device))
             self.v.append(torch.zeros(shape, dtype=dtype, device=device) if g.spec.values else None)
-        self.state: List[Optional[torch.Tensor]] = [
-            None if s is None else torch.zeros((num_slots, *s.shape), dtype=s.dtype, device=device)
-            for s in plan.site_state]
+        def slabs(specs) -> List[Optional[torch.Tensor]]:
+            return [None if s is None else torch.zeros((num_slots, *s.shape), dtype=s.dtype, device=device) for s in specs]
+        self.state, self.block_state = slabs(plan.site_state), slabs(plan.site_block_state)
         self.sites: List[SiteCache] = []
         for k in range(len(plan.site_group)):
             g = plan.site_group[k]
             self.sites.append(SiteCache(
                 group=g, k=self.k[g][plan.site_layer[k]] if g >= 0 else None,
                 v=self.v[g][plan.site_layer[k]] if g >= 0 and self.v[g] is not None else None,
-                writes=plan.site_writes[k], state=self.state[k]))
+                writes=plan.site_writes[k], state=self.state[k], block_state=self.block_state[k]))
 
     def reset_slot(self, slot: int) -> None:
         """A request that starts (again) from its first token starts from zero state."""
-        for s in self.state:
+        for s in self.state + self.block_state:
             if s is not None:
                 s[slot].zero_()
 

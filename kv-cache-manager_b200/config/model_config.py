@@ -609,3 +609,112 @@ class LobutarConfig(ModelConfig):
     def to_json_dict(self) -> Dict[str, Any]:
         return {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
                 "streams": self.streams, "layers": json.loads(json.dumps(list(self.layers)))}
+
+
+# ------------------------------------------------------------------------------------ Bimepel
+
+@dataclass(frozen=True)
+class BimepelConfig(ModelConfig):
+    """Bimepel: a decoder whose layers are listed one by one, parallel layers with a norm for each sublayer and a token
+    shift in front of every mixer, with a span of layers that runs several times in a row; the output head is the
+    token table.
+
+    Top level: ``vocab``, ``width``, ``norm.eps``, ``loop`` {start, stop, times} (optional) and ``layers``: a list of
+    {type, mixer, mlp}.  ``type`` "attention": mixer {heads, kv_heads, dim, vdim, scale, rot {base, dims, scaling
+    {factor, original, fast, slow} (optional)} (optional), mask {size} (optional: chunks of that many positions)};
+    "lightning": mixer {heads, dim, vdim, decay (one number per head)}.  ``mlp`` is null, {kind: "dense", ff, limit} or
+    {kind: "moe", expert {ff}, router {experts, top, scale}}.  ``layers`` is kept as the parsed JSON after validation; the
+    builder reads every size from it."""
+    vocab: int = 0
+    width: int = 0
+    norm_eps: float = 1e-6
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 1
+    layers: tuple = ()
+
+    @classmethod
+    def from_json_dict(cls, d: Dict[str, Any]) -> "BimepelConfig":
+        w = "config.json (Bimepel)"
+        norm = _section(d, "norm", w)
+        loop = _section(d, "loop", w, optional=True)
+        layers = d.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError(f"{w}: 'layers' must be a non-empty list")
+        cfg = cls(architecture="Bimepel", vocab=_require(d, "vocab", int, w), width=_require(d, "width", int, w),
+                  norm_eps=_require(norm, "eps", float, w + " norm"),
+                  loop_start=_require(loop, "start", int, w + " loop") if loop else 0,
+                  loop_stop=_require(loop, "stop", int, w + " loop") if loop else 0,
+                  loop_times=_require(loop, "times", int, w + " loop") if loop else 1,
+                  layers=tuple(json.loads(json.dumps(layers))))
+        cfg.validate()
+        return cfg
+
+    @property
+    def has_loop(self) -> bool:
+        return self.loop_stop > self.loop_start
+
+    def validate(self) -> None:
+        w = "BimepelConfig"
+        if self.vocab <= 0 or self.width <= 0:
+            raise ConfigError(f"{w}: 'vocab' and 'width' must be positive")
+        if not (self.norm_eps > 0):
+            raise ConfigError(f"{w}: norm.eps must be positive, got {self.norm_eps}")
+        n = len(self.layers)
+        if not (0 <= self.loop_start <= self.loop_stop <= n) or self.loop_times < 1:
+            raise ConfigError(f"{w}: loop needs 0 <= start <= stop <= {n} layers and times >= 1, got "
+                              f"start {self.loop_start}, stop {self.loop_stop}, times {self.loop_times}")
+        for i, layer in enumerate(self.layers):
+            lw = f"{w}: layer {i}"
+            if not isinstance(layer, dict):
+                raise ConfigError(f"{lw} must be an object")
+            kind = layer.get("type")
+            m = _section(layer, "mixer", lw)
+            mw = lw + " mixer"
+            if kind == "attention":
+                _check_heads(m, mw)
+                _require(m, "scale", float, mw)
+                _check_rot(m, mw)
+                scaling = _section(m.get("rot") or {}, "scaling", mw + " rot", optional=True)
+                if scaling:
+                    for k in ("factor", "original", "fast", "slow"):
+                        if not (_require(scaling, k, float, mw + " rot.scaling") > 0):
+                            raise ConfigError(f"{mw}: rot.scaling.{k} must be positive")
+                    if m["rot"]["base"] <= 1:
+                        raise ConfigError(f"{mw}: a scaled rotation needs a base above 1")
+                mask = _section(m, "mask", mw, optional=True)
+                if mask is not None and _require(mask, "size", int, mw + " mask") <= 0:
+                    raise ConfigError(f"{mw}: mask.size must be positive")
+            elif kind == "lightning":
+                _positive_ints(m, ("heads", "dim", "vdim"), mw)
+                decay = m.get("decay")
+                if not isinstance(decay, list) or len(decay) != m["heads"] or \
+                        any(isinstance(v, bool) or not isinstance(v, (int, float)) for v in decay):
+                    raise ConfigError(f"{mw}: decay must list one number for each of the {m['heads']} heads, got {decay!r}")
+            else:
+                raise ConfigError(f"{lw}: unknown type {kind!r} (known: attention, lightning)")
+            mlp = layer.get("mlp")
+            if mlp is None:
+                continue
+            pw = lw + " mlp"
+            if not isinstance(mlp, dict) or mlp.get("kind") not in ("dense", "moe"):
+                raise ConfigError(f"{lw}: mlp must be null or of kind 'dense' or 'moe', got {mlp!r}")
+            if mlp["kind"] == "dense":
+                _positive_ints(mlp, ("ff",), pw)
+                if not (_require(mlp, "limit", float, pw) > 0):
+                    raise ConfigError(f"{pw}: limit must be positive")
+                continue
+            _positive_ints(_section(mlp, "expert", pw), ("ff",), pw + " expert")
+            r = _section(mlp, "router", pw)
+            _positive_ints(r, ("experts", "top"), pw + " router")
+            if r["top"] > r["experts"]:
+                raise ConfigError(f"{pw}: router cannot choose {r['top']} of {r['experts']} experts")
+            if "scale" in r:
+                _require(r, "scale", float, pw + " router")
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        d = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+             "layers": json.loads(json.dumps(list(self.layers)))}
+        if self.has_loop:
+            d["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return d

@@ -150,9 +150,11 @@ PYBIND11_MODULE(kvcm_core, m) {
       .def("lru_order", &PrefixCache::lru_order);
 
   py::class_<LayerGroupSpec>(m, "LayerGroupSpec")
-      .def(py::init([](int window) { LayerGroupSpec g; g.window = window; return g; }),
-           py::arg("window") = 0)
-      .def_readwrite("window", &LayerGroupSpec::window);
+      .def(py::init([](int window, int chunk) { LayerGroupSpec g; g.window = window; g.chunk = chunk; return g; }),
+           py::arg("window") = 0, py::arg("chunk") = 0)
+      .def("first_live", &LayerGroupSpec::first_live)
+      .def_readwrite("window", &LayerGroupSpec::window)
+      .def_readwrite("chunk", &LayerGroupSpec::chunk);
 
   py::class_<KVStats>(m, "KVStats")
       .def_readonly("num_blocks", &KVStats::num_blocks)
@@ -186,6 +188,7 @@ PYBIND11_MODULE(kvcm_core, m) {
       .def("max_seq_len", &KVManager::max_seq_len)
       .def("num_groups", &KVManager::num_groups)
       .def("group_window", [](const KVManager& k, int g) { return k.group(g).window; })
+      .def("group_chunk", [](const KVManager& k, int g) { return k.group(g).chunk; })
       .def("can_admit", &KVManager::can_admit)
       .def("admit", &KVManager::admit)
       .def("ensure", &KVManager::ensure)

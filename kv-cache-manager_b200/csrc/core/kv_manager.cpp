@@ -15,7 +15,7 @@ KVManager::KVManager(int num_blocks, int block_size, int max_seq_len,
   if (num_blocks_ < 0) throw std::invalid_argument("KVManager: num_blocks must not be negative");
   if (groups_.empty()) throw std::invalid_argument("KVManager: at least one layer group is needed");
   for (const auto& g : groups_)
-    if (g.window < 0) throw std::invalid_argument("KVManager: negative window");
+    if (g.window < 0 || g.chunk < 0) throw std::invalid_argument("KVManager: negative window or chunk");
 }
 
 void KVManager::start_tables(Sequence& seq) const {

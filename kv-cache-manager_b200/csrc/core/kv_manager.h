@@ -6,8 +6,9 @@
 //    request that is prefetched in portions holds only the pages its computed part needs
 //    (the reference's admit()+append_slot() always cover the whole token list);
 //  * a request has one page table per *layer group*.  A group is a set of layers with the
-//    same cache needs: all keys (window 0) or only the last `window` keys, in which case
-//    commit() gives back the pages that the window has passed.
+//    same cache needs: all keys (window 0), only the last `window` keys, or only the keys of the
+//    chunk that a position lies in (chunks of `chunk` positions, counted from the request's first):
+//    commit() gives back the pages that the window or the chunk has passed.
 #pragma once
 #include <cstdint>
 #include <memory>
@@ -21,6 +22,13 @@ namespace kvcm {
 
 struct LayerGroupSpec {
   int window = 0;        // 0: every key is kept; w > 0: only keys of the last w positions
+  int chunk = 0;         // c > 0: position i needs keys j >= i - i % c only
+  // The first key that a query at `pos` or later can still need.
+  int first_live(int pos) const {
+    int first = window > 0 && pos + 1 > window ? pos + 1 - window : 0;
+    if (chunk > 0 && pos - pos % chunk > first) first = pos - pos % chunk;
+    return first;
+  }
 };
 
 struct KVStats {

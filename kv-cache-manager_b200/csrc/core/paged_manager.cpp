@@ -11,9 +11,9 @@ PagedManager::PagedManager(int num_blocks, int block_size, int max_seq_len, bool
                            int watermark_blocks, std::vector<LayerGroupSpec> groups)
     : KVManager(num_blocks, block_size, max_seq_len, std::move(groups)),
       watermark_(watermark_blocks) {
-  if (prefix_caching && (groups_.size() != 1 || groups_[0].window != 0))
+  if (prefix_caching && (groups_.size() != 1 || groups_[0].window != 0 || groups_[0].chunk != 0))
     throw std::invalid_argument(
-        "prefix caching needs a single layer group that keeps every key (no window)");
+        "prefix caching needs a single layer group that keeps every key (no window, no chunks)");
   for (size_t g = 0; g < groups_.size(); ++g)
     pools_.push_back(std::make_unique<Pool>(num_blocks, block_size, prefix_caching));
 }
@@ -70,11 +70,10 @@ void PagedManager::commit(Sequence& seq) {
     }
   }
   for (size_t g = 0; g < pools_.size(); ++g) {
-    const int w = groups_[g].window;
-    if (w <= 0) continue;
-    // The next query sits at position >= num_computed and reads keys t > position - w, so every
-    // key below num_computed - w + 1 is dead; a page is given back once all its keys are.
-    const int first_live = std::max(0, seq.num_computed - w + 1);
+    if (groups_[g].window <= 0 && groups_[g].chunk <= 0) continue;
+    // The next query sits at position >= num_computed and reads keys t > position - window (or the
+    // keys of its own chunk), so every earlier key is dead; a page is given back once all its keys are.
+    const int first_live = groups_[g].first_live(seq.num_computed);
     const int dead_pages = std::min<int>(first_live / block_size_, seq.tables[g].size());
     for (int i = seq.window_freed[g]; i < dead_pages; ++i) {
       pools_[g]->cache.release(seq.tables[g][i]);

@@ -1,5 +1,5 @@
-// Pages on demand: a request holds ceil(len / B) pages per group (fewer once a window has
-// passed some), so the only waste is the unfilled tail of its last page.  Optional reuse of
+// Pages on demand: a request holds ceil(len / B) pages per group (fewer once a window or a
+// chunk has passed some), so the only waste is the unfilled tail of its last page.  Optional reuse of
 // equal prefixes through the PrefixCache.  Policy after the reference's PagedManager
 // (src/core/paged_manager.cpp:9-66).
 #pragma once

@@ -22,7 +22,7 @@ struct Sequence {
   int num_computed = 0;
 
   // tables[g][i] = physical page of logical page i in layer group g; -1 once a sliding
-  // window has passed the page and it was given back.
+  // window or the chunk has passed the page and it was given back.
   std::vector<std::vector<int32_t>> tables;
   std::vector<int32_t> window_freed;      // per group: leading logical pages already given back
   std::vector<uint64_t> page_hashes;      // chain hashes of the leading full pages (prefix cache)

@@ -11,7 +11,8 @@
 //           a second kernel.  With one partition the block writes the result itself (v1).
 // (Portions of more than one token: attention_tcgen05.cu and attention_prefill_mma.cu.)
 // Any head_dim that is a multiple of 16 up to 256, any page size, any number of heads and groups,
-// optional window (keys t > position - window).  Scores are scaled in float after the product;
+// optional window (keys t > position - window) or chunk (keys of the position's own chunk; the partitions then
+// split the chunk's part of the context, not all of it).  Scores are scaled in float after the product;
 // softmax by exp2 with log2(e) folded into the scale; probabilities are rounded to bfloat16 for
 // the P*V product, sums stay float.
 #include <cooperative_groups.h>
@@ -33,6 +34,7 @@ struct DecodeParams {
   float* part_o; float* part_ml;
   int nh, nkv, block_size, window, part_size, num_parts;
   int keep_first;                      // with a window: the first keep_first keys of a request stay visible to every row
+  int chunk;                           // > 0: only the keys of the position's own chunk of this many positions
   float scale_log2;                    // what a score is multiplied by on its way into exp2
   float cap_pre;                       // > 0: capped scores, s <- tanh(s * cap_pre) first (cap_pre = scale / cap, scale_log2 = cap * log2 e)
   const float* sink;                   // per head, or null: exp(sink) joins the denominator where the result is normalised
@@ -140,10 +142,10 @@ attn_decode_kernel(DecodeParams p) {
   const int g = lane >> 2, t4 = lane & 3;
 
   const int ctx = p.seq_ctx_len[seq];
-  const int lo = (p.window > 0 && ctx > p.window) ? ctx - p.window : 0;
-  const int pbeg = part * p.part_size;
+  const int lo = ctx > 0 ? first_visible(ctx - 1, p.window, p.chunk) : 0;
+  const int pbeg = (p.chunk > 0 ? lo / kKeyTile * kKeyTile : 0) + part * p.part_size;
   const int begin = max(lo, pbeg);
-  const int end = min(ctx, (part + 1) * p.part_size);
+  const int end = min(ctx, pbeg + p.part_size);
   // Kept first keys that lie below the window: [pbeg, kend) of this partition (kend <= lo <= begin).
   const int kend = p.keep_first > 0 ? min(min(p.keep_first, lo), end) : 0;
   const bool has_kept = kend > pbeg;
@@ -465,11 +467,13 @@ KVCM_API int kvcm_attention_decode_cluster_parts(void) { return kMaxClusterParts
 // merge runs inside a cluster (cluster_merge != 0 and num_parts <= kvcm_attention_decode_cluster_parts()).
 // `softcap` > 0: scaled scores are capped as cap * tanh(score / cap); `sink` (per head, optional): exp(sink)
 // joins the softmax's denominator.
-// `keep_first` > 0 (with a window): the first keep_first keys of every request stay visible.
+// `keep_first` > 0 (with a window): the first keep_first keys of every request stay visible.  `chunk` > 0: a row sees
+// only its own chunk of positions, and the num_parts partitions of part_size keys cover [chunk's first key rounded down
+// to a tile of 64, context).
 KVCM_API int kvcm_attention_decode_keep_bf16(const void* q, int q_stride, void* out, int out_stride,
                                              const void* k_cache, const void* v_cache, const int* block_tables,
                                              int max_blocks, const int* seq_ctx_len, int seqs, int nh, int nkv,
-                                             int hd, int block_size, float scale, int window, int keep_first, int part_size,
+                                             int hd, int block_size, float scale, int window, int keep_first, int chunk, int part_size,
                                              int num_parts, float* scratch, int cluster_merge, float softcap,
                                              const float* sink, void* stream) {
   if (seqs == 0) return 0;
@@ -481,6 +485,7 @@ KVCM_API int kvcm_attention_decode_keep_bf16(const void* q, int q_stride, void* 
     if (sm_count <= 0) sm_count = 148;
   }
   if (nkv <= 0 || nh % nkv || part_size <= 0 || part_size % kKeyTile || num_parts < 1) return KVCM_ERR_UNSUPPORTED;
+  if (chunk < 0 || (chunk > 0 && keep_first > 0)) return KVCM_ERR_UNSUPPORTED;
   if (cluster_merge && (num_parts < 2 || num_parts > kMaxClusterParts)) cluster_merge = 0;
   if (num_parts > 1 && !cluster_merge && scratch == nullptr) return KVCM_ERR_UNSUPPORTED;
   DecodeParams p;
@@ -490,6 +495,7 @@ KVCM_API int kvcm_attention_decode_keep_bf16(const void* q, int q_stride, void* 
   p.part_o = scratch; p.part_ml = scratch ? scratch + (size_t)seqs * nh * num_parts * hd : nullptr;
   p.nh = nh; p.nkv = nkv; p.block_size = block_size; p.window = window;
   p.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
+  p.chunk = chunk;
   p.part_size = part_size; p.num_parts = num_parts; p.cluster_merge = cluster_merge;
   p.scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
   p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
@@ -512,7 +518,7 @@ KVCM_API int kvcm_attention_decode_capped_bf16(const void* q, int q_stride, void
                                                int num_parts, float* scratch, int cluster_merge, float softcap,
                                                const float* sink, void* stream) {
   return kvcm_attention_decode_keep_bf16(q, q_stride, out, out_stride, k_cache, v_cache, block_tables, max_blocks, seq_ctx_len,
-                                         seqs, nh, nkv, hd, block_size, scale, window, 0, part_size, num_parts, scratch,
+                                         seqs, nh, nkv, hd, block_size, scale, window, 0, 0, part_size, num_parts, scratch,
                                          cluster_merge, softcap, sink, stream);
 }
 

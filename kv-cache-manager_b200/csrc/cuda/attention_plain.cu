@@ -12,6 +12,7 @@
 // the causal mask is the loop bound ctx = position + 1, o = (sum_t p_t v_t) / sum_t p_t.
 // With a window, `keep_first` > 0 keeps the first keep_first keys of the request visible to every row: the
 // keys walked are [0, min(keep_first, lo)) followed by the window [lo, ctx).
+// With `chunk` > 0 a row sees only the keys of its own chunk of positions (chunks counted from position 0).
 #include "common.cuh"
 
 namespace kvcm {
@@ -27,7 +28,7 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
                        const int* __restrict__ block_tables, int max_blocks,
                        const int* __restrict__ row_seq, const int* __restrict__ positions,
                        int nh, int nkv, int hd, int block_size, float scale, int window, float softcap,
-                       const float* __restrict__ sink, int keep_first) {
+                       const float* __restrict__ sink, int keep_first, int chunk) {
   extern __shared__ float smem[];
   float* qs = smem;                     // [hd]
   float* sc = qs + hd;                  // [kPlainChunk]
@@ -35,7 +36,7 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
   const int row = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const int kvh = h / (nh / nkv);
   const int ctx = positions[row] + 1;
-  const int lo = (window > 0 && ctx > window) ? ctx - window : 0;
+  const int lo = first_visible(ctx - 1, window, chunk);
   const int kept = min(keep_first, lo);          // keys [0, kept) come first, then [lo, ctx)
   const int total = kept + ctx - lo;
   const int* table = block_tables + size_t(row_seq[row]) * max_blocks;
@@ -102,7 +103,8 @@ template <typename T>
 int launch_attention_plain(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
                            const void* v_cache, const int* block_tables, int max_blocks,
                            const int* row_seq, const int* positions, int rows, int nh, int nkv, int hd,
-                           int block_size, float scale, int window, float softcap, const float* sink, int keep_first, cudaStream_t s) {
+                           int block_size, float scale, int window, float softcap, const float* sink, int keep_first, int chunk,
+                           cudaStream_t s) {
   if (rows == 0) return 0;
   if (hd > kPlainMaxDimsPerThread * kPlainThreads || nkv <= 0 || nh % nkv) return KVCM_ERR_UNSUPPORTED;
   const size_t smem = (size_t(hd) + kPlainChunk + 33) * sizeof(float);
@@ -110,7 +112,7 @@ int launch_attention_plain(const void* q, int q_stride, void* out, int out_strid
   attention_plain_kernel<T><<<grid, kPlainThreads, smem, s>>>(
       (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_cache, (const T*)v_cache, block_tables,
       max_blocks, row_seq, positions, nh, nkv, hd, block_size, scale, window, softcap, sink,
-      window > 0 && keep_first > 0 ? keep_first : 0);
+      window > 0 && keep_first > 0 ? keep_first : 0, chunk);
   return KVCM_LAUNCH_RESULT();
 }
 
@@ -123,21 +125,21 @@ using namespace kvcm;
       const int *block_tables, int max_blocks, const int *row_seq, const int *positions, int rows, int nh, int nkv, \
       int hd, int block_size, float scale, int window, float softcap, const float *sink
 
-KVCM_API int kvcm_attention_plain_keep_f32(KVCM_PLAIN_ARGS, int keep_first, void* stream) {
+KVCM_API int kvcm_attention_plain_keep_f32(KVCM_PLAIN_ARGS, int keep_first, int chunk, void* stream) {
   return launch_attention_plain<float>(q, q_stride, out, out_stride, k_cache, v_cache, block_tables, max_blocks, row_seq,
                                        positions, rows, nh, nkv, hd, block_size, scale, window, softcap, sink, keep_first,
-                                       (cudaStream_t)stream);
+                                       chunk, (cudaStream_t)stream);
 }
-KVCM_API int kvcm_attention_plain_keep_bf16(KVCM_PLAIN_ARGS, int keep_first, void* stream) {
+KVCM_API int kvcm_attention_plain_keep_bf16(KVCM_PLAIN_ARGS, int keep_first, int chunk, void* stream) {
   return launch_attention_plain<bf16>(q, q_stride, out, out_stride, k_cache, v_cache, block_tables, max_blocks, row_seq,
                                       positions, rows, nh, nkv, hd, block_size, scale, window, softcap, sink, keep_first,
-                                      (cudaStream_t)stream);
+                                      chunk, (cudaStream_t)stream);
 }
 KVCM_API int kvcm_attention_plain_f32(KVCM_PLAIN_ARGS, void* stream) {
   return kvcm_attention_plain_keep_f32(q, q_stride, out, out_stride, k_cache, v_cache, block_tables, max_blocks, row_seq,
-                                       positions, rows, nh, nkv, hd, block_size, scale, window, softcap, sink, 0, stream);
+                                       positions, rows, nh, nkv, hd, block_size, scale, window, softcap, sink, 0, 0, stream);
 }
 KVCM_API int kvcm_attention_plain_bf16(KVCM_PLAIN_ARGS, void* stream) {
   return kvcm_attention_plain_keep_bf16(q, q_stride, out, out_stride, k_cache, v_cache, block_tables, max_blocks, row_seq,
-                                        positions, rows, nh, nkv, hd, block_size, scale, window, softcap, sink, 0, stream);
+                                        positions, rows, nh, nkv, hd, block_size, scale, window, softcap, sink, 0, 0, stream);
 }

@@ -4,7 +4,8 @@
 // from the pages, K and V of the portion included (they were written before), so a portion may
 // start anywhere in a request.  The reference has no such kernel (it runs prefill rows through the
 // decode kernel, docs/design.md:113-114).  Any head_dim that is a multiple of 16 up to 256, any
-// page size, any number of heads and groups, optional window (keys t > position - window).
+// page size, any number of heads and groups, optional window (keys t > position - window) or
+// chunk (keys of the position's own chunk).
 // Scores are scaled in float after the product; softmax by exp2 with log2(e) folded into the
 // scale; probabilities are rounded to bfloat16 for the P*V product, sums stay float.
 #include "attention_mma.cuh"
@@ -21,6 +22,7 @@ struct PrefillParams {
   const int* seq_q_start; const int* seq_q_len; const int* seq_ctx_len;
   int nh, nkv, block_size, window;
   int keep_first;                   // with a window: the first keep_first keys of a request stay visible to every row
+  int chunk;                        // > 0: only the keys of a row's own chunk of this many positions
   float scale_log2;                 // what a score is multiplied by on its way into exp2
   float cap_pre;                    // > 0: capped scores, s <- tanh(s * cap_pre) first (cap_pre = scale / cap, scale_log2 = cap * log2 e)
   const float* sink;                // per head, or null: exp(sink) joins every row's denominator at the end
@@ -49,7 +51,7 @@ attn_prefill_kernel(PrefillParams p) {
   const int rows_here = min(BM, q_len - q0);
   const int pos0 = ctx - q_len + q0;                                // position of the tile's first row
   const int hi = pos0 + rows_here;                                  // keys [lo, hi) matter to the tile
-  const int lo = (p.window > 0) ? max(0, pos0 - p.window + 1) : 0;
+  const int lo = first_visible(pos0, p.window, p.chunk);
   const int* table = p.block_tables + size_t(seq) * p.max_blocks;
 
   for (int c = tid; c < BM * (HD / 8); c += kAttnThreads) {
@@ -78,7 +80,8 @@ attn_prefill_kernel(PrefillParams p) {
   const int row_pos[2] = {pos0 + warp * 16 + g, pos0 + warp * 16 + g + 8};   // positions of this thread's rows
   const bool warp_live = warp * 16 < rows_here;
   const int warp_last_pos = pos0 + min(warp * 16 + 15, rows_here - 1);
-  const int warp_first_lo = (p.window > 0) ? pos0 + warp * 16 - p.window + 1 : 0;
+  const int warp_first_lo = first_visible(pos0 + warp * 16, p.window, p.chunk), warp_last_lo = first_visible(warp_last_pos, p.window, p.chunk);
+  const int row_lo[2] = {first_visible(row_pos[0], p.window, p.chunk), first_visible(row_pos[1], p.window, p.chunk)};
 
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[HD / 8][4];
@@ -125,7 +128,7 @@ attn_prefill_kernel(PrefillParams p) {
       }
       // scale; mask only where the tile touches the diagonal, the window's edge or the key range's edge
       const bool needs_mask = t0 + kKeyTile - 1 > pos0 + warp * 16 || t0 < lo || p.keep_first > 0 ||
-                              (p.window > 0 && t0 <= warp_last_pos - p.window) || t0 + kKeyTile > hi;
+                              t0 < warp_last_lo || t0 + kKeyTile > hi;
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int n = 0; n < kKeyTile / 8; ++n)
@@ -135,7 +138,7 @@ attn_prefill_kernel(PrefillParams p) {
           if (needs_mask) {
             const int key = t0 + 8 * n + 2 * t4 + (j & 1);
             const int rp = row_pos[j >> 1];
-            const bool ok = key <= rp && key < hi && ((key >= lo && (p.window <= 0 || key > rp - p.window)) || key < p.keep_first);
+            const bool ok = key <= rp && key < hi && ((key >= lo && key >= row_lo[j >> 1]) || key < p.keep_first);
             v = ok ? v : -INFINITY;
           }
           s[n][j] = v;
@@ -223,9 +226,9 @@ KVCM_API int kvcm_attention_prefill_keep_bf16(const void* q, int q_stride, void*
                                               int max_blocks, const int* tile_seq, const int* tile_q0,
                                               const int* seq_q_start, const int* seq_q_len, const int* seq_ctx_len,
                                               int tiles, int nh, int nkv, int hd, int block_size, float scale,
-                                              int window, int keep_first, float softcap, const float* sink, void* stream) {
+                                              int window, int keep_first, int chunk, float softcap, const float* sink, void* stream) {
   if (tiles == 0) return 0;
-  if (nkv <= 0 || nh % nkv) return KVCM_ERR_UNSUPPORTED;
+  if (nkv <= 0 || nh % nkv || chunk < 0 || (chunk > 0 && keep_first > 0)) return KVCM_ERR_UNSUPPORTED;
   PrefillParams p;
   p.q = (const bf16*)q; p.q_stride = q_stride; p.out = (bf16*)out; p.out_stride = out_stride;
   p.k_cache = (const bf16*)k_cache; p.v_cache = (const bf16*)v_cache;
@@ -233,6 +236,7 @@ KVCM_API int kvcm_attention_prefill_keep_bf16(const void* q, int q_stride, void*
   p.seq_q_start = seq_q_start; p.seq_q_len = seq_q_len; p.seq_ctx_len = seq_ctx_len;
   p.nh = nh; p.nkv = nkv; p.block_size = block_size; p.window = window;
   p.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
+  p.chunk = chunk;
   p.scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
   p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   p.sink = sink;
@@ -253,5 +257,5 @@ KVCM_API int kvcm_attention_prefill_bf16(const void* q, int q_stride, void* out,
                                          int window, float softcap, const float* sink, void* stream) {
   return kvcm_attention_prefill_keep_bf16(q, q_stride, out, out_stride, k_cache, v_cache, block_tables, max_blocks, tile_seq,
                                           tile_q0, seq_q_start, seq_q_len, seq_ctx_len, tiles, nh, nkv, hd, block_size, scale,
-                                          window, 0, softcap, sink, stream);
+                                          window, 0, 0, softcap, sink, stream);
 }

@@ -22,8 +22,8 @@
 // of shared memory and 256 columns of tensor memory each); at 128 a block takes 192 KB.  Keys come from the pages, the portion's own
 // included (they were written before), so a portion may start anywhere in a request; masks: key <=
 // row's position, key > position - window (or key < keep_first: a window that keeps a request's first
-// keys; the tiles that hold them are walked before the window's own), key < end of the request's computed
-// part.  Scores are
+// keys; the tiles that hold them are walked before the window's own), key in the row's own chunk of positions
+// (`chunk` > 0), key < end of the request's computed part.  Scores are
 // scaled in float; softmax by exp2 with log2(e) folded into the scale; probabilities are rounded
 // to bfloat16 for the product with V, their sums stay float.
 // Every wait on an mbarrier is bounded; when one runs out the block records it
@@ -57,6 +57,7 @@ struct PrefillTcParams {
   const int* seq_q_start; const int* seq_q_len; const int* seq_ctx_len;
   int nh, nkv, block_size, window;
   int keep_first;                   // with a window: keys below this stay visible to every later row (0: none)
+  int chunk;                        // > 0: only the keys of a row's own chunk of this many positions
   float scale_log2;                 // what a score is multiplied by on its way into exp2
   float cap_pre;                    // > 0: scores are capped, s <- tanh(s * cap_pre) first (cap_pre = scale / cap and
                                     // scale_log2 = cap * log2(e))
@@ -122,7 +123,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
   const int rows_here = min(kFaRows, q_len - q0);
   const int pos0 = ctx - q_len + q0;                           // position of the block's first row
   const int hi = pos0 + rows_here;                             // keys [lo, hi) matter to the block
-  const int lo = (p.window > 0 && pos0 + 1 > p.window) ? pos0 + 1 - p.window : 0;
+  const int lo = first_visible(pos0, p.window, p.chunk);
+  const int last_lo = first_visible(pos0 + kFaRows - 1, p.window, p.chunk);   // first key of the block's last row
   const int j0 = lo / kFaKeys;
   // Kept first keys below the window's own tiles: n_keep tiles from key 0 come first, then tiles j0, j0 + 1, ...
   const int keep = (p.window > 0 && lo > 0 && p.keep_first > 0) ? min(p.keep_first, lo) : 0;
@@ -246,7 +248,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const int quarter = warp & 3;
     const int r = quarter * 32 + lane;
     const int pos = pos0 + r;                                  // rows beyond rows_here compute and store nothing
-    const int first = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;   // first key of the row
+    const int first = first_visible(pos, p.window, p.chunk);   // first key of the row
     const uint32_t lane_addr = tmem + (uint32_t(quarter * 32) << 16);
     float m = -INFINITY, l = 0.f;                              // m: the maximum the row currently scales by
     for (int n = 0; n < n_tiles; ++n) {
@@ -275,7 +277,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       const int kk = (p.window > 0 ? p.keep_first : 0) - key0;
       // Masks are needed only where the tile touches the diagonal, the window's edge or the end of
       // the keys; for every other tile (most of a long prompt) there is none.
-      const bool full = key0 + kFaKeys - 1 <= pos0 && (p.window <= 0 || key0 >= pos0 + kFaRows - p.window || kk >= kFaKeys);
+      const bool full = key0 + kFaKeys - 1 <= pos0 && (key0 >= last_lo || kk >= kFaKeys);
       float mx[2] = {-INFINITY, -INFINITY};
       if (full) {
         // eight chains of three-input maxima, four steps deep, instead of two chains of 32
@@ -456,10 +458,11 @@ KVCM_API int kvcm_attention_prefill_tcgen05_bf16(const void* q, int q_stride, in
                                                  const int* block_tables, int max_blocks, const int* tile_seq,
                                                  const int* tile_q0, const int* seq_q_start, const int* seq_q_len,
                                                  const int* seq_ctx_len, int tiles, int nh, int nkv, int hd,
-                                                 int block_size, float scale, int window, int keep_first, float softcap,
+                                                 int block_size, float scale, int window, int keep_first, int chunk, float softcap,
                                                  const float* sink, void* stream) {
   if (tiles == 0) return 0;
-  if (!kvcm_attention_tcgen05_supports_kv(hd, block_size, k_cache == v_cache) || nkv <= 0 || nh % nkv || keep_first < 0)
+  if (!kvcm_attention_tcgen05_supports_kv(hd, block_size, k_cache == v_cache) || nkv <= 0 || nh % nkv || keep_first < 0 ||
+      chunk < 0 || (chunk > 0 && keep_first > 0))
     return KVCM_ERR_UNSUPPORTED;
   if ((q_stride % 8) || (out_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(out) & 15) ||
       (reinterpret_cast<uintptr_t>(k_cache) & 15) || (reinterpret_cast<uintptr_t>(v_cache) & 15))
@@ -479,6 +482,7 @@ KVCM_API int kvcm_attention_prefill_tcgen05_bf16(const void* q, int q_stride, in
   p.seq_q_start = seq_q_start; p.seq_q_len = seq_q_len; p.seq_ctx_len = seq_ctx_len;
   p.nh = nh; p.nkv = nkv; p.block_size = block_size; p.window = window;
   p.keep_first = window > 0 ? keep_first : 0;
+  p.chunk = chunk;
   p.scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
   p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   p.sink = sink;

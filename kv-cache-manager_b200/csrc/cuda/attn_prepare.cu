@@ -5,12 +5,14 @@
 //   1. proj row [q: nh*dk | k: nkv*dk | v: nkv*dv] (float) + bias (optional)
 //   2. norm over the WHOLE q projection and over the whole k projection (optional):
 //        q <- wq * q / sqrt(mean(q^2) + eps),  k likewise with wk
+//      or norm per head before the rotation, with a weight of dk elements shared by the heads (`hq`, `hk`)
 //   3. rotation of the first `rot` dimensions of every q and k head in rotate-half pairs
 //        (i, i + rot/2), or with `interleaved` in neighbouring pairs (2i, 2i + 1),
-//        angle = position * inv_freq[i]   (rot == 0: none)
+//        angle = position * inv_freq[i]   (rot == 0: none); cosine and sine times `amplitude`
 //   4. norm per head, without weights (optional):  x <- x / sqrt(mean_head(x^2) + eps)
 //   5. values: `v_keep` (optional, float [rows, nkv*dv]) receives v as projected;
 //        `v_first` (optional, the same layout) mixes:  v <- v + lambda (v_first - v), evaluated as (1 - lambda) v + lambda v_first;
+//        `v_norm` divides every value head by its root mean square over dv (no weight);
 //        `v_inv_freq` (optional, dv/2 frequencies) turns every value head by its own position over all dv
 //        dimensions, in the same pairing as q and k (what is cached is the turned value; the reader turns
 //        the attention's output back by its own position)
@@ -26,7 +28,7 @@
 // in the usual grouped way (M*dk <= HD).
 //
 // All arithmetic is float; the order of steps is the parameter list's, so a mixer that wants the
-// norm before the rotation uses step 2 and one that wants it after uses step 4.
+// norm before the rotation uses step 2 (in one of its two forms) and one that wants it after uses step 4.
 #include "common.cuh"
 #include "pdl.cuh"
 
@@ -46,6 +48,9 @@ struct AttnPrepareParams {
   int interleaved;                   // pairs (2i, 2i+1) instead of (i, i + half)
   const float* v_inv_freq;           // [dv/2] or null
   int maps;                          // score maps per head (1: ordinary attention)
+  const float* hq; const float* hk;  // [dk] weights of the per-head norm ahead of the rotation, or null
+  int v_norm;                        // 1: every value head divided by its root mean square
+  float amplitude;                   // factor of the rotation's cosines and sines
 };
 
 __device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
@@ -71,7 +76,12 @@ attn_prepare_kernel(AttnPrepareParams p) {
   // the row's cosines and sines depend on nothing the step computes: before the wait
   if (half > 0 || vhalf > 0) {
     const float pos = float(p.positions[r]);
-    for (int j = tid; j < half; j += blockDim.x) sincosf(pos * p.inv_freq[j], &cs_table[half + j], &cs_table[j]);
+    for (int j = tid; j < half; j += blockDim.x) {
+      float sn, cs;
+      sincosf(pos * p.inv_freq[j], &sn, &cs);
+      cs_table[j] = cs * p.amplitude;
+      cs_table[half + j] = sn * p.amplitude;
+    }
     for (int j = tid; j < vhalf; j += blockDim.x) sincosf(pos * p.v_inv_freq[j], &vcs_table[vhalf + j], &vcs_table[j]);
   }
   pdl_wait();
@@ -111,6 +121,14 @@ attn_prepare_kernel(AttnPrepareParams p) {
         const float inv = is_q ? iq : ik;
         const float* w = is_q ? p.wq + size_t(u) * p.dk : p.wk + size_t(u - nqu) * p.dk;
         for (int i = lane; i < p.dk; i += 32) x[i] = x[i] * inv * w[i];
+        __syncwarp();
+      }
+      if (p.hq) {
+        float ss = 0.f;
+        for (int i = lane; i < p.dk; i += 32) ss = fmaf(x[i], x[i], ss);
+        const float f = 1.f / sqrtf(warp_sum(ss) / float(p.dk) + p.eps);
+        const float* w = is_q ? p.hq : p.hk;
+        for (int i = lane; i < p.dk; i += 32) x[i] = x[i] * f * w[i];
         __syncwarp();
       }
       for (int j = lane; j < half; j += 32) {
@@ -169,6 +187,13 @@ attn_prepare_kernel(AttnPrepareParams p) {
         __syncwarp();
       }
       if (slot < 0) continue;
+      if (p.v_norm) {
+        float ss = 0.f;
+        for (int i = lane; i < p.dv; i += 32) ss = fmaf(x[i], x[i], ss);
+        const float f = 1.f / sqrtf(warp_sum(ss) / float(p.dv) + p.eps);
+        for (int i = lane; i < p.dv; i += 32) x[i] *= f;
+        __syncwarp();
+      }
       if (vhalf > 0) {
         for (int j = lane; j < vhalf; j += 32) {
           const int ia = p.interleaved ? 2 * j : j, ib = p.interleaved ? 2 * j + 1 : j + vhalf;
@@ -189,7 +214,7 @@ template <typename T>
 int launch_attn_prepare(const AttnPrepareParams& p, int rows, cudaStream_t s) {
   if (rows == 0) return 0;
   if (p.rot % 2 || p.rot > p.dk || p.maps < 1 || p.HD < p.maps * p.dk || p.HD < p.dv || p.HD % 2 || (p.v_inv_freq && p.dv % 2) ||
-      (p.maps > 1 && p.wq))
+      (p.maps > 1 && p.wq) || (p.hq == nullptr) != (p.hk == nullptr))
     return KVCM_ERR_UNSUPPORTED;
   const size_t smem = size_t((p.nh + p.nkv) * p.maps * p.dk + p.nkv * p.dv + p.rot + (p.v_inv_freq ? p.dv : 0)) * sizeof(float);
   if (smem > 200 * 1024) return KVCM_ERR_UNSUPPORTED;
@@ -210,7 +235,8 @@ using namespace kvcm;
   const float *proj, int ldp, const float *bias, const float *wq, const float *wk, const int *positions,              \
       const float *inv_freq, int rot, int head_norm, float eps, float *v_keep, const float *v_first,                  \
       const float *lambda, const int *slot_mapping, int block_size, void *q_out, void *k_cache, void *v_cache,        \
-      int rows, int nh, int nkv, int dk, int dv, int HD, int interleaved, const float *v_inv_freq, int maps, void *stream
+      int rows, int nh, int nkv, int dk, int dv, int HD, int interleaved, const float *v_inv_freq, int maps, const float *hq, const float *hk, int v_norm,       \
+      float amplitude, void *stream
 
 static AttnPrepareParams make_params(KVCM_ATTN_PREPARE_ARGS) {
   (void)rows; (void)stream;
@@ -219,16 +245,17 @@ static AttnPrepareParams make_params(KVCM_ATTN_PREPARE_ARGS) {
   p.rot = inv_freq ? rot : 0; p.head_norm = head_norm; p.eps = eps; p.v_keep = v_keep; p.v_first = v_first; p.lambda = lambda;
   p.slot_mapping = slot_mapping; p.block_size = block_size; p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache;
   p.nh = nh; p.nkv = nkv; p.dk = dk; p.dv = dv; p.HD = HD; p.interleaved = interleaved; p.v_inv_freq = v_inv_freq; p.maps = maps;
+  p.hq = hq; p.hk = hk; p.v_norm = v_norm; p.amplitude = amplitude;
   return p;
 }
 
 KVCM_API int kvcm_attn_prepare_f32(KVCM_ATTN_PREPARE_ARGS) {
   return launch_attn_prepare<float>(make_params(proj, ldp, bias, wq, wk, positions, inv_freq, rot, head_norm, eps, v_keep,
                                                 v_first, lambda, slot_mapping, block_size, q_out, k_cache, v_cache, rows, nh,
-                                                nkv, dk, dv, HD, interleaved, v_inv_freq, maps, stream), rows, (cudaStream_t)stream);
+                                                nkv, dk, dv, HD, interleaved, v_inv_freq, maps, hq, hk, v_norm, amplitude, stream), rows, (cudaStream_t)stream);
 }
 KVCM_API int kvcm_attn_prepare_bf16(KVCM_ATTN_PREPARE_ARGS) {
   return launch_attn_prepare<bf16>(make_params(proj, ldp, bias, wq, wk, positions, inv_freq, rot, head_norm, eps, v_keep,
                                                v_first, lambda, slot_mapping, block_size, q_out, k_cache, v_cache, rows, nh,
-                                               nkv, dk, dv, HD, interleaved, v_inv_freq, maps, stream), rows, (cudaStream_t)stream);
+                                               nkv, dk, dv, HD, interleaved, v_inv_freq, maps, hq, hk, v_norm, amplitude, stream), rows, (cudaStream_t)stream);
 }

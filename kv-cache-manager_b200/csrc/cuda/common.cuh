@@ -42,6 +42,14 @@ __device__ __forceinline__ void rotate_pair(float a, float b, float cs, float sn
   rb = __fadd_rn(__fmul_rn(b, cs), __fmul_rn(a, sn));
 }
 
+// The first key that the query at `pos` sees: with a window the last `window` positions, with chunks
+// (positions [n * chunk, (n + 1) * chunk) see only each other) the start of its own chunk, else 0.
+__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
+  int first = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+  if (chunk > 0) first = max(first, pos - pos % chunk);
+  return first;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -221,7 +221,9 @@ __device__ __forceinline__ void dr_copy16(float* dst, const float* src, bool ok)
 //   kScanLinear       S <- g S + k (beta v)^T;  o = S^T q        (no correction by the state's own
 //                     read-out: the selective state-space recurrence with k = B, q = C, beta = dt, v = x)
 //   kScanLinearChannel  S <- diag(gd) S + k (beta v)^T;  o = S^T q   (the linear form with channel-wise decays:
-//                     gated linear attention; `beta` may be null and then counts as one)
+//                     gated linear attention)
+// In the linear forms `beta` may be null and then counts as one, and `silu` asks for SiLU of q, k and v as they are
+// staged (lightning attention: kScanLinear with a constant decay per head, g_ld = 0).
 // Where q, k and v of a row lie is given by `q_base`, `k_base`, `v_base` (floats from the row's start).
 struct ScanArgs {
   const float* qkv; int channels; int q_base, k_base, v_base;
@@ -231,6 +233,7 @@ struct ScanArgs {
   float* state; long long state_stride;
   const int* seq_q_start; const int* seq_q_len; const int* seq_state_slot;
   float* out; int heads, qk_heads, dk, dv;
+  int silu;                              // linear forms: q, k and v are projections that SiLU is still to be applied to
 };
 constexpr int kScanDelta = 0, kScanDeltaChannel = 1, kScanLinear = 2, kScanLinearChannel = 3;
 
@@ -356,6 +359,16 @@ delta_scan_kernel(const ScanArgs A) {
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
     __syncthreads();                                   // this tile has landed; the other buffer has been consumed
     if (t0 + TT < n) stage(buf ^ 1, t0 + TT);
+    if constexpr (LIN) {
+      if (A.silu) {                                     // once per tile, in place (elements that hold no data are zero and stay so)
+        for (int idx = threadIdx.x; idx < nt * DKP; idx += blockDim.x) {
+          (&qs[buf][0][0])[idx] = silu_f((&qs[buf][0][0])[idx]);
+          (&ks[buf][0][0])[idx] = silu_f((&ks[buf][0][0])[idx]);
+        }
+        for (int idx = threadIdx.x; idx < nt * DR_COLS; idx += blockDim.x) (&vs[buf][0][0])[idx] = silu_f((&vs[buf][0][0])[idx]);
+        __syncthreads();
+      }
+    }
     // One token: the state's step and the read-out.  `whole` false leaves the read-out as this lane's partial sum
     // (the caller adds the lanes of a column), so that the shuffles of several tokens can be in flight together.
     auto token = [&](int t, bool whole) -> float {
@@ -611,20 +624,22 @@ static int launch_scan(const ScanArgs& A, int rows, int seqs, cudaStream_t s) {
 
 // mode: 0 delta rule with one decay per head (g), 1 delta rule with a decay per head and key channel (gd),
 // 2 linear recurrence, 3 linear recurrence with a decay per head and key channel (see the kernel).  The row layout of `qkv` is given by the three bases.
+// g_ld 0: the same decays in every row.  `silu` (linear forms): q, k and v pass SiLU first.
 KVCM_API int kvcm_state_scan(int mode, const float* qkv, int channels, int q_base, int k_base, int v_base,
                              const float* beta, int beta_ld, const float* g, int g_ld, const float* gd, float* state,
                              long long state_stride, const int* seq_q_start, const int* seq_q_len,
                              const int* seq_state_slot, float* out, int rows, int seqs, int heads, int qk_heads, int dk,
-                             int dv, void* stream) {
+                             int dv, int silu, void* stream) {
   if (seqs == 0) return 0;
   if (dk < 1 || dk > 256 || qk_heads < 1 || heads % qk_heads) return KVCM_ERR_UNSUPPORTED;
   const bool channel = mode == kScanDeltaChannel || mode == kScanLinearChannel;
-  if (channel != (gd != nullptr) || (!channel && !g) || (!beta && mode != kScanLinearChannel)) return KVCM_ERR_UNSUPPORTED;
+  const bool linear = mode == kScanLinear || mode == kScanLinearChannel;
+  if (channel != (gd != nullptr) || (!channel && !g) || (!linear && (!beta || silu))) return KVCM_ERR_UNSUPPORTED;
   ScanArgs A;
   A.qkv = qkv; A.channels = channels; A.q_base = q_base; A.k_base = k_base; A.v_base = v_base;
   A.beta = beta; A.beta_ld = beta_ld; A.g = g; A.g_ld = g_ld; A.gd = gd; A.state = state; A.state_stride = state_stride;
   A.seq_q_start = seq_q_start; A.seq_q_len = seq_q_len; A.seq_state_slot = seq_state_slot; A.out = out;
-  A.heads = heads; A.qk_heads = qk_heads; A.dk = dk; A.dv = dv;
+  A.heads = heads; A.qk_heads = qk_heads; A.dk = dk; A.dv = dv; A.silu = silu;
   cudaStream_t s = (cudaStream_t)stream;
   if (mode == kScanDelta) return launch_scan<kScanDelta>(A, rows, seqs, s);
   if (mode == kScanDeltaChannel) return launch_scan<kScanDeltaChannel>(A, rows, seqs, s);
@@ -639,7 +654,7 @@ KVCM_API int kvcm_delta_scan(const float* qkv, int channels, const float* bg, fl
                              int rows, int seqs, int heads, int qk_heads, int dk, int dv, void* stream) {
   return kvcm_state_scan(kScanDelta, qkv, channels, 0, qk_heads * dk, 2 * qk_heads * dk, bg, 2 * heads, bg + heads, 2 * heads,
                          nullptr, state, state_stride, seq_q_start, seq_q_len, seq_state_slot, out, rows, seqs, heads,
-                         qk_heads, dk, dv, stream);
+                         qk_heads, dk, dv, 0, stream);
 }
 
 // ---------------------------------------------------- what the other recurrent mixers need around the scan
@@ -690,15 +705,15 @@ ssm_prepare_kernel(const T* __restrict__ raw, int ld, const float* __restrict__ 
 // Norm of the recurrent mixers' outputs in groups of `group` neighbouring elements, with a gate:
 //   v_i   = (o_i + skip_coef[i / head] * skip_i)  [* act(z_i) when the gate is applied ahead of the norm]
 //   out_i = storage( v_i / sqrt(mean_group(v^2) + eps) * w[i % wlen]  [* act(z_i) when it comes after] )
-// act: 0 = SiLU, 1 = sigmoid.  o float [rows, n]; z storage type (row stride ldz); skip float (row stride lds,
+// act: 0 = SiLU, 1 = sigmoid.  o float [rows, n]; z storage type or float (row stride ldz); skip float (row stride lds,
 // optional, with one coefficient per `head` elements).  One warp per (row, group).
 __device__ __forceinline__ float gate_act(float z, int act) {
   const float sg = 1.f / (1.f + expf(-z));
   return act == 0 ? z * sg : sg;
 }
-template <typename T>
+template <typename T, typename Z>
 __global__ void __launch_bounds__(128)
-group_rms_gate_kernel(const float* __restrict__ o, const T* __restrict__ z, int ldz, const float* __restrict__ skip, int lds,
+group_rms_gate_kernel(const float* __restrict__ o, const Z* __restrict__ z, int ldz, const float* __restrict__ skip, int lds,
                       const float* __restrict__ skip_coef, int head, const float* __restrict__ w, int wlen,
                       T* __restrict__ out, int n, int group, int gate_first, int act, float eps) {
   const int row = blockIdx.x;
@@ -731,9 +746,9 @@ group_rms_gate_kernel(const float* __restrict__ o, const T* __restrict__ z, int 
 
 // The same for groups of more than 256 elements: one block per (row, group), so that a long group's
 // loads are in flight together instead of one warp walking it.
-template <typename T>
+template <typename T, typename Z>
 __global__ void __launch_bounds__(256)
-group_rms_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ z, int ldz, const float* __restrict__ skip,
+group_rms_gate_wide_kernel(const float* __restrict__ o, const Z* __restrict__ z, int ldz, const float* __restrict__ skip,
                            int lds, const float* __restrict__ skip_coef, int head, const float* __restrict__ w, int wlen,
                            T* __restrict__ out, int n, int group, int gate_first, int act, float eps) {
   __shared__ float scratch[33];
@@ -770,7 +785,7 @@ group_rms_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ z,
   }
 }
 
-template <typename T>
+template <typename T, typename Z>
 static int launch_group_rms_gate(const float* o, const void* z, int ldz, const float* skip, int lds, const float* skip_coef,
                                  int head, const float* w, int wlen, void* out, int rows, int n, int group, int gate_first,
                                  int act, float eps, cudaStream_t s) {
@@ -778,11 +793,11 @@ static int launch_group_rms_gate(const float* o, const void* z, int ldz, const f
   if (group < 1 || n % group || wlen < 1 || (skip && head < 1)) return KVCM_ERR_UNSUPPORTED;
   const int groups = n / group;
   if (group > 256 && groups <= 65535) {
-    group_rms_gate_wide_kernel<T><<<dim3(rows, groups), 256, 0, s>>>(o, (const T*)z, ldz, skip, lds, skip_coef, head, w, wlen,
+    group_rms_gate_wide_kernel<T, Z><<<dim3(rows, groups), 256, 0, s>>>(o, (const Z*)z, ldz, skip, lds, skip_coef, head, w, wlen,
                                                                       (T*)out, n, group, gate_first, act, eps);
     return KVCM_LAUNCH_RESULT();
   }
-  group_rms_gate_kernel<T><<<dim3(rows, (groups + 3) / 4), 128, 0, s>>>(o, (const T*)z, ldz, skip, lds, skip_coef, head, w, wlen,
+  group_rms_gate_kernel<T, Z><<<dim3(rows, (groups + 3) / 4), 128, 0, s>>>(o, (const Z*)z, ldz, skip, lds, skip_coef, head, w, wlen,
                                                                        (T*)out, n, group, gate_first, act, eps);
   return KVCM_LAUNCH_RESULT();
 }
@@ -791,11 +806,15 @@ static int launch_group_rms_gate(const float* o, const void* z, int ldz, const f
   const float *o, const void *z, int ldz, const float *skip, int lds, const float *skip_coef, int head, const float *w, \
       int wlen, void *out, int rows, int n, int group, int gate_first, int act, float eps, void *stream
 KVCM_API int kvcm_group_rms_gate_f32(KVCM_GROUP_RMS_ARGS) {
-  return launch_group_rms_gate<float>(o, z, ldz, skip, lds, skip_coef, head, w, wlen, out, rows, n, group, gate_first, act, eps,
+  return launch_group_rms_gate<float, float>(o, z, ldz, skip, lds, skip_coef, head, w, wlen, out, rows, n, group, gate_first, act, eps,
                                       (cudaStream_t)stream);
 }
 KVCM_API int kvcm_group_rms_gate_bf16(KVCM_GROUP_RMS_ARGS) {
-  return launch_group_rms_gate<bf16>(o, z, ldz, skip, lds, skip_coef, head, w, wlen, out, rows, n, group, gate_first, act, eps,
+  return launch_group_rms_gate<bf16, bf16>(o, z, ldz, skip, lds, skip_coef, head, w, wlen, out, rows, n, group, gate_first, act, eps,
+                                     (cudaStream_t)stream);
+}
+KVCM_API int kvcm_group_rms_gate_zf32_bf16(KVCM_GROUP_RMS_ARGS) {
+  return launch_group_rms_gate<bf16, float>(o, z, ldz, skip, lds, skip_coef, head, w, wlen, out, rows, n, group, gate_first, act, eps,
                                      (cudaStream_t)stream);
 }
 

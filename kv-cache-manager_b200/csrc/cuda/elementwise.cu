@@ -1,6 +1,6 @@
 // Row-wise kernels of the forward pass: embedding gather, RMSNorm fused with the residual add
 // that precedes it, rotary position encoding fused with the write of K and V into cache pages,
-// and SiLU(gate)*up.  Each is instantiated for float (the true 32-bit path) and bfloat16.
+// and the gated activations (SiLU(gate)*up and its kin).  Each is instantiated for float (the true 32-bit path) and bfloat16.
 // Statistics, angles and the residual stream are always float.
 //
 // Formulas after the reference's kernels (src/cuda/kernels.cu:27-88, src/cuda/kv_cache.cu:19-38);
@@ -8,6 +8,7 @@
 #include <algorithm>
 
 #include "common.cuh"
+#include "gated_act.cuh"
 #include "pdl.cuh"
 
 namespace kvcm {
@@ -311,24 +312,23 @@ rope_cache_table_kernel(bf16* __restrict__ qkv, int row_stride, const float* __r
   *reinterpret_cast<uint4*>(dst + half + j0) = vb;
 }
 
-// --------------------------------------------------------------------------- SiLU(g) * u
-// gate = columns [0, I) of the fused product, up = columns [I, 2I).  silu is rounded to the
-// storage type before the product (src/cuda/kernels.cu:72-82).
-template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
+// ------------------------------------------------- gate and up of a gated feed-forward: SiLU(g) * u and its kin
+// gate = columns [0, I) of the fused product, up = columns [I, 2I) (activations: gated_act.cuh; SiLU is rounded
+// to the storage type before the product, src/cuda/kernels.cu:72-82).
+template <typename T, int KIND>
+__global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, GatedAct act) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   const int i = blockIdx.y * blockDim.x + threadIdx.x;
   if (i >= inter) return;
   const T* g = gate_up + size_t(t) * 2 * inter;
-  const float x = ldf(g + i);
-  const float s = Store<T>::round(x / (1.f + expf(-x)));
-  stf(out + size_t(t) * inter + i, s * ldf(g + inter + i));
+  stf(out + size_t(t) * inter + i, gated_act<KIND, T>(ldf(g + i), ldf(g + inter + i), act));
 }
 
 // bfloat16, width a multiple of 8: eight elements per thread through 16-byte loads and stores.
-__global__ void silu_mul_vec_kernel(const bf16* __restrict__ gate_up, bf16* __restrict__ out, int inter) {
+template <int KIND>
+__global__ void gated_act_vec_kernel(const bf16* __restrict__ gate_up, bf16* __restrict__ out, int inter, GatedAct act) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -344,22 +344,18 @@ __global__ void silu_mul_vec_kernel(const bf16* __restrict__ gate_up, bf16* __re
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const float2 x = __bfloat1622float2(gp[k]), u = __bfloat1622float2(up[k]);
-    const float s0 = Store<bf16>::round(x.x / (1.f + expf(-x.x)));
-    const float s1 = Store<bf16>::round(x.y / (1.f + expf(-x.y)));
-    op[k] = __floats2bfloat162_rn(s0 * u.x, s1 * u.y);
+    op[k] = __floats2bfloat162_rn(gated_act<KIND, bf16>(x.x, u.x, act), gated_act<KIND, bf16>(x.y, u.y, act));
   }
   *reinterpret_cast<uint4*>(out + size_t(t) * inter + i) = ov;
 }
 
-template <typename T>
-int launch_silu_mul(const T* gate_up, T* out, int rows, int inter, cudaStream_t s) {
-  return pdl_launch(silu_mul_kernel<T>, dim3(rows, (inter + 255) / 256), dim3(256), 0, s, gate_up, out, inter);
-}
-template <>
-int launch_silu_mul<bf16>(const bf16* gate_up, bf16* out, int rows, int inter, cudaStream_t s) {
-  if ((inter % 8) == 0 && ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0)
-    return pdl_launch(silu_mul_vec_kernel, dim3(rows, (inter / 8 + 255) / 256), dim3(256), 0, s, gate_up, out, inter);
-  return pdl_launch(silu_mul_kernel<bf16>, dim3(rows, (inter + 255) / 256), dim3(256), 0, s, gate_up, out, inter);
+template <typename T, int KIND>
+int launch_gated_act(const T* gate_up, T* out, int rows, int inter, GatedAct act, cudaStream_t s) {
+  if constexpr (sizeof(T) == 2) {
+    if ((inter % 8) == 0 && ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0)
+      return pdl_launch(gated_act_vec_kernel<KIND>, dim3(rows, (inter / 8 + 255) / 256), dim3(256), 0, s, gate_up, out, inter, act);
+  }
+  return pdl_launch(gated_act_kernel<T, KIND>, dim3(rows, (inter + 255) / 256), dim3(256), 0, s, gate_up, out, inter, act);
 }
 
 // Gathers rows of a [*, width] matrix of T into a dense [n, width] matrix (used for the rows
@@ -456,7 +452,14 @@ using namespace kvcm;
   KVCM_API int kvcm_silu_mul_##SUFFIX(const void* gate_up, void* out, int rows, int inter,            \
                                       void* stream) {                                                 \
     if (rows == 0) return 0;                                                                          \
-    return launch_silu_mul<T>((const T*)gate_up, (T*)out, rows, inter, (cudaStream_t)stream);         \
+    return launch_gated_act<T, kGatedSilu>((const T*)gate_up, (T*)out, rows, inter, GatedAct{},       \
+                                           (cudaStream_t)stream);                                     \
+  }                                                                                                   \
+  KVCM_API int kvcm_clamped_gate_##SUFFIX(const void* gate_up, void* out, int rows, int inter,        \
+                                          float limit, float alpha, void* stream) {                   \
+    if (rows == 0) return 0;                                                                          \
+    return launch_gated_act<T, kGatedClamped>((const T*)gate_up, (T*)out, rows, inter,                \
+                                              GatedAct{limit, alpha}, (cudaStream_t)stream);          \
   }                                                                                                   \
   KVCM_API int kvcm_gather_rows_##SUFFIX(const void* src, const int* rows, void* dst, int n,          \
                                          int width, void* stream) {                                   \

@@ -41,6 +41,7 @@
 // quad owns k = 8t..8t+7), which makes every shared-memory read of W and X a 16-byte vector.
 // The reference calls cuBLAS here (src/model/llama.cpp:45-52).
 #include "common.cuh"
+#include "gated_act.cuh"
 #include "pdl.cuh"
 
 namespace kvcm {
@@ -75,7 +76,8 @@ __device__ int g_stream_skip_stage = -1;
 //              into the row's cache page slot.  Bit-for-bit what the separate product + rotary +
 //              cache-write kernels produce.
 //  kSiluMul  : the 16 weight rows are 8 gate rows i..i+7 and the 8 up rows I+i..: y[m][i] =
-//              round(round(silu(round(gate))) * round(up)), as the separate activation kernel.
+//              round(round(silu(round(gate))) * round(up)), as the separate activation kernel (or the clamped
+//              form of gated_act.cuh, `gate_kind`).
 //  kResidual : resid[m][n] += round(sum) (the float residual stream, in place; the sum rounded to
 //              bfloat16 as the plain product would store it), ss_out[tile][m] = the sum over the
 //              tile's 16 columns of the new resid[m][n]^2 (what the next norm needs of this tile),
@@ -104,6 +106,8 @@ struct StreamParams {
   const float* ss_in; int ss_tiles; float eps;
   // kStore: 1 = the stored value is max(y, 0)^2 of the rounded sum y (an ungated feed-forward's activation)
   int relu_sq;
+  // kSiluMul: which activation joins gate and up (GatedKind; 0 counts as SiLU)
+  int gate_kind; GatedAct gate_act;
 };
 
 __device__ __forceinline__ uint32_t s32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
@@ -505,8 +509,9 @@ gemm_stream_kernel(StreamParams p) {
         const float xa = Store<bf16>::round(total_of(pr, m) * r);   // what the plain product stores
         const float xb = Store<bf16>::round(total_of(pr + 8, m) * r);
         if constexpr (EPI == kSiluMul) {
-          const float sl = Store<bf16>::round(xa / (1.f + expf(-xa)));
-          stf(Y + size_t(m) * p.ldy + 8 * tile + pr, sl * xb);
+          const float v = p.gate_kind == kGatedClamped ? gated_act<kGatedClamped, bf16>(xa, xb, p.gate_act)
+                                                       : gated_act<kGatedSilu, bf16>(xa, xb, p.gate_act);
+          stf(Y + size_t(m) * p.ldy + 8 * tile + pr, v);
         } else {
           const int head = tile / p.pair_blocks;
           const int j = 8 * (tile - head * p.pair_blocks) + pr;
@@ -713,9 +718,8 @@ KVCM_API int kvcm_qkv_rope_cache_bf16(const void* X, const void* Wqkv, void* Yq,
 // Fused input side of a gated feed-forward: act[M, I] = silu(X Wg^T) * (X Wu^T) with Wg, Wu the
 // two halves of W [2I, K] (gate rows first).  Needs I a multiple of 8.  With ss_in: both products
 // scaled per row first (see kvcm_qkv_rope_cache_scaled_bf16): the norm in front of the feed-forward.
-KVCM_API int kvcm_gate_up_silu_scaled_bf16(const void* X, const float* ss_in, int ss_tiles, float eps, const void* W,
-                                           void* Y, int M, int I, int K, int ldx, int ldw, int ldy, int sm_count,
-                                           void* stream) {
+static int gate_up_stream(const void* X, const float* ss_in, int ss_tiles, float eps, const void* W, void* Y, int M, int I, int K,
+                          int ldx, int ldw, int ldy, int sm_count, int kind, GatedAct act, void* stream) {
   if (M == 0) return 0;
   if ((I % 8) || !stream_ok(M, 2 * I, K, sm_count, false) || (ldw % 8) || (ldx % 8)) return KVCM_ERR_UNSUPPORTED;
   if ((reinterpret_cast<uintptr_t>(W) & 15) || (reinterpret_cast<uintptr_t>(X) & 15)) return KVCM_ERR_UNSUPPORTED;
@@ -725,8 +729,19 @@ KVCM_API int kvcm_gate_up_silu_scaled_bf16(const void* X, const float* ss_in, in
   p.ss_in = ss_in; p.ss_tiles = ss_tiles; p.eps = eps;
   p.Y = Y; p.ldy = ldy;
   p.pair_blocks = I / 8; p.group_stride = 0; p.pair_offset = I;
+  p.gate_kind = kind; p.gate_act = act;
   cudaStream_t s = (cudaStream_t)stream;
   return M <= 8 ? launch_stream<1, bf16, kSiluMul>(p, sm_count, s) : launch_stream<2, bf16, kSiluMul>(p, sm_count, s);
+}
+KVCM_API int kvcm_gate_up_silu_scaled_bf16(const void* X, const float* ss_in, int ss_tiles, float eps, const void* W,
+                                           void* Y, int M, int I, int K, int ldx, int ldw, int ldy, int sm_count,
+                                           void* stream) {
+  return gate_up_stream(X, ss_in, ss_tiles, eps, W, Y, M, I, K, ldx, ldw, ldy, sm_count, kGatedSilu, GatedAct{}, stream);
+}
+// The same with the clamped activation (no row scale).
+KVCM_API int kvcm_gate_up_clamped_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw, int ldy,
+                                       float limit, float alpha, int sm_count, void* stream) {
+  return gate_up_stream(X, nullptr, 0, 0.f, W, Y, M, I, K, ldx, ldw, ldy, sm_count, kGatedClamped, GatedAct{limit, alpha}, stream);
 }
 
 KVCM_API int kvcm_gate_up_silu_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw,

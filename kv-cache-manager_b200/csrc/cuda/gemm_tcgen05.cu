@@ -17,6 +17,7 @@
 // is a multiple of 8 work.  Every wait on an mbarrier is bounded; when one runs out the block
 // records it (kvcm_tcgen05_error), stops waiting, frees its tensor memory and leaves.
 // The reference calls cuBLAS for these products (src/model/llama.cpp:45-52).
+#include "gated_act.cuh"
 #include "tcgen05_common.cuh"
 
 namespace kvcm {
@@ -30,11 +31,12 @@ __device__ int g_tcgen05_error = 0;
 // GATED: W is [2N, K], gate rows first; a tile's 256 accumulator columns are 128 gate columns
 // n0..n0+127 and the 128 up columns N+n0.., and the epilogue stores
 // y[m][n] = round(round(silu(round(gate))) * round(up)) -- the roundings of the separate product
-// and activation kernels -- so the [M, 2N] intermediate never goes to memory.
-template <typename OutT, int BN, bool GATED>
+// and activation kernels -- so the [M, 2N] intermediate never goes to memory.  (GATED is a GatedKind: SiLU or the
+// clamped activation, gated_act.cuh.)
+template <typename OutT, int BN, int GATED>
 __global__ void __launch_bounds__(kTcThreads)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                    OutT* __restrict__ Y, int M, int N, int K, int ldy) {
+                    OutT* __restrict__ Y, int M, int N, int K, int ldy, GatedAct act) {
   static_assert(!GATED || BN == 256, "the gated tile is 128 + 128 columns");
   constexpr int BNOUT = GATED ? BN / 2 : BN;                   // output columns per tile
   constexpr int kBBytes = BN * kTcBK * 2;
@@ -156,7 +158,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
       }
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       const int row = m0 + quarter * 32 + lane;
-      if constexpr (GATED) {
+      if constexpr (GATED != kGatedNone) {
 #pragma unroll 1
         for (int c = 0; c < BNOUT / 32; ++c) {
           uint32_t g[32], u[32];
@@ -171,8 +173,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               const float xa = Store<bf16>::round(__uint_as_float(g[i])), xb = Store<bf16>::round(__uint_as_float(u[i]));
-              const float sl = Store<bf16>::round(xa / (1.f + expf(-xa)));
-              const bf16 y = __float2bfloat16_rn(sl * xb);
+              const bf16 y = __float2bfloat16_rn(gated_act<GATED, bf16>(xa, xb, act));
               if (i & 1) h2[i / 2].y = y; else h2[i / 2].x = y;
             }
             if (col0 + 32 <= N && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
@@ -241,9 +242,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 // ---------------------------------------------------------------------------------- host
 
 // GATED: N is the number of output columns; W has 2N rows.
-template <typename OutT, int BN, bool GATED = false>
+template <typename OutT, int BN, int GATED = kGatedNone>
 int launch_tcgen05_bn(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                      int sm_count, cudaStream_t s) {
+                      int sm_count, cudaStream_t s, GatedAct act = GatedAct{}) {
   CUtensorMap mx, mw;
   int rc = tc5::make_map(&mx, X, M, K, ldx, kTcBM);
   if (rc) return rc;
@@ -259,7 +260,7 @@ int launch_tcgen05_bn(const void* X, const void* W, void* Y, int M, int N, int K
   }
   constexpr int BNOUT = GATED ? BN / 2 : BN;
   const int tiles = ((N + BNOUT - 1) / BNOUT) * ((M + kTcBM - 1) / kTcBM);
-  kernel<<<dim3(tiles < sm_count ? tiles : sm_count), kTcThreads, smem, s>>>(mx, mw, reinterpret_cast<OutT*>(Y), M, N, K, ldy);
+  kernel<<<dim3(tiles < sm_count ? tiles : sm_count), kTcThreads, smem, s>>>(mx, mw, reinterpret_cast<OutT*>(Y), M, N, K, ldy, act);
   return KVCM_LAUNCH_RESULT();
 }
 
@@ -287,8 +288,9 @@ using namespace kvcm;
 
 // act[M, I] = silu(X Wg^T) * (X Wu^T) with Wg, Wu the halves of W [2I, K] (gate rows first), the
 // roundings of the separate product and activation kernels; bfloat16.
-KVCM_API int kvcm_gate_up_silu_tcgen05_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx,
-                                            int ldw, int ldy, void* stream) {
+template <int KIND>
+static int gate_up_tcgen05(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw, int ldy, GatedAct act,
+                           void* stream) {
   if (M == 0 || I == 0) return 0;
   if (M < 1 || I < 1 || K < 8 || (K % 8) || (ldx % 8) || (ldw % 8)) return KVCM_ERR_UNSUPPORTED;
   if ((reinterpret_cast<uintptr_t>(X) & 15) || (reinterpret_cast<uintptr_t>(W) & 15)) return KVCM_ERR_UNSUPPORTED;
@@ -296,7 +298,16 @@ KVCM_API int kvcm_gate_up_silu_tcgen05_bf16(const void* X, const void* W, void* 
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   if (sms <= 0) sms = 148;
-  return launch_tcgen05_bn<bf16, 256, true>(X, W, Y, M, I, K, ldx, ldw, ldy, sms, (cudaStream_t)stream);
+  return launch_tcgen05_bn<bf16, 256, KIND>(X, W, Y, M, I, K, ldx, ldw, ldy, sms, (cudaStream_t)stream, act);
+}
+KVCM_API int kvcm_gate_up_silu_tcgen05_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx,
+                                            int ldw, int ldy, void* stream) {
+  return gate_up_tcgen05<kGatedSilu>(X, W, Y, M, I, K, ldx, ldw, ldy, GatedAct{}, stream);
+}
+// The same with the clamped activation.
+KVCM_API int kvcm_gate_up_clamped_tcgen05_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw,
+                                               int ldy, float limit, float alpha, void* stream) {
+  return gate_up_tcgen05<kGatedClamped>(X, W, Y, M, I, K, ldx, ldw, ldy, GatedAct{limit, alpha}, stream);
 }
 
 KVCM_API int kvcm_gemm_tcgen05_supports(int M, int N, int K, int ldx, int ldw) {

@@ -13,7 +13,8 @@
 //   diff_combine   per row and head, from the two maps' attention outputs a1, a2 (heads 2h, 2h+1 of the attention
 //                  kernel's output, padded heads of HD):  o = a1 - lambda a2;  o <- o / sqrt(mean(o^2) + eps) * post
 //                  over the head's dv values;  o <- o * sigmoid(gate logit of the head);  storage type out
-//   gate_mul       out = x * sigmoid(gate logits), element by element (gate logits float32 with a row stride)
+//   gate_mul       out = x * sigmoid(gate logits), element by element (gate logits float32 with a row stride; x may be the
+//                  attention kernel's padded heads)
 //
 // All arithmetic is float32 in both storage types.
 #include "common.cuh"
@@ -235,25 +236,27 @@ diff_combine_kernel(const T* __restrict__ a, const float* __restrict__ gate, int
   }
 }
 
-// out = x * sigmoid(gate): four neighbouring elements a thread where the rows allow 8- and 16-byte accesses.
+// out = x * sigmoid(gate): four neighbouring elements a thread where the rows allow 8- and 16-byte accesses.  x holds
+// heads of HD elements of which the first dv count (HD == dv: plain rows); gate and out have them side by side.
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
-gate_mul_kernel(const T* __restrict__ x, const float* __restrict__ gate, int ldg, T* __restrict__ out, int n) {
+gate_mul_kernel(const T* __restrict__ x, const float* __restrict__ gate, int ldg, T* __restrict__ out, int n, int dv, int HD) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x;
-  const T* xr = x + size_t(row) * n;
+  const T* xr = x + size_t(row) * (n / dv) * HD;
   const float* gr = gate + size_t(row) * ldg;
   T* dst = out + size_t(row) * n;
-  if constexpr (V == 4) {
-    for (int i = 4 * threadIdx.x; i < n; i += 4 * blockDim.x) {
+  for (int i = V * threadIdx.x; i < n; i += V * blockDim.x) {
+    const T* src = xr + (HD == dv ? i : i + (i / dv) * (HD - dv));
+    if constexpr (V == 4) {
       const float4 g = *reinterpret_cast<const float4*>(gr + i);
-      const float2 a = Pair<T>::load(xr + i), b = Pair<T>::load(xr + i + 2);
+      const float2 a = Pair<T>::load(src), b = Pair<T>::load(src + 2);
       Pair<T>::store(dst + i, a.x / (1.f + expf(-g.x)), a.y / (1.f + expf(-g.y)));
       Pair<T>::store(dst + i + 2, b.x / (1.f + expf(-g.z)), b.y / (1.f + expf(-g.w)));
+    } else {
+      stf(dst + i, ldf(src) / (1.f + expf(-gr[i])));
     }
-  } else {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) stf(dst + i, ldf(xr + i) / (1.f + expf(-gr[i])));
   }
 }
 
@@ -316,17 +319,19 @@ KVCM_API int kvcm_diff_combine_bf16(KVCM_DIFF_COMBINE_ARGS) {
 }
 
 template <typename T>
-static int launch_gate_mul(const void* x, const float* gate, int ldg, void* out, int rows, int n, void* stream) {
+static int launch_gate_mul(const void* x, const float* gate, int ldg, void* out, int rows, int n, int dv, int HD, void* stream) {
   if (rows == 0) return 0;
-  const bool vec = (n & 3) == 0 && (ldg & 3) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
+  if (dv < 1 || HD < dv || n % dv) return KVCM_ERR_UNSUPPORTED;
+  const bool vec = (n & 3) == 0 && (ldg & 3) == 0 && (HD == dv || ((dv & 3) == 0 && (HD & 3) == 0)) &&
+                   (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(gate) & 15) == 0;
   if (vec)
-    return pdl_launch(gate_mul_kernel<T, 4>, dim3(rows), dim3(256), 0, (cudaStream_t)stream, (const T*)x, gate, ldg, (T*)out, n);
-  return pdl_launch(gate_mul_kernel<T, 1>, dim3(rows), dim3(256), 0, (cudaStream_t)stream, (const T*)x, gate, ldg, (T*)out, n);
+    return pdl_launch(gate_mul_kernel<T, 4>, dim3(rows), dim3(256), 0, (cudaStream_t)stream, (const T*)x, gate, ldg, (T*)out, n, dv, HD);
+  return pdl_launch(gate_mul_kernel<T, 1>, dim3(rows), dim3(256), 0, (cudaStream_t)stream, (const T*)x, gate, ldg, (T*)out, n, dv, HD);
 }
-KVCM_API int kvcm_gate_mul_f32(const void* x, const float* gate, int ldg, void* out, int rows, int n, void* stream) {
-  return launch_gate_mul<float>(x, gate, ldg, out, rows, n, stream);
+KVCM_API int kvcm_gate_mul_f32(const void* x, const float* gate, int ldg, void* out, int rows, int n, int dv, int HD, void* stream) {
+  return launch_gate_mul<float>(x, gate, ldg, out, rows, n, dv, HD, stream);
 }
-KVCM_API int kvcm_gate_mul_bf16(const void* x, const float* gate, int ldg, void* out, int rows, int n, void* stream) {
-  return launch_gate_mul<bf16>(x, gate, ldg, out, rows, n, stream);
+KVCM_API int kvcm_gate_mul_bf16(const void* x, const float* gate, int ldg, void* out, int rows, int n, int dv, int HD, void* stream) {
+  return launch_gate_mul<bf16>(x, gate, ldg, out, rows, n, dv, HD, stream);
 }

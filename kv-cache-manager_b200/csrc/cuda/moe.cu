@@ -7,7 +7,8 @@
 //            router matrix, if present, is a per-row gate: sigmoid of its logit.  Options: scores
 //            sigmoid(z) instead of the softmax; a `correction` per expert that is added to the scores
 //            for the choice only (choice scores may then be negative; the weights use the scores
-//            themselves); a group's score as the sum of its two largest choice scores.
+//            themselves); a group's score as the sum of its two largest choice scores; the chosen scores divided by
+//            their sum before the scale (`renorm`).
 //   sort     the (row, choice) pairs ordered by expert, cut into tiles of 64 pairs of one expert.
 //   gate_up  act[pair] = silu(h[row] Wg_e^T) * (h[row] Wu_e^T)      per tile, float accumulation
 //   down     y[pair]   = act[pair] Wd_e^T                           per tile, float results
@@ -66,7 +67,7 @@ template <typename T, typename W, int RB>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int rows, int D, int E, int G, int keep,
                  int top, float scale, int has_gate, int vec_ok, int sigmoid_scores, const float* __restrict__ correction,
-                 int group_top, int* __restrict__ idx, float* __restrict__ wt, float* __restrict__ gate_out) {
+                 int group_top, int renorm, int* __restrict__ idx, float* __restrict__ wt, float* __restrict__ gate_out) {
   extern __shared__ float route_smem[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row0 = blockIdx.x * RB;
@@ -177,6 +178,7 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int
         __syncwarp();
       }
     }
+    float chosen = 0.f;                                        // sum of the chosen scores, in the order of choice
     for (int k = 0; k < top; ++k) {
       float bv = -INFINITY;
       int bi = 0x7fffffff;
@@ -187,6 +189,7 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int
       }
       warp_argmax(bv, bi);
       __syncwarp();
+      if (bi < E) chosen += z[bi];
       if (lane == 0) {
         const bool ok = bi < E;
         idx[size_t(row) * top + k] = ok ? bi : 0;
@@ -195,6 +198,8 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int
       }
       __syncwarp();
     }
+    if (renorm && lane == 0)
+      for (int k = 0; k < top; ++k) wt[size_t(row) * top + k] = wt[size_t(row) * top + k] / (chosen + 1e-20f);
   }
 }
 
@@ -373,7 +378,7 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place_of
 
 template <typename T>
 int launch_moe_route(const void* h, int ldh, const void* wr, int w_f32, int rows, int D, int E, int G, int keep, int top,
-                     float scale, int has_gate, int sigmoid_scores, const float* correction, int group_top, int* idx,
+                     float scale, int has_gate, int sigmoid_scores, const float* correction, int group_top, int renorm, int* idx,
                      float* wt, float* gate_out, cudaStream_t s) {
   if (rows == 0) return 0;
   if (E < 1 || G < 1 || E % G || keep < 1 || keep > G || top < 1 || top > (E / G) * keep || group_top < 1 || group_top > 2)
@@ -391,7 +396,7 @@ int launch_moe_route(const void* h, int ldh, const void* wr, int w_f32, int rows
       cudaFuncSetAttribute(moe_route_kernel<T, W, RB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
     moe_route_kernel<T, W, RB><<<(rows + RB - 1) / RB, ROUTE_WARPS * 32, smem, s>>>(                                  \
         (const T*)h, ldh, (const W*)wr, rows, D, E, G, keep, top, scale, has_gate, vec_ok, sigmoid_scores, correction, \
-        group_top, idx, wt, gate_out);                                                                                \
+        group_top, renorm, idx, wt, gate_out);                                                                                \
   } while (0)
 #define KVCM_ROUTE_RB(W)                                                                                              \
   do {                                                                                                                \
@@ -483,10 +488,10 @@ KVCM_API int kvcm_moe_experts_tc_bf16(const void* h, int ldh, const void* wgu, c
 #define KVCM_MOE(SUFFIX, T)                                                                                          \
   KVCM_API int kvcm_moe_route_##SUFFIX(const void* h, int ldh, const void* wr, int w_f32, int rows, int D, int E,    \
                                        int G, int keep, int top, float scale, int has_gate, int sigmoid_scores,      \
-                                       const float* correction, int group_top, int* idx, float* wt,                  \
+                                       const float* correction, int group_top, int renorm, int* idx, float* wt,      \
                                        float* gate_out, void* stream) {                                              \
     return launch_moe_route<T>(h, ldh, wr, w_f32, rows, D, E, G, keep, top, scale, has_gate, sigmoid_scores,         \
-                               correction, group_top, idx, wt, gate_out, (cudaStream_t)stream);                      \
+                               correction, group_top, renorm, idx, wt, gate_out, (cudaStream_t)stream);              \
   }                                                                                                                  \
   KVCM_API int kvcm_moe_experts_##SUFFIX(const void* h, int ldh, const void* wgu, const void* wd, const int* idx,    \
                                          int rows, int top, int E, int F, int D, int* work, void* act, float* y,     \

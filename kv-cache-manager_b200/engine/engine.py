@@ -106,7 +106,7 @@ class Engine:
             max_rows=max(max_rows, kv.max_seq_len), max_seqs=sc.max_num_seqs,
             max_logit_rows=max(self.max_logit_rows, kv.max_seq_len),
             options={"attn_version": cfg.attn, "gemm": cfg.gemm, "fuse_norms": cfg.fuse_norms})
-        self.kv = manager_from_config(kv, self.runner.windows)
+        self.kv = manager_from_config(kv, self.runner.windows, self.runner.chunks)
         s = core.SchedulerConfig()
         s.max_num_seqs, s.max_batched_tokens = sc.max_num_seqs, sc.max_batched_tokens
         s.prefill_chunk, s.chunked_prefill, s.eos_token_id = sc.prefill_chunk, sc.chunked_prefill, cfg.eos_token_id

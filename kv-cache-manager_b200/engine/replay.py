@@ -42,7 +42,7 @@ class ReplaySession:
                                   max_logit_rows=rows, options=options or {})
         self.kv = manager_from_config(KVManagerConfig(policy=policy, num_blocks=num_blocks, block_size=B,
                                                       max_seq_len=max_seq_len, prefix_caching=prefix_caching,
-                                                      watermark_blocks=0), self.runner.windows)
+                                                      watermark_blocks=0), self.runner.windows, self.runner.chunks)
         self.slots = core.StateSlots(max_live)
         self.vocab = spec.lm_head.vocab
         self.live: Dict[object, object] = {}

@@ -39,6 +39,7 @@ class ModelRunner:
         self.pools = CachePools(self.plan, num_blocks, block_size, num_slots, dtype, self.device)
         self.num_groups = max(1, len(self.plan.groups))
         self.windows = self.plan.windows or [0]
+        self.chunks = self.plan.chunks or [0]
         self.builder = core.BatchBuilder(block_size, self.max_blocks, self.num_groups, PREFILL_TILE_ROWS)
         cap = int(self.builder.capacity_for(max_rows, max_seqs, max_logit_rows))
         self.capacity = cap
@@ -144,7 +145,11 @@ class ModelRunner:
             if call.enter is not None:
                 part, arg = call.enter
                 x, pending = part.forward(x, pending, ctx, arg)
-            pending = spec.blocks[call.layer].forward(x, pending, ctx, self.pools.sites[k])
+            block = spec.blocks[call.layer]
+            if block.moves_stream:
+                x, pending = block.forward(x, pending, ctx, self.pools.sites[k])
+            else:
+                pending = block.forward(x, pending, ctx, self.pools.sites[k])
         n = ctx.logit_rows.numel()
         if n == 0:
             return None

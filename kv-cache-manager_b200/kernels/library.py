@@ -255,6 +255,16 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
     _check(fn(_p(gate_up), _p(out), T, I, _stream()), "silu_mul")
 
 
+def clamped_gate(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float) -> None:
+    """out = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); gate_up [T, 2I]."""
+    _cuda(gate_up, out)
+    T, I = out.shape
+    _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.shape == (T, 2 * I)
+          and gate_up.dtype == out.dtype, "clamped_gate: gate_up must be [T, 2I]")
+    fn = getattr(_lib(), "kvcm_clamped_gate_" + _suffix(out))
+    _check(fn(_p(gate_up), _p(out), T, I, ctypes.c_float(limit), ctypes.c_float(alpha), _stream()), "clamped_gate")
+
+
 def gather_rows(src: torch.Tensor, rows: torch.Tensor, dst: torch.Tensor) -> None:
     _cuda(src, rows, dst)
     n, W = dst.shape
@@ -287,11 +297,12 @@ def gemm_plain(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor) -> None:
 def attention_plain(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                     block_tables: torch.Tensor, row_seq: torch.Tensor, positions: torch.Tensor,
                     nh: int, nkv: int, hd: int, scale: float, window: int = 0, softcap: float = 0.0,
-                    sink: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                    sink: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0) -> None:
     """Row-per-query paged attention.  q: [T, >= nh*hd] (row stride free), out: [T, nh*hd];
     caches [pages, nkv, block, hd]; block_tables int32 [S, max_blocks].  ``softcap`` > 0 caps the
     scaled scores as cap * tanh(score / cap); ``sink`` (float32 [nh]) adds exp(sink) of each head to
-    its softmax denominators; with a window, ``keep_first`` > 0 keeps a request's first keys visible to every row."""
+    its softmax denominators; with a window, ``keep_first`` > 0 keeps a request's first keys visible to every row;
+    ``chunk`` > 0: a row sees only the keys of its own chunk of that many positions."""
     _cuda(q, out, k_cache, v_cache, block_tables, row_seq, positions, sink)
     _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh),
           "attention: sink float32 [heads]")
@@ -307,7 +318,8 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
     fn = getattr(_lib(), "kvcm_attention_plain_keep_" + _suffix(q))
     _check(fn(_p(q), q.stride(0), _p(out), out.stride(0), _p(k_cache), _p(v_cache), _p(block_tables),
               block_tables.shape[1], _p(row_seq), _p(positions), T, nh, nkv, hd, k_cache.shape[2],
-              ctypes.c_float(scale), int(window), ctypes.c_float(softcap), _p(sink), int(keep_first), _stream()), "attention_plain",
+              ctypes.c_float(scale), int(window), ctypes.c_float(softcap), _p(sink), int(keep_first), int(chunk),
+              _stream()), "attention_plain",
            f"(hd={hd}, nh={nh}, nkv={nkv})")
 
 
@@ -391,22 +403,22 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, seed: torch.Tensor,
 def paged_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                     block_tables: torch.Tensor, ctx, nh: int, nkv: int, hd: int, scale: float,
                     window: int = 0, softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
-                    keep_first: int = 0) -> None:
+                    keep_first: int = 0, chunk: int = 0) -> None:
     """Attention of all rows of a step.  Rows [0, ctx.decode_seqs) are single-row entries, the
     rest are the rows of longer portions.  ``ctx.options['attention']``: 'plain' forces the plain
     kernel for every row; float32 storage always uses it (the true 32-bit path)."""
     mode = ctx.options.get("attention", "auto")
     if mode == "plain" or q.dtype == torch.float32 or not fast_attention_supported(nh, nkv, hd, k_cache.shape[2]):
         attention_plain(q, out, k_cache, v_cache, block_tables, ctx.row_seq, ctx.positions,
-                        nh, nkv, hd, scale, window, softcap, sink, keep_first)
+                        nh, nkv, hd, scale, window, softcap, sink, keep_first, chunk)
         return
     nd = ctx.decode_seqs
     if nd > 0:
         attention_decode(q[:nd], out[:nd], k_cache, v_cache, block_tables, ctx, nh, nkv, hd, scale, window, softcap, sink,
-                         keep_first)
+                         keep_first, chunk)
     if ctx.rows > nd:
         attention_prefill(q, out, k_cache, v_cache, block_tables, ctx, nh, nkv, hd, scale, window, softcap, sink,
-                          keep_first)
+                          keep_first, chunk)
 
 
 def fast_attention_supported(nh: int, nkv: int, hd: int, block_size: int) -> bool:
@@ -469,9 +481,10 @@ def decode_partitions(seqs: int, nh: int, nkv: int, hd: int, max_ctx: int, devic
 def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                      block_tables: torch.Tensor, ctx, nh: int, nkv: int, hd: int, scale: float,
                      window: int = 0, softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
-                     keep_first: int = 0) -> None:
+                     keep_first: int = 0, chunk: int = 0) -> None:
     """Single-row entries: q/out hold one row per request, in the order of the batch's entries.
-    ``softcap`` / ``sink`` as in ``attention_plain``."""
+    ``softcap`` / ``sink`` / ``chunk`` as in ``attention_plain``; with chunks the partitions split the longest
+    part of a context that a chunk can hold (and the tile its start lies in)."""
     _cuda(q, out, k_cache, v_cache, block_tables, sink)
     _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh),
           "attention_decode: sink float32 [heads]")
@@ -481,7 +494,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
     _need(q.stride(1) == 1 and out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous(),
           "attention_decode: layout")
     _need(q.data_ptr() % 16 == 0 and (q.stride(0) * 2) % 16 == 0, "attention_decode: q rows must be 16-byte aligned")
-    size, parts = decode_partitions(S, nh, nkv, hd, ctx.max_decode_ctx, q.device,
+    span = ctx.max_decode_ctx if chunk <= 0 else min(ctx.max_decode_ctx, int(chunk) + KEY_TILE - 1)
+    size, parts = decode_partitions(S, nh, nkv, hd, span, q.device,
                                     ctx.options.get("attn_version", "auto"), int(ctx.options.get("attn_parts", 0)))
     scratch = None
     # Up to 8 partitions merge inside a thread-block cluster; more go through scratch memory
@@ -493,7 +507,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
     rc = _lib().kvcm_attention_decode_keep_bf16(
         _p(q), q.stride(0), _p(out), out.stride(0), _p(k_cache), _p(v_cache), _p(block_tables),
         block_tables.shape[1], _p(ctx.seq_ctx_len), S, nh, nkv, hd, k_cache.shape[2],
-        ctypes.c_float(scale), int(window), int(keep_first), size, parts, _p(scratch), int(in_cluster), ctypes.c_float(softcap), _p(sink),
+        ctypes.c_float(scale), int(window), int(keep_first), int(chunk), size, parts, _p(scratch), int(in_cluster), ctypes.c_float(softcap), _p(sink),
         _stream())
     _check(rc, "attention_decode", f"(hd={hd}, nh={nh}, nkv={nkv})")
     if parts > 1 and not in_cluster:
@@ -504,7 +518,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
 def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       block_tables: torch.Tensor, ctx, nh: int, nkv: int, hd: int, scale: float,
                       window: int = 0, softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
-                      keep_first: int = 0) -> None:
+                      keep_first: int = 0, chunk: int = 0) -> None:
     """Rows of portions longer than one token; q/out are the step's full row arrays.
     ``ctx.options['attn_prefill']``: 'tcgen05' | 'mma' force a kernel; 'auto' takes the tcgen05
     kernel where it supports the sizes (head_dim 64 or 128, 256 when keys and values are the same pages; pages of
@@ -528,14 +542,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
             _p(q), q.stride(0), q.shape[0], _p(out), out.stride(0), _p(k_cache), _p(v_cache), k_cache.shape[0],
             _p(block_tables), block_tables.shape[1], _p(ctx.tile_seq), _p(ctx.tile_q0), _p(ctx.seq_q_start),
             _p(ctx.seq_q_len), _p(ctx.seq_ctx_len), ctx.prefill_tiles, nh, nkv, hd, B, ctypes.c_float(scale),
-            int(window), kept, ctypes.c_float(softcap), _p(sink), _stream())
+            int(window), kept, int(chunk), ctypes.c_float(softcap), _p(sink), _stream())
         _check(rc, "attention_prefill_tcgen05", f"(hd={hd}, nh={nh}, nkv={nkv}, block={B})")
         return
     rc = _lib().kvcm_attention_prefill_keep_bf16(
         _p(q), q.stride(0), _p(out), out.stride(0), _p(k_cache), _p(v_cache), _p(block_tables),
         block_tables.shape[1], _p(ctx.tile_seq), _p(ctx.tile_q0), _p(ctx.seq_q_start), _p(ctx.seq_q_len),
         _p(ctx.seq_ctx_len), ctx.prefill_tiles, nh, nkv, hd, B, ctypes.c_float(scale),
-        int(window), kept, ctypes.c_float(softcap), _p(sink), _stream())
+        int(window), kept, int(chunk), ctypes.c_float(softcap), _p(sink), _stream())
     _check(rc, "attention_prefill", f"(hd={hd}, nh={nh}, nkv={nkv})")
 
 
@@ -677,6 +691,32 @@ def gate_up_silu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor,
                                               _p(w_gate_up), _p(act), M, I, K, x.stride(0), w_gate_up.stride(0),
                                               act.stride(0), sm_count(x.device), _stream())
     _check(rc, "gate_up_silu", f"(M={M}, I={I}, K={K})")
+
+
+def gate_up_clamped(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, limit: float, alpha: float) -> None:
+    """Fused decode kernel: the products of ``gate_up_silu`` joined by the activation of ``clamped_gate``."""
+    _cuda(x, w_gate_up, act)
+    M, K = x.shape
+    I = act.shape[1]
+    _need(w_gate_up.shape == (2 * I, K) and act.shape[0] == M, "gate_up_clamped: shapes")
+    _need(x.dtype == w_gate_up.dtype == act.dtype == torch.bfloat16, "gate_up_clamped: bfloat16 only")
+    _need(x.stride(1) == 1 and w_gate_up.stride(1) == 1 and act.stride(1) == 1, "gate_up_clamped: layout")
+    rc = _lib().kvcm_gate_up_clamped_bf16(_p(x), _p(w_gate_up), _p(act), M, I, K, x.stride(0), w_gate_up.stride(0),
+                                          act.stride(0), ctypes.c_float(limit), ctypes.c_float(alpha), sm_count(x.device), _stream())
+    _check(rc, "gate_up_clamped", f"(M={M}, I={I}, K={K})")
+
+
+def gate_up_clamped_tcgen05(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, limit: float, alpha: float) -> None:
+    """``gate_up_silu_tcgen05`` with the activation of ``clamped_gate``."""
+    _cuda(x, w_gate_up, act)
+    M, K = x.shape
+    I = act.shape[1]
+    _need(w_gate_up.shape == (2 * I, K) and act.shape[0] == M, "gate_up_clamped_tcgen05: shapes")
+    _need(x.dtype == w_gate_up.dtype == act.dtype == torch.bfloat16, "gate_up_clamped_tcgen05: bfloat16 only")
+    _need(x.stride(1) == 1 and w_gate_up.stride(1) == 1 and act.stride(1) == 1, "gate_up_clamped_tcgen05: rows must be dense")
+    rc = _lib().kvcm_gate_up_clamped_tcgen05_bf16(_p(x), _p(w_gate_up), _p(act), M, I, K, x.stride(0), w_gate_up.stride(0),
+                                                  act.stride(0), ctypes.c_float(limit), ctypes.c_float(alpha), _stream())
+    _check(rc, "gate_up_clamped_tcgen05", f"(M={M}, I={I}, K={K})")
 
 
 def gate_up_silu_supported(M: int, I: int, K: int) -> bool:
@@ -1046,12 +1086,13 @@ def latent_norm_cache(v: torch.Tensor, weight: torch.Tensor, slot_mapping: torch
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, groups: int, keep: int, top: int, scale: float,
               idx: torch.Tensor, wt: torch.Tensor, gate: Optional[torch.Tensor], scores: str = "softmax",
-              correction: Optional[torch.Tensor] = None, group_top: int = 1) -> None:
+              correction: Optional[torch.Tensor] = None, group_top: int = 1, renorm: bool = False) -> None:
     """Per row: float32 router logits, scores (``scores``: "softmax" over all experts or "sigmoid" of each
     logit), group-limited choice of ``top`` experts; ``idx`` int32 [T, top], ``wt`` float32 [T, top] =
     score * scale; ``gate`` float32 [T] = sigmoid of the logit of the router matrix's extra row (row
     ``experts``).  ``correction`` (float32 [experts]) is added to the scores for the choice only;
-    ``group_top``: a group's score is the sum of its 1 or 2 largest choice scores."""
+    ``group_top``: a group's score is the sum of its 1 or 2 largest choice scores; ``renorm``: the chosen scores are
+    divided by their sum (+ 1e-20) before the scale."""
     _cuda(h, router, idx, wt, gate, correction)
     _need(scores in ("softmax", "sigmoid") and group_top in (1, 2), "moe_route: scores 'softmax' | 'sigmoid', group_top 1 | 2")
     _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == experts),
@@ -1065,7 +1106,7 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, groups: int, 
     fn = getattr(_lib(), "kvcm_moe_route_" + _suffix(h))
     _check(fn(_p(h), h.stride(0), _p(router), int(router.dtype == torch.float32), T, D, experts, groups, keep, top,
               ctypes.c_float(scale), int(gate is not None), int(scores == "sigmoid"), _p(correction), int(group_top),
-              _p(idx), _p(wt), _p(gate), _stream()), "moe_route",
+              int(bool(renorm)), _p(idx), _p(wt), _p(gate), _stream()), "moe_route",
            f"(experts={experts}, groups={groups}, keep={keep}, top={top})")
 
 
@@ -1135,14 +1176,16 @@ SCAN_DELTA, SCAN_DELTA_CHANNEL, SCAN_LINEAR, SCAN_LINEAR_CHANNEL = 0, 1, 2, 3
 
 def state_scan(mode: int, qkv: torch.Tensor, bases, beta: Optional[torch.Tensor], g: Optional[torch.Tensor],
                gd: Optional[torch.Tensor], state: torch.Tensor, ctx, out: torch.Tensor, heads: int, qk_heads: int,
-               dk: int, dv: int) -> None:
+               dk: int, dv: int, silu: bool = False) -> None:
     """The matrix-state recurrences over every request's rows of the step, from and into its state row
     (csrc/cuda/delta_rule.cu).  ``bases`` = where a row's q, k and v start; ``beta`` [T, >= heads] (a view
     with a row stride is fine), ``g`` likewise (one decay per head) or ``gd`` [T, heads*dk] (one per head
-    and key channel).  ``beta`` may be None for SCAN_LINEAR_CHANNEL (it then counts as one)."""
+    and key channel).  The linear forms take ``beta`` None (it then counts as one) and ``silu``: q, k and v are
+    projections that pass SiLU first.  A row stride of zero in ``g`` gives every row the same decays."""
     _cuda(qkv, beta, g, gd, state, out)
     _need(all(t is None or t.dtype == torch.float32 for t in (qkv, beta, g, gd, state, out)), "state_scan: float32")
-    _need(beta is not None or mode == SCAN_LINEAR_CHANNEL, "state_scan: beta")
+    linear = mode in (SCAN_LINEAR, SCAN_LINEAR_CHANNEL)
+    _need(linear or (beta is not None and not silu), "state_scan: beta")
     _need(qkv.is_contiguous() and out.is_contiguous() and state.is_contiguous() and (beta is None or beta.stride(1) == 1)
           and (g is None or g.stride(1) == 1) and (gd is None or (gd.is_contiguous() and gd.shape == (qkv.shape[0], heads * dk))),
           "state_scan: layout")
@@ -1153,7 +1196,7 @@ def state_scan(mode: int, qkv: torch.Tensor, bases, beta: Optional[torch.Tensor]
     _check(_lib().kvcm_state_scan(int(mode), _p(qkv), C, qb, kb, vb, _p(beta), beta.stride(0) if beta is not None else 0, _p(g),
                                   g.stride(0) if g is not None else 0, _p(gd), _p(state), _ll(state.stride(0)),
                                   _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out), qkv.shape[0],
-                                  ctx.seqs, heads, qk_heads, dk, dv, _stream()), "state_scan", f"(mode={mode}, dk={dk}, dv={dv})")
+                                  ctx.seqs, heads, qk_heads, dk, dv, int(bool(silu)), _stream()), "state_scan", f"(mode={mode}, dk={dk}, dv={dv})")
 
 
 def delta_prepare_channel(qkv: torch.Tensor, b: torch.Tensor, beta: torch.Tensor, a: torch.Tensor, a_log: torch.Tensor,
@@ -1188,17 +1231,18 @@ def group_rms_gate(o: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, out: 
                    skip_coef: Optional[torch.Tensor] = None, head: int = 1) -> None:
     """Norm in groups of ``group`` neighbouring elements with a gate ``act`` ('silu' | 'sigmoid') of z before or
     after it; ``weight`` is indexed modulo its length; optional skip term ``skip_coef[i // head] * skip[:, i]``
-    added to o first.  o/skip float32, z/out storage dtype (z and skip may have a row stride)."""
+    added to o first.  o/skip float32, out storage dtype, z that or float32 (z and skip may have a row stride)."""
     _cuda(o, z, weight, out, skip, skip_coef)
     T, n = o.shape
     _need(o.dtype == torch.float32 and o.is_contiguous() and out.is_contiguous() and out.shape == o.shape
-          and z.stride(1) == 1 and z.shape[1] >= n and z.dtype == out.dtype and weight.dtype == torch.float32
+          and z.stride(1) == 1 and z.shape[1] >= n and z.dtype in (torch.float32, out.dtype) and weight.dtype == torch.float32
           and weight.is_contiguous() and n % group == 0, "group_rms_gate: layout")
     _need((skip is None) == (skip_coef is None), "group_rms_gate: skip and its coefficients come together")
     if skip is not None:
         _need(skip.dtype == torch.float32 and skip.stride(1) == 1 and skip.shape[1] >= n and skip_coef.dtype == torch.float32
               and skip_coef.is_contiguous() and skip_coef.numel() * head >= n, "group_rms_gate: skip layout")
-    fn = getattr(_lib(), "kvcm_group_rms_gate_" + _suffix(out))
+    mixed = z.dtype != out.dtype
+    fn = getattr(_lib(), "kvcm_group_rms_gate_" + ("zf32_" if mixed else "") + _suffix(out))
     _check(fn(_p(o), _p(z), z.stride(0), _p(skip), skip.stride(0) if skip is not None else 0, _p(skip_coef), int(head),
               _p(weight), weight.numel(), _p(out), T, n, int(group), int(bool(gate_first)), {"silu": 0, "sigmoid": 1}[act],
               ctypes.c_float(eps), _stream()), "group_rms_gate")
@@ -1245,7 +1289,8 @@ def attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: Optional[
                  v_keep: Optional[torch.Tensor], v_first: Optional[torch.Tensor], lam: Optional[torch.Tensor],
                  slot_mapping: Optional[torch.Tensor], q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                  nh: int, nkv: int, dk: int, dv: int, interleaved: bool = False,
-                 v_inv_freq: Optional[torch.Tensor] = None, maps: int = 1) -> None:
+                 v_inv_freq: Optional[torch.Tensor] = None, maps: int = 1, hq: Optional[torch.Tensor] = None,
+                 hk: Optional[torch.Tensor] = None, v_norm: bool = False, amplitude: float = 1.0) -> None:
     """From the float32 q|k|v projection of a step's rows to the attention kernel's inputs: optional bias,
     optional norm over the whole q and k projections (weights wq, wk), rotation of the first ``rot``
     dimensions of every head, optional per-head norm without weights, optional mixing of the values with
@@ -1253,7 +1298,10 @@ def attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: Optional[
     cache's head size HD (csrc/cuda/attn_prepare.cu).  ``interleaved``: rotary pairs (2i, 2i+1) instead of
     (i, i + rot/2); ``v_inv_freq`` (float32 [dv/2]): the values too are turned by their position, over all dv.
     ``maps`` > 1: every q and k head holds that many score maps of ``dk`` elements side by side; ``q_out`` is
-    [T, nh*maps*HD], one padded head per map with the map at its own place, and a key head caches its maps in a row."""
+    [T, nh*maps*HD], one padded head per map with the map at its own place, and a key head caches its maps in a row.
+    ``hq``/``hk`` (float32 [dk]): q and k of every head are divided by their root mean square and multiplied by these
+    BEFORE the rotation; ``v_norm``: every value head is divided by its root mean square; ``amplitude``: factor of the
+    rotation's cosines and sines."""
     _cuda(proj, bias, wq, wk, positions, inv_freq, v_keep, v_first, lam, slot_mapping, q_out, k_cache, v_cache, v_inv_freq)
     _need(v_inv_freq is None or (v_inv_freq.dtype == torch.float32 and v_inv_freq.is_contiguous() and v_inv_freq.numel() * 2 == dv),
           "attn_prepare: v_inv_freq float32 [dv/2]")
@@ -1262,9 +1310,9 @@ def attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: Optional[
     n = (nh + nkv) * maps * dk + nkv * dv
     _need(maps >= 1 and (maps == 1 or wq is None), "attn_prepare: several maps go without the whole-projection norm")
     _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= n and proj.shape[0] >= T, "attn_prepare: proj float32 [T, q|k|v]")
-    for t, m in ((bias, n), (wq, nh * maps * dk), (wk, nkv * maps * dk), (lam, 1)):
+    for t, m in ((bias, n), (wq, nh * maps * dk), (wk, nkv * maps * dk), (lam, 1), (hq, dk), (hk, dk)):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == m), "attn_prepare: float32 vectors")
-    _need((wq is None) == (wk is None) and (v_first is None) == (lam is None), "attn_prepare: arguments that come in pairs")
+    _need((wq is None) == (wk is None) and (v_first is None) == (lam is None) and (hq is None) == (hk is None), "attn_prepare: arguments that come in pairs")
     for t in (v_keep, v_first):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, nkv * dv)), "attn_prepare: values float32 [T, nkv*dv]")
     _need(q_out.is_contiguous() and q_out.shape == (T, nh * maps * HD) and q_out.dtype == k_cache.dtype == v_cache.dtype
@@ -1276,7 +1324,8 @@ def attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: Optional[
     fn = getattr(_lib(), "kvcm_attn_prepare_" + _suffix(q_out))
     _check(fn(_p(proj), proj.stride(0), _p(bias), _p(wq), _p(wk), _p(positions), _p(inv_freq), int(rot), int(bool(head_norm)),
               ctypes.c_float(eps), _p(v_keep), _p(v_first), _p(lam), _p(slot_mapping), B, _p(q_out), _p(k_cache), _p(v_cache),
-              T, nh, nkv, dk, dv, HD, int(bool(interleaved)), _p(v_inv_freq), int(maps), _stream()), "attn_prepare", f"(nh={nh}, nkv={nkv}, dk={dk}, dv={dv}, HD={HD})")
+              T, nh, nkv, dk, dv, HD, int(bool(interleaved)), _p(v_inv_freq), int(maps), _p(hq), _p(hk), int(bool(v_norm)),
+              ctypes.c_float(amplitude), _stream()), "attn_prepare", f"(nh={nh}, nkv={nkv}, dk={dk}, dv={dv}, HD={HD})")
 
 
 # ------------------------------------------- blocks normalised on both sides, and what comes with them
@@ -1484,11 +1533,58 @@ def diff_combine(a: torch.Tensor, gate: Optional[torch.Tensor], lam: torch.Tenso
               ctypes.c_float(post), _stream()), "diff_combine")
 
 
-def gate_mul(x: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> None:
-    """out = x * sigmoid(gate), element by element; x and out [T, n] in the storage dtype, gate float32 [T, n] (row stride free)."""
+def gate_mul(x: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, heads: int = 1) -> None:
+    """out = x * sigmoid(gate), element by element; out [T, n] in the storage dtype, gate float32 [T, n] (row stride
+    free).  x [T, n], or the attention kernel's padded heads [T, heads * HD] of which the first n / heads elements count."""
     _cuda(x, gate, out)
-    T, n = x.shape
-    _need(x.is_contiguous() and out.is_contiguous() and out.shape == x.shape and out.dtype == x.dtype and gate.dtype == torch.float32
-          and gate.stride(1) == 1 and gate.shape == (T, n), "gate_mul: layout")
+    T, n = out.shape
+    _need(x.is_contiguous() and out.is_contiguous() and x.shape[0] == T and out.dtype == x.dtype and gate.dtype == torch.float32
+          and gate.stride(1) == 1 and gate.shape == (T, n) and n % heads == 0 and x.shape[1] % heads == 0 and x.shape[1] >= n,
+          "gate_mul: layout")
     fn = getattr(_lib(), "kvcm_gate_mul_" + _suffix(x))
-    _check(fn(_p(x), _p(gate), gate.stride(0), _p(out), T, n, _stream()), "gate_mul")
+    _check(fn(_p(x), _p(gate), gate.stride(0), _p(out), T, n, n // heads, x.shape[1] // heads, _stream()), "gate_mul")
+
+
+# ------------------------------------------------- two norms of one stream, and the row before mixed in
+
+def norm_pair(x: torch.Tensor, pending, experts, w1: torch.Tensor, eps1: float, out1: torch.Tensor,
+              w2: Optional[torch.Tensor] = None, eps2: float = 1e-6, out2: Optional[torch.Tensor] = None,
+              shift: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, ctx=None,
+              x_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> None:
+    """x' = x + what is pending (up to three (float32 tensor, scale) pairs, and ``experts``: a parts.base.ExpertSum or
+    None); out1 = w1 * x' / rms(x') with ``shift`` (float32 [D]) mixing in the row before of the same request,
+    h + (h_before - h) * shift, whose h comes from ``state`` (float32 [slots, D], also brought up to date) at a portion's
+    first row; out2 = w2 * x' / rms(x') (optional).  ``x_out`` receives x' (never x itself); ``rows`` (int32): the outputs
+    are formed for these rows only (final norm).  Weights are float32 multipliers."""
+    pend = list(pending or [])
+    _need(len(pend) <= 3, "norm_pair: at most three pending outputs")
+    e = experts
+    _cuda(x, w1, out1, w2, out2, shift, state, x_out, rows, *[t for t, _ in pend], *((e.y, e.work, e.wt) if e is not None else ()))
+    T, D = x.shape
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "norm_pair: x float32 [T, D]")
+    for t in [t for t, _ in pend] + [x_out]:
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == x.shape), "norm_pair: float32 like x")
+    _need(x_out is None or x_out.data_ptr() != x.data_ptr(), "norm_pair: the new stream is a tensor of its own")
+    for w in (w1, w2, shift):
+        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == D), "norm_pair: weights float32 [D]")
+    n = T if rows is None else out1.shape[0]
+    _need(out1.is_contiguous() and out1.shape == (n, D) and (out2 is None or (out2.is_contiguous() and out2.shape == (n, D)
+          and out2.dtype == out1.dtype and w2 is not None)), "norm_pair: outputs [rows, D]")
+    _need(rows is None or (rows.dtype == _I32 and rows.numel() >= n and shift is None and x_out is None), "norm_pair: gathered rows")
+    _need(shift is None or (ctx is not None and state is not None and state.dtype == torch.float32 and state.is_contiguous()
+                            and state.dim() == 2 and state.shape[1] == D), "norm_pair: a shift needs the requests' state [slots, D]")
+    ey = place = wt = None
+    top = 0
+    if e is not None:
+        top = e.wt.shape[1]
+        _need(e.y.dtype == e.wt.dtype == torch.float32 and e.y.is_contiguous() and e.wt.is_contiguous() and e.y.shape == (T * top, D)
+              and e.wt.shape == (T, top) and e.work.dtype == _I32, "norm_pair: the experts' outputs")
+        ey, wt = _p(e.y), _p(e.wt)
+        place = ctypes.c_void_p(e.work.data_ptr() + 4 * (e.experts + 2 + T * top))      # as the experts' sort leaves it
+    pend += [(None, 0.0)] * (3 - len(pend))
+    rs, qs, ql, sl = (ctx.row_seq, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_state_slot) if shift is not None else (None,) * 4
+    fn = getattr(_lib(), "kvcm_norm_pair_" + _suffix(out1))
+    _check(fn(_p(x), _p(x_out), _p(pend[0][0]), ctypes.c_float(pend[0][1]), _p(pend[1][0]), ctypes.c_float(pend[1][1]),
+              _p(pend[2][0]), ctypes.c_float(pend[2][1]), ey, place, wt, top, _p(w1), ctypes.c_float(eps1), _p(out1), _p(w2),
+              ctypes.c_float(eps2), _p(out2), _p(shift), _p(state), _ll(state.stride(0) if state is not None else 0), _p(rs), _p(qs),
+              _p(ql), _p(sl), _p(rows), n, D, _stream()), "norm_pair", f"(width={D})")

@@ -3,18 +3,19 @@ from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, Blo
                    FeedForward, GroupView, LayerCall, Mixer, Norm, ParamSpec, Part,
                    PositionEncoding, Registry, SiteCache, StateSpec, StepContext, StreamPart)
 from .linear import Linear, matmul_nt
-from .norm import DynamicTanh, OffsetRMSNorm, OutputRMSNorm, RMSNorm
+from .norm import DynamicTanh, Float32RMSNorm, OffsetRMSNorm, OutputRMSNorm, RMSNorm
 from .rope import NoPositionEncoding, RotaryEmbedding
 from .attention import GeneralAttention, PagedAttention
 from .delta import ChannelDecayDeltaMixer, GatedDeltaMixer, SideBySideMixer
 from .ssm import Mamba2Mixer
 from .latent_attention import LatentAttention, LatentRopeAttention
 from .gla import GatedLinearAttention
+from .lightning import LightningAttention
 from .loop import LoopEntry
 from .mlp import DenseMLP, GatedMLP
 from .moe import RoutedExperts
 from .embedding import Embedding, LMHead, ScaledEmbedding, SummedEmbedding
-from .block import OutputNormBlock, ParallelBlock, PreNormBlock, SandwichBlock
+from .block import OutputNormBlock, ParallelBlock, ParallelNormsBlock, PreNormBlock, SandwichBlock
 
 __all__ = [
     "BLOCKS", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITION_ENCODINGS", "Block", "CacheSpec",
@@ -25,4 +26,5 @@ __all__ = [
     "LatentAttention", "RoutedExperts", "DynamicTanh", "GeneralAttention", "ChannelDecayDeltaMixer",
     "SideBySideMixer", "Mamba2Mixer", "DenseMLP", "ParallelBlock", "StreamPart", "OffsetRMSNorm", "LatentRopeAttention",
     "GatedLinearAttention", "LoopEntry", "ScaledEmbedding", "SandwichBlock",
+    "Float32RMSNorm", "LightningAttention", "ParallelNormsBlock",
 ]

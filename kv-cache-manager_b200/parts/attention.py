@@ -19,6 +19,12 @@ from .base import CacheSpec, MIXERS, Mixer, PositionEncoding, SiteCache, StepCon
 from .linear import Linear, matmul_nt
 
 
+def plain_amplitude(position: PositionEncoding) -> None:
+    """For mixers whose kernels rotate with plain cosines and sines."""
+    if getattr(position, "amplitude", 1.0) != 1.0:
+        raise ValueError("this mixer has no kernel for a rotary encoding whose cosines and sines are scaled")
+
+
 @MIXERS.register("attention")
 class PagedAttention(Mixer):
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, head_dim: int,
@@ -26,6 +32,7 @@ class PagedAttention(Mixer):
         super().__init__()
         if num_heads % num_kv_heads:
             raise ValueError(f"attention: {num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
+        plain_amplitude(position)
         self.hidden, self.nh, self.nkv, self.hd = hidden, num_heads, num_kv_heads, head_dim
         self.window = int(window or 0)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
@@ -89,6 +96,11 @@ class GeneralAttention(Mixer):
     * ``rotate_values``: every value is turned by its own position over all ``dv`` dimensions (frequencies
       base^(-2m/dv) with the position encoding's base, the same pairing) before it is cached, and a head's
       output at position i (the weighted sum of the turned values) is turned back by -i;
+    * ``qk_norm``: q and k of every head divided by their root mean square over dk and multiplied by a weight [dk]
+      shared by the heads, before the rotation; ``value_norm``: every value head divided by its root mean square over
+      dv (no weight) before it is cached;
+    * ``chunk``: row i sees keys j <= i with j // chunk == i // chunk only (its page group gives passed chunks back);
+    * ``gate``: the concatenated heads multiplied element by element by sigmoid(W_g h), in front of the output product;
     * ``head_norm``: q and k of every head scaled to unit root mean square (no weights), after the
       rotation;
     * ``softcap``: score <- cap * tanh(score / cap) after the scale;
@@ -107,7 +119,8 @@ class GeneralAttention(Mixer):
                  position: PositionEncoding, scale: Optional[float] = None, window: int = 0, softcap: float = 0.0,
                  sink: bool = False, bias: bool = False, proj_norm: bool = False, head_norm: bool = False,
                  norm_eps: float = 1e-6, value_mix: Optional[str] = None, mix_key: str = "v_first",
-                 rotate_values: bool = False, keep_first: int = 0) -> None:
+                 rotate_values: bool = False, keep_first: int = 0, qk_norm: bool = False, value_norm: bool = False,
+                 chunk: int = 0, gate: bool = False) -> None:
         super().__init__()
         if num_kv_heads < 1 or num_heads % num_kv_heads:
             raise ValueError(f"attention: {num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
@@ -122,16 +135,23 @@ class GeneralAttention(Mixer):
         self.window, self.softcap = int(window or 0), float(softcap or 0.0)
         self.keep_first = int(keep_first or 0) if self.window > 0 else 0
         self.rotate_values = bool(rotate_values)
+        self.qk_norm, self.value_norm, self.has_gate, self.chunk = bool(qk_norm), bool(value_norm), bool(gate), int(chunk or 0)
+        if self.chunk > 0 and self.keep_first > 0:
+            raise ValueError("attention_general: chunks do not keep first keys")
         self._v_inv_freq = None
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(dk)
         self.has_sink, self.has_bias, self.proj_norm, self.head_norm = bool(sink), bool(bias), bool(proj_norm), bool(head_norm)
         self.norm_eps, self.value_mix, self.mix_key = float(norm_eps), value_mix, mix_key
         self.position = self.add_child("position", position)
         nq, nk, nv = num_heads * dk, num_kv_heads * dk, num_kv_heads * dv
-        self.qkv = self.add_child("qkv", Linear(hidden, nq + nk + nv, hidden ** -0.5))
+        # rows q | k | v, and with a gate its nh * dv rows behind them
+        self.qkv = self.add_child("qkv", Linear(hidden, nq + nk + nv + (num_heads * dv if gate else 0), hidden ** -0.5))
         self.o = self.add_child("o", Linear(num_heads * dv, hidden, (num_heads * dv) ** -0.5))
         if self.has_bias:
             self.declare("bias", (nq + nk + nv,), ("normal", 0.1), "vector")
+        if self.qk_norm:
+            self.declare("q_head_norm", (dk,), ("ones_jitter", 0.1), "vector")
+            self.declare("k_head_norm", (dk,), ("ones_jitter", 0.1), "vector")
         if self.proj_norm:
             self.declare("q_norm", (nq,), ("ones_jitter", 0.1), "vector")
             self.declare("k_norm", (nk,), ("ones_jitter", 0.1), "vector")
@@ -143,7 +163,7 @@ class GeneralAttention(Mixer):
         self._o_weight = None
 
     def cache_spec(self) -> CacheSpec:
-        return CacheSpec(self.nkv, self.hd, 0 if self.keep_first > 0 else self.window)
+        return CacheSpec(self.nkv, self.hd, 0 if self.keep_first > 0 else self.window, chunk=self.chunk)
 
     def prepare(self, device, dtype) -> None:
         super().prepare(device, dtype)
@@ -154,7 +174,7 @@ class GeneralAttention(Mixer):
             self._v_inv_freq = (1.0 / torch.pow(torch.tensor(self.position.theta, dtype=torch.float64),
                                                 2.0 * m / self.dv)).to(torch.float32).to(device)
         w = self.o.param("weight")
-        if self.hd != self.dv:                              # zero columns where the attention output is padding
+        if self.hd != self.dv and not self.has_gate:        # (the gate's kernel takes the padding out itself)  zero columns where the attention output is padding
             wide = torch.zeros((self.hidden, self.nh, self.hd), dtype=w.dtype, device=w.device)
             wide[:, :, :self.dv] = w.view(self.hidden, self.nh, self.dv)
             w = wide.view(self.hidden, self.nh * self.hd)
@@ -174,12 +194,18 @@ class GeneralAttention(Mixer):
         K.attn_prepare(proj, f.get("bias"), f.get("q_norm"), f.get("k_norm"), ctx.positions, pos.inv_freq,
                        pos.rotary_dim if pos.inv_freq is not None else 0, self.head_norm, self.norm_eps, keep, first,
                        f["vmix"] if first is not None else None, g.slot_mapping if site.writes else None, q, site.k, site.v,
-                       self.nh, self.nkv, self.dk, self.dv, bool(getattr(pos, "interleaved", False)), self._v_inv_freq)
+                       self.nh, self.nkv, self.dk, self.dv, bool(getattr(pos, "interleaved", False)), self._v_inv_freq,
+                       hq=f.get("q_head_norm"), hk=f.get("k_head_norm"), v_norm=self.value_norm,
+                       amplitude=getattr(pos, "amplitude", 1.0))
         out = torch.empty((T, self.nh * self.hd), dtype=h.dtype, device=h.device)
         K.paged_attention(q, out, site.k, site.v, g.block_tables, ctx, self.nh, self.nkv, self.hd, self.scale,
-                          self.window, self.softcap, f.get("sink"), self.keep_first)
+                          self.window, self.softcap, f.get("sink"), self.keep_first, self.chunk)
         if self.rotate_values:
             K.rotate_heads(out, ctx.positions, self._v_inv_freq, self.nh, self.hd, bool(getattr(pos, "interleaved", False)), -1.0)
+        if self.has_gate:
+            gated = torch.empty((T, self.nh * self.dv), dtype=h.dtype, device=h.device)
+            K.gate_mul(out, proj[:, self.qkv.out_features - self.nh * self.dv:], gated, self.nh)
+            out = gated
         return matmul_nt(out, self._o_weight, torch.float32, ctx.options)
 
 
@@ -207,6 +233,7 @@ class DifferentialAttention(Mixer):
         super().__init__()
         if num_kv_heads < 1 or num_heads % num_kv_heads:
             raise ValueError(f"attention: {num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
+        plain_amplitude(position)
         if getattr(position, "rotary_dim", 0) > dk:
             raise ValueError("differential_attention: the rotation covers at most one map's size")
         self.hidden, self.nh, self.nkv, self.dk, self.dv = hidden, num_heads, num_kv_heads, dk, dv

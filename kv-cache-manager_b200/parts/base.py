@@ -109,6 +109,7 @@ class CacheSpec:
     head_dim: int
     window: int = 0                 # 0: every key is kept; w: only the last w positions
     values: bool = True             # False: one pool only (a mixer that derives keys AND values from what it caches)
+    chunk: int = 0                  # c: position i needs only the keys of its own chunk, j >= i - i % c
 
 
 @dataclass(frozen=True)
@@ -151,7 +152,8 @@ class SiteCache:
     k: Optional[torch.Tensor] = None        # [pages, nkv, block, hd]
     v: Optional[torch.Tensor] = None        # None when the group's spec keeps no values
     writes: bool = True
-    state: Optional[torch.Tensor] = None    # [slots, *shape]
+    state: Optional[torch.Tensor] = None    # [slots, *shape], the mixer's
+    block_state: Optional[torch.Tensor] = None   # [slots, *shape], the block's own (see Block.state_spec)
 
 
 @dataclass
@@ -258,11 +260,54 @@ class ClosingNorm:
         self.y, self.multiplier, self.eps = y, multiplier, float(eps)
 
 
+class ExpertSum:
+    """A routed feed-forward's output before its weighted sum: ``y`` float32 [rows * top, width] in the order of the
+    sorted pairs, ``wt`` float32 [rows, top], ``work`` the sort's scratch (it holds every pair's place).  A block may hand
+    this on as pending, so that the reader of the stream forms the sum in its own kernel."""
+    __slots__ = ("y", "work", "wt", "experts")
+
+    def __init__(self, y: torch.Tensor, work: torch.Tensor, wt: torch.Tensor, experts: int) -> None:
+        self.y, self.work, self.wt, self.experts = y, work, wt, int(experts)
+
+    def combined(self) -> torch.Tensor:
+        from ..kernels import library as K
+        out = torch.empty((self.wt.shape[0], self.y.shape[1]), dtype=torch.float32, device=self.y.device)
+        K.moe_combine(self.y, self.work, self.wt, self.experts, None, None, out)
+        return out
+
+
+def split_pending(pending):
+    """What a layer left pending as ([(float32 tensor, scale), ...], one ``ExpertSum`` or None)."""
+    if pending is None:
+        return [], None
+    items = list(pending) if isinstance(pending, (list, tuple)) else [pending if isinstance(pending, ExpertSum) else (pending, 1.0)]
+    dense, experts = [], None
+    for item in items:
+        if not isinstance(item, ExpertSum):
+            t, scale = item
+            dense.append((t if t.dtype == torch.float32 else t.float(), scale))
+        elif experts is None:
+            experts = item
+        else:
+            dense.append((item.combined(), 1.0))
+    return dense, experts
+
+
 def settle(x: torch.Tensor, pending) -> None:
     """Brings the float32 stream ``x`` up to date with what the layer before left pending: nothing, a tensor
-    to add, or a ``ClosingNorm``."""
+    to add, a ``ClosingNorm``, an ``ExpertSum``, or a list of (tensor, scale) pairs and ``ExpertSum``s."""
     from ..kernels import library as K
     if pending is None:
+        return
+    if isinstance(pending, (list, tuple)):
+        for item in pending:
+            if isinstance(item, ExpertSum):
+                settle(x, item)
+            else:
+                settle(x, item[0] if item[1] == 1.0 else item[0] * item[1])
+        return
+    if isinstance(pending, ExpertSum):
+        K.add_residual(x, pending.combined())
         return
     if isinstance(pending, ClosingNorm):
         K.norm_post_pre(x, pending.y, pending.multiplier, None, None, pending.eps)
@@ -279,7 +324,15 @@ class StreamPart(Part):
 
 
 class Block(Part):
+    """``moves_stream``: ``forward`` leaves x as it is and returns (x', pending') with the stream in a new tensor
+    (a kernel that reads neighbouring rows of the old stream cannot write the new one in place).
+    ``state_spec``: fixed-size per-request state that the arrangement itself keeps, beside the mixer's; it arrives
+    as ``site.block_state``."""
     mixer: Mixer
+    moves_stream = False
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return None
 
     def forward(self, x: torch.Tensor, pending: Optional[torch.Tensor], ctx: StepContext,
                 site: SiteCache) -> torch.Tensor:

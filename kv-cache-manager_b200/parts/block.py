@@ -10,7 +10,8 @@ from typing import Optional
 import torch
 
 from ..kernels import library as K
-from .base import BLOCKS, Block, ClosingNorm, FeedForward, Mixer, Norm, SiteCache, StepContext, settle
+from .base import (BLOCKS, Block, ClosingNorm, ExpertSum, FeedForward, Mixer, Norm, SiteCache, StateSpec, StepContext, settle,
+                   split_pending)
 
 
 @BLOCKS.register("pre_norm")
@@ -87,6 +88,62 @@ class ParallelBlock(Block):
         if self.ffn is not None:
             out.append((self.ffn.forward(h, ctx, out_dtype=torch.float32), 1.0))
         return out
+
+
+@BLOCKS.register("parallel_norms")
+class ParallelNormsBlock(Block):
+    """x += mixer(shift(norm1(x))) + ffn(norm2(x)): both sublayers read the SAME stream, each through an RMS norm of its own
+    ("rmsnorm_f32").  ``token_shift``: what the mixer reads is mixed with the row before of the same request, h + (h_before
+    - h) * shift with a learned vector; the h of a request's last row is per-request state of the block (zeros at the start).
+
+    One kernel adds what the layer before left pending (in the order mixer, feed-forward; the experts' weighted sum
+    included), takes the row's one root mean square for both norms, applies the shift and stores the new stream in a tensor of
+    its own.  ``fuse`` off: the feed-forward forms its sum itself and the pending outputs are added by launches of
+    their own.  ``ffn`` may be None: a layer of a mixer only."""
+
+    moves_stream = True
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm] = None, ffn: Optional[FeedForward] = None,
+                 token_shift: bool = False, shift_init=("normal", 0.3)) -> None:
+        super().__init__()
+        self.norm1 = self.add_child("norm1", norm1)
+        self.mixer = self.add_child("mixer", mixer)
+        self.norm2 = self.add_child("norm2", norm2) if norm2 is not None else None
+        self.ffn = self.add_child("ffn", ffn) if ffn is not None else None
+        if (self.norm2 is None) != (self.ffn is None):
+            raise ValueError("parallel_norms block: a feed-forward and its norm come together")
+        self.hidden, self.token_shift = norm1.hidden, bool(token_shift)
+        if self.token_shift:
+            self.declare("shift", (self.hidden,), shift_init, "vector")
+        self._shift: Optional[torch.Tensor] = None
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec((self.hidden,), torch.float32) if self.token_shift else None
+
+    def prepare(self, device, dtype) -> None:
+        super().prepare(device, dtype)
+        if self.token_shift:
+            self._shift = self.param("shift").to(device=device, dtype=torch.float32).contiguous()
+
+    def forward(self, x: torch.Tensor, pending, ctx: StepContext, site: SiteCache):
+        fuse = ctx.options.get("fuse", True)
+        if pending is not None and not fuse:
+            settle(x, pending)                        # (x is this step's own tensor: nobody else reads the old one)
+            pending = None
+        dense, experts = split_pending(pending)
+        new = torch.empty_like(x) if dense or experts is not None else None
+        h1 = torch.empty(x.shape, dtype=ctx.dtype, device=x.device)
+        h2 = torch.empty_like(h1) if self.ffn is not None else None
+        K.norm_pair(x, dense, experts, self.norm1.multiplier, self.norm1.eps, h1,
+                    self.norm2.multiplier if h2 is not None else None, self.norm2.eps if h2 is not None else 1.0, h2,
+                    self._shift, site.block_state, ctx, new)
+        y = self.mixer.forward(h1, ctx, site)
+        out = list(y) if isinstance(y, (list, tuple)) else [(y, 1.0)]
+        if self.ffn is not None:
+            deferred = getattr(self.ffn, "forward_unsummed", None) if fuse else None
+            z = deferred(h2, ctx) if deferred is not None else self.ffn.forward(h2, ctx, out_dtype=torch.float32)
+            out.append(z if isinstance(z, ExpertSum) else (z, 1.0))
+        return (x if new is None else new), out
 
 
 @BLOCKS.register("sandwich")

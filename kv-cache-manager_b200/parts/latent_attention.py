@@ -114,7 +114,8 @@ class LatentRopeAttention(Mixer):
     def __init__(self, hidden: int, heads: int, dn: int, dr: int, dv: int, rank: int, q_rank: int, scale: float,
                  norm_eps: float, position, window: int = 0, sink: bool = False, gate: bool = False) -> None:
         super().__init__()
-        from .attention import padded_head_dim
+        from .attention import padded_head_dim, plain_amplitude
+        plain_amplitude(position)
         if getattr(position, "rotary_dim", 0) > dr:
             raise ValueError("latent_rope_attention: the rotation covers at most the rotated part")
         self.hidden, self.heads, self.dn, self.dr, self.dv, self.rank, self.q_rank = hidden, heads, dn, dr, dv, rank, int(q_rank or 0)

@@ -1,0 +1,60 @@
+"""Lightning attention: a linear-attention mixer with a fixed-size state per request and ONE constant decay per head.
+
+Per head a float32 matrix S [dk, dv], zero at a request's start, is carried from token to token:
+
+    S <- decay_h S + k v^T;    o = S^T q
+
+with q = silu(W_q h), k = silu(W_k h) (heads x dk) and v = silu(W_v h) (heads x dv); no other scale.  The heads' outputs
+side by side are divided by their root mean square over all of them and multiplied by a weight [heads * dv] and
+by sigmoid(W_g h), and go through the output projection.
+
+State of a request: one float32 row per call site, S of every head.  One product gives q | k | v | g (float32 result).
+The recurrence is the engine's matrix-state scan in its linear form (csrc/cuda/delta_rule.cu) with the same decays for
+every row; it applies SiLU to q, k and v as it stages them.  Everything between the two products is float32 in both
+storage dtypes.
+"""
+from __future__ import annotations
+
+from typing import Sequence
+
+import torch
+
+from ..kernels import library as K
+from .base import MIXERS, Mixer, SiteCache, StateSpec, StepContext
+from .linear import Linear
+
+
+@MIXERS.register("lightning")
+class LightningAttention(Mixer):
+    def __init__(self, hidden: int, heads: int, dk: int, dv: int, decay: Sequence[float], norm_eps: float) -> None:
+        super().__init__()
+        if len(decay) != heads:
+            raise ValueError(f"lightning: {len(decay)} decays for {heads} heads")
+        self.hidden, self.heads, self.dk, self.dv, self.norm_eps = hidden, heads, dk, dv, float(norm_eps)
+        self.decay = tuple(float(d) for d in decay)
+        n = heads * dv
+        self.qkvg = self.add_child("qkvg", Linear(hidden, heads * 2 * dk + 2 * n, hidden ** -0.5))
+        self.o = self.add_child("o", Linear(n, hidden, n ** -0.5))
+        self.declare("norm", (n,), ("ones_jitter", 0.1), "vector")
+        self._norm = self._decay = None
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.heads * self.dk * self.dv,), torch.float32)
+
+    def prepare(self, device, dtype) -> None:
+        super().prepare(device, dtype)
+        if self.dk > K.delta_scan_max_dk():
+            raise ValueError(f"lightning: key size {self.dk} exceeds the recurrence kernel's {K.delta_scan_max_dk()}")
+        self._norm = self.param("norm").to(device=device, dtype=torch.float32).contiguous()
+        self._decay = torch.tensor(self.decay, dtype=torch.float32, device=device).view(1, self.heads)
+
+    def forward(self, h: torch.Tensor, ctx: StepContext, site: SiteCache) -> torch.Tensor:
+        T, H, dk, dv = h.shape[0], self.heads, self.dk, self.dv
+        n, v0 = H * dv, 2 * H * dk
+        proj = self.qkvg.forward(h, ctx, out_dtype=torch.float32)
+        o = torch.empty((T, n), dtype=torch.float32, device=h.device)                # (the scan zeroes padding rows)
+        K.state_scan(K.SCAN_LINEAR, proj, (0, H * dk, v0), None, self._decay.expand(T, H), None, site.state, ctx, o, H, H, dk, dv,
+                     silu=True)
+        gated = torch.empty((T, n), dtype=h.dtype, device=h.device)
+        K.group_rms_gate(o, proj[:, v0 + n:], self._norm, gated, n, self.norm_eps, False, "sigmoid")
+        return self.o.forward(gated, ctx, out_dtype=torch.float32)

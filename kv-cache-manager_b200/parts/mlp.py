@@ -1,6 +1,9 @@
-"""Gated feed-forward: down( act(x Wg^T) * (x Wu^T) ), gate and up fused into one matrix
+"""Gated feed-forward: down( act(x Wg^T, x Wu^T) ), gate and up fused into one matrix
 [2I, H] (gate rows first) so that one product feeds the activation kernel
 (``src/model/llama.cpp:120-122``; activation ``src/cuda/kernels.cu:72-82``).
+
+Activations: "silu": silu(g) * u; "clamped": g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit) and u' = u clamped to
+[-limit, limit].
 """
 from __future__ import annotations
 
@@ -13,11 +16,14 @@ from .linear import Linear, STREAM_MAX_BYTES, TCGEN05_GATED_MAX_HIDDEN, TCGEN05_
 
 @FEED_FORWARDS.register("gated_mlp")
 class GatedMLP(FeedForward):
-    def __init__(self, hidden: int, intermediate: int, activation: str = "silu") -> None:
+    def __init__(self, hidden: int, intermediate: int, activation: str = "silu", limit: float = 0.0, alpha: float = 1.702) -> None:
         super().__init__()
-        if activation != "silu":
-            raise ValueError(f"gated_mlp: activation '{activation}' has no kernel (only 'silu')")
-        self.hidden, self.intermediate = hidden, intermediate
+        if activation not in ("silu", "clamped"):
+            raise ValueError(f"gated_mlp: activation '{activation}' has no kernel (only 'silu', 'clamped')")
+        if activation == "clamped" and not (limit > 0):
+            raise ValueError("gated_mlp: the clamped activation needs a positive limit")
+        self.hidden, self.intermediate, self.activation = hidden, intermediate, activation
+        self.limit, self.alpha = float(limit), float(alpha)
         self.gate_up = self.add_child("gate_up", Linear(hidden, 2 * intermediate))
         self.down = self.add_child("down", Linear(intermediate, hidden))
 
@@ -29,7 +35,10 @@ class GatedMLP(FeedForward):
         if (h.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and ctx.options.get("gemm", "auto") in ("auto", "native")
                 and ctx.options.get("fuse", True) and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0
                 and K.gate_up_silu_supported(h.shape[0], self.intermediate, h.shape[1])):
-            K.gate_up_silu(h, w, act)
+            if self.activation == "clamped":
+                K.gate_up_clamped(h, w, act, self.limit, self.alpha)
+            else:
+                K.gate_up_silu(h, w, act)
         elif (h.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and ctx.options.get("fuse", True)
               and ctx.options.get("gemm", "auto") in ("auto", "native", "tcgen05", "pair") and h.shape[0] >= TCGEN05_MIN_ROWS
               and (ctx.options.get("gemm", "auto") != "auto"
@@ -42,10 +51,14 @@ class GatedMLP(FeedForward):
             # (TinyLlama shape: 84 us against 76 + 15; Llama-3-8B shape: the library wins).
             # Beyond that size the two-SM form of the kernel is the faster of this engine's two
             # (Llama-3-8B shape: about 0.4 against 0.58 ms).
-            if ctx.options.get("gemm", "auto") == "pair" or h.shape[1] > TCGEN05_GATED_MAX_HIDDEN:
+            if self.activation == "clamped":                       # (the two-SM form has the SiLU epilogue only)
+                K.gate_up_clamped_tcgen05(h, w, act, self.limit, self.alpha)
+            elif ctx.options.get("gemm", "auto") == "pair" or h.shape[1] > TCGEN05_GATED_MAX_HIDDEN:
                 K.gate_up_silu_tcgen05_pair(h, w, act)
             else:
                 K.gate_up_silu_tcgen05(h, w, act)
+        elif self.activation == "clamped":
+            K.clamped_gate(self.gate_up.forward(h, ctx), act, self.limit, self.alpha)
         else:
             K.silu_mul(self.gate_up.forward(h, ctx), act)
         return self.down.forward(act, ctx, out_dtype)

@@ -9,7 +9,8 @@
 Options (constructor parameters): ``scores`` "sigmoid" takes s = sigmoid(z) instead of the softmax; ``correction``
 declares a learned number per expert that is added to s for the CHOICE only (choice scores may be negative, the
 weights use s itself); ``group_top`` = 2 scores a group by the sum of its two largest choice scores;
-``shared_gate`` False runs the shared expert ungated (the router matrix then has no extra row).
+``shared_gate`` False runs the shared expert ungated (the router matrix then has no extra row); ``renorm`` divides the
+chosen scores by their sum (+ 1e-20) before the scale.
 
 The experts' matrices are stacked ([E, 2F, D] gate rows before up rows, [E, D, F]); the optional
 shared expert is the engine's gated feed-forward and runs for every row; its per-row gate is one
@@ -23,7 +24,7 @@ from typing import Optional
 import torch
 
 from ..kernels import library as K
-from .base import FEED_FORWARDS, FeedForward, StepContext
+from .base import FEED_FORWARDS, ExpertSum, FeedForward, StepContext
 from .mlp import GatedMLP
 
 
@@ -31,7 +32,7 @@ from .mlp import GatedMLP
 class RoutedExperts(FeedForward):
     def __init__(self, hidden: int, experts: int, expert_ff: int, top: int, scale: float = 1.0, groups: int = 1,
                  keep: int = 1, shared_ff: int = 0, scores: str = "softmax", correction: bool = False, group_top: int = 1,
-                 shared_gate: bool = True) -> None:
+                 shared_gate: bool = True, renorm: bool = False) -> None:
         super().__init__()
         if experts < 1 or groups < 1 or experts % groups or not (1 <= keep <= groups):
             raise ValueError(f"routed_experts: {experts} experts do not form {groups} equal groups of which {keep} are kept")
@@ -43,6 +44,7 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: scores 'softmax' | 'sigmoid', group_top 1 | 2")
         self.scores, self.group_top = scores, int(group_top)
         self.shared_gate = bool(shared_gate) and bool(shared_ff)
+        self.renorm = bool(renorm)
         self.shared: Optional[GatedMLP] = None
         if shared_ff:
             self.shared = self.add_child("shared", GatedMLP(hidden, shared_ff))
@@ -69,13 +71,28 @@ class RoutedExperts(FeedForward):
         """Returns float32 rows (``out_dtype`` is accepted for the feed-forward interface and must allow that)."""
         if out_dtype not in (None, torch.float32):
             raise ValueError("routed_experts: the weighted sum is float32")
+        y, work, wt, gate = self._experts(h, ctx)
+        shared_y = self.shared.forward(h, ctx, out_dtype=torch.float32) if self.shared is not None else None
+        out = torch.empty((h.shape[0], self.hidden), dtype=torch.float32, device=h.device)
+        K.moe_combine(y, work, wt, self.experts, shared_y, gate, out)
+        return out
+
+    def forward_unsummed(self, h: torch.Tensor, ctx: StepContext):
+        """The experts' outputs as an ``ExpertSum`` for a caller that forms the weighted sum itself; with a shared expert
+        the summed rows as ``forward`` returns them."""
+        if self.shared is not None:
+            return self.forward(h, ctx)
+        y, work, wt, _ = self._experts(h, ctx)
+        return ExpertSum(y, work, wt, self.experts)
+
+    def _experts(self, h: torch.Tensor, ctx: StepContext):
         M, D, top = h.shape[0], self.hidden, self.top
         dev = h.device
         idx = torch.empty((M, top), dtype=torch.int32, device=dev)
         wt = torch.empty((M, top), dtype=torch.float32, device=dev)
         gate = torch.empty((M,), dtype=torch.float32, device=dev) if self.shared_gate else None
         K.moe_route(h, self._router, self.experts, self.groups, self.keep, top, self.scale, idx, wt, gate, self.scores,
-                    self._correction, self.group_top)
+                    self._correction, self.group_top, self.renorm)
         work = torch.empty((K.moe_work_ints(M, top, self.experts),), dtype=torch.int32, device=dev)
         act = torch.empty((M * top, self.expert_ff), dtype=h.dtype, device=dev)
         y = torch.empty((M * top, D), dtype=torch.float32, device=dev)
@@ -84,7 +101,4 @@ class RoutedExperts(FeedForward):
                 and K.moe_tcgen05_supported(self.expert_ff, D) and h.stride(0) % 8 == 0):
             xs = torch.empty((M * top, D), dtype=h.dtype, device=dev)        # tensor-core products
         K.moe_experts(h, self._wgu, self._wd, idx, work, act, y, xs)
-        shared_y = self.shared.forward(h, ctx, out_dtype=torch.float32) if self.shared is not None else None
-        out = torch.empty((M, D), dtype=torch.float32, device=dev)
-        K.moe_combine(y, work, wt, self.experts, shared_y, gate, out)
-        return out
+        return y, work, wt, gate

@@ -11,7 +11,7 @@ from typing import Optional
 import torch
 
 from ..kernels import library as K
-from .base import NORMS, ClosingNorm, Norm, settle
+from .base import NORMS, ClosingNorm, Norm, settle, split_pending
 
 
 @NORMS.register("rmsnorm")
@@ -72,6 +72,28 @@ class DynamicTanh(Norm):
             pending = [(pending if pending.dtype == torch.float32 else pending.float(), 1.0)]
         f = self._f32
         K.dyt_norm(x, pending, f["weight"], f["bias"], f["alpha"], out, rows)
+
+
+@NORMS.register("rmsnorm_f32")
+class Float32RMSNorm(Norm):
+    """RMS norm all in float32 up to the one rounding of its result: out = w * x / sqrt(mean(x^2) + eps).  ``pending`` may
+    be a list of (float32 tensor, scale) pairs and one ``ExpertSum`` (a block whose sublayers' outputs are summed hands
+    them on unsummed); ``forward`` reads the stream with them and leaves x as it is: the final norm, with its row gather.
+    The "parallel_norms" block uses two of these (``multiplier``, ``eps``) in one kernel."""
+
+    def __init__(self, hidden: int, eps: float, init=("ones",)) -> None:
+        super().__init__()
+        self.hidden, self.eps = hidden, float(eps)
+        self.declare("weight", (hidden,), init, "vector")
+        self.multiplier: Optional[torch.Tensor] = None
+
+    def prepare(self, device, dtype) -> None:
+        super().prepare(device, dtype)
+        self.multiplier = self.param("weight").to(device=device, dtype=torch.float32).contiguous()
+
+    def forward(self, x: torch.Tensor, pending, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        dense, experts = split_pending(pending)
+        K.norm_pair(x, dense, experts, self.multiplier, self.eps, out, rows=rows)
 
 
 @NORMS.register("rmsnorm_offset")

@@ -6,9 +6,15 @@ applied to pairs (j, j + rotary_dim/2) ("half", the reference's pairing,
 elements of every q and k head.  The frequency table is float32, computed once on the host in
 float64; a scaled variant only needs another table.  ``NoPositionEncoding`` leaves q and k as
 they are.
+
+``scaling`` (YaRN): {factor, original, fast, slow}.  With turns(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta), the
+pair index at which a wave makes t turns over ``original`` positions, the frequencies between lo = max(floor(turns(fast)), 0)
+and hi = min(ceil(turns(slow)), rotary_dim - 1) pass linearly from f_i to f_i / factor, and cosines and sines are multiplied
+by ``amplitude`` = 0.1 ln(factor) + 1.
 """
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -19,7 +25,7 @@ from .base import POSITION_ENCODINGS, PositionEncoding
 @POSITION_ENCODINGS.register("rope")
 class RotaryEmbedding(PositionEncoding):
     def __init__(self, head_dim: int, theta: float, rotary_dim: Optional[int] = None,
-                 pairing: str = "half") -> None:
+                 pairing: str = "half", scaling: Optional[dict] = None) -> None:
         super().__init__()
         self.head_dim = head_dim
         self.theta = float(theta)
@@ -29,12 +35,21 @@ class RotaryEmbedding(PositionEncoding):
         if pairing not in ("half", "interleaved"):
             raise ValueError(f"unknown rotary pairing '{pairing}'")
         self.interleaved = pairing == "interleaved"
+        self.scaling = dict(scaling) if scaling else None
+        self.amplitude = 0.1 * math.log(self.scaling["factor"]) + 1.0 if self.scaling else 1.0
         self.inv_freq: Optional[torch.Tensor] = None
 
     def frequency_table(self) -> torch.Tensor:
         j = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
-        return (1.0 / torch.pow(torch.tensor(self.theta, dtype=torch.float64),
-                                2.0 * j / self.rotary_dim)).to(torch.float32)
+        f = 1.0 / torch.pow(torch.tensor(self.theta, dtype=torch.float64), 2.0 * j / self.rotary_dim)
+        if self.scaling:
+            def turns(t: float) -> float:
+                return self.rotary_dim * math.log(self.scaling["original"] / (2.0 * math.pi * t)) / (2.0 * math.log(self.theta))
+            lo = max(math.floor(turns(self.scaling["fast"])), 0)
+            hi = min(math.ceil(turns(self.scaling["slow"])), self.rotary_dim - 1)
+            ramp = ((j - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            f = f / self.scaling["factor"] * ramp + f * (1.0 - ramp)
+        return f.to(torch.float32)
 
     def prepare(self, device, dtype) -> None:
         self.inv_freq = self.frequency_table().to(device)
@@ -46,4 +61,5 @@ class NoPositionEncoding(PositionEncoding):
         super().__init__()
         self.rotary_dim = 0
         self.interleaved = False
+        self.amplitude = 1.0
         self.inv_freq = None
