@@ -525,6 +525,64 @@ def lobutar_work(z, T, ctx, decode):
     }
 
 
+# --compare bimepel: the Bimepel design (parallel layers with a norm for each sublayer and a token shift in every layer;
+# chunked attention with per-head norms and an output gate; lightning attention; clamped gated feed-forward or routed
+# experts with normalised weights; a looped span of layers) beside the Llama decoder at equal width, number of layer
+# runs, head count and active feed-forward size.
+BIMEPEL_SIZES = {
+    "p2048": dict(width=2048, order=("attention", "lightning", "attention", "lightning"), loop=None, heads=16, kv_heads=4, dim=128,
+                  chunk=1024, experts=32, moe_top=8, expert_ff=512, llama_ff=4096),
+    "p4096": dict(width=4096, order=("attention", "lightning", "attention"), loop=(0, 2, 2), heads=32, kv_heads=8, dim=128,
+                  chunk=1024, experts=64, moe_top=8, expert_ff=1024, llama_ff=8192),
+}
+
+
+def bimepel_configs(z):
+    """(Bimepel config, Llama config) of one size.  Attention layers carry the dense feed-forward, lightning layers the
+    experts (the chosen ones = Llama's inner size).  Llama gets as many layers as Bimepel has layer runs."""
+    from kvcm.config import LlamaConfig, config_from_dict
+    D, H, G, d = z["width"], z["heads"], z["kv_heads"], z["dim"]
+    rot = {"base": 500000.0, "dims": d, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}
+    layers = []
+    for kind in z["order"]:
+        if kind == "attention":
+            layers.append({"type": kind, "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "rot": rot,
+                                                   "mask": {"size": z["chunk"]}},
+                           "mlp": {"kind": "dense", "ff": z["llama_ff"], "limit": 7.0}})
+        else:
+            layers.append({"type": kind, "mixer": {"heads": H, "dim": d, "vdim": d, "decay": [1.0 - 2.0 ** (-1 - 8.0 * h / H) for h in range(H)]},
+                           "mlp": {"kind": "moe", "expert": {"ff": z["expert_ff"]},
+                                   "router": {"experts": z["experts"], "top": z["moe_top"], "scale": 2.0}}})
+    top = {"architecture": "Bimepel", "vocab": COMPARE_VOCAB, "width": D, "norm": {"eps": 1e-6}, "layers": layers}
+    if z["loop"]:
+        top["loop"] = dict(zip(("start", "stop", "times"), z["loop"]))
+    lla = LlamaConfig(architecture="LlamaForCausalLM", vocab_size=COMPARE_VOCAB, hidden_size=D, intermediate_size=z["llama_ff"],
+                      num_hidden_layers=len(rivetar_runs(z)), num_attention_heads=H, num_key_value_heads=G, head_dim=d,
+                      max_position_embeddings=4096, rope_theta=10000.0, rms_norm_eps=1e-6, tie_word_embeddings=False)
+    return config_from_dict(top), lla
+
+
+def bimepel_work(z, T, ctx, decode):
+    """What the families of one Bimepel step have to do at least: flops, or bytes they must move."""
+    D, H, G, d, C = z["width"], z["heads"], z["kv_heads"], z["dim"], z["chunk"]
+    runs = rivetar_runs(z)
+    n_att, n_lin, L = runs.count("attention"), runs.count("lightning"), len(runs)
+    own = (ctx - 1) % C + 1                                       # keys of the last position's chunk
+    seen = T * own if decode else sum(i % C + 1 for i in range(T))
+    hit = min(z["experts"], T * z["moe_top"])
+    return {
+        "attention": dict(flops=4.0 * H * d * seen * n_att, bytes=2.0 * 2 * G * d * T * own * n_att if decode else None),
+        "state_scan": dict(flops=T * 4.0 * H * d * d * n_lin, bytes=8.0 * T * H * d * d * n_lin if decode else None),
+        "moe_experts_tcgen05": dict(flops=2.0 * T * z["moe_top"] * 3 * z["expert_ff"] * D * n_lin,
+                                    bytes=2.0 * hit * 3 * z["expert_ff"] * D * n_lin if decode else None),
+        "feed_forward": dict(flops=2.0 * T * 3 * z["llama_ff"] * D * n_att, bytes=2.0 * 3 * z["llama_ff"] * D * n_att if decode else None),
+        # the stream read and written, the pending outputs read (two, or the mixer's and the chosen experts'), two outputs
+        "norm_pair": dict(flops=None, bytes=T * D * ((4.0 * 4 + 4.0) * n_att + (4.0 * (3 + z["moe_top"]) + 4.0) * n_lin)),
+        "group_rms_gate": dict(flops=None, bytes=T * H * d * (4.0 + 4.0 + 2.0) * n_lin),
+        "gate_mul": dict(flops=None, bytes=T * H * d * (2.0 + 4.0 + 2.0) * n_att),
+    }
+
+
 def compare_main(args) -> int:
     import torch
     from kvcm.config import EngineConfig, KVManagerConfig, SchedulerConfig
@@ -535,6 +593,7 @@ def compare_main(args) -> int:
     sizes, configs, first_work = {"bifatar": (BIFATAR_SIZES, bifatar_configs, bifatar_work),
                                   "rivetar": (RIVETAR_SIZES, rivetar_configs, rivetar_work),
                                   "lobutar": (LOBUTAR_SIZES, lobutar_configs, lobutar_work),
+                                  "bimepel": (BIMEPEL_SIZES, bimepel_configs, bimepel_work),
                                   "tolanex": (COMPARE_SIZES, compare_configs, tolanex_work)}[first]
     out = {"compare": f"{first} beside llama at equal width, depth and (active) feed-forward size", "dtype": "bf16",
            "data": "synthetic: random weights, uniform random token ids", "peaks": pk, "sizes": {}}
@@ -544,7 +603,7 @@ def compare_main(args) -> int:
             continue
         if first == "bifatar":
             z = dict(z, layers=len(z["order"]), top=1, ff=z["llama_ff"], shared=0)      # the keys llama_work reads
-        elif first == "rivetar":
+        elif first in ("rivetar", "bimepel"):
             z = dict(z, layers=len(rivetar_runs(z)), top=1, ff=z["llama_ff"], shared=0)
         elif first == "lobutar":
             z = dict(z, layers=len(z["order"]), top=1, ff=z["llama_ff"], shared=0)
@@ -702,10 +761,10 @@ def main() -> int:
                          "'native' this engine's kernels only, 'library' the library wherever it can stand")
     ap.add_argument("--only", default="all", choices=["all", "prefill"],
                     help="'prefill': run only the 2,048-token prefill step and print its numbers (for profiling)")
-    ap.add_argument("--compare", default="", choices=["", "tolanex", "bifatar", "rivetar", "lobutar"],
-                    help="'tolanex' | 'bifatar' | 'rivetar' | 'lobutar': instead of the default workload, prefill and decode of that design beside "
+    ap.add_argument("--compare", default="", choices=["", "tolanex", "bifatar", "rivetar", "lobutar", "bimepel"],
+                    help="'tolanex' | 'bifatar' | 'rivetar' | 'lobutar' | 'bimepel': instead of the default workload, prefill and decode of that design beside "
                          "the Llama decoder at equal sizes, with device time per kernel family")
-    ap.add_argument("--size", default="all", choices=["all"] + sorted(COMPARE_SIZES) + sorted(BIFATAR_SIZES) + sorted(RIVETAR_SIZES) + sorted(LOBUTAR_SIZES),
+    ap.add_argument("--size", default="all", choices=["all"] + sorted(COMPARE_SIZES) + sorted(BIFATAR_SIZES) + sorted(RIVETAR_SIZES) + sorted(LOBUTAR_SIZES) + sorted(BIMEPEL_SIZES),
                     help="with --compare: one size only")
     args = ap.parse_args()
 

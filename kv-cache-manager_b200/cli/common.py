@@ -96,6 +96,22 @@ def _lobutar_mini():
             ]}
 
 
+def _bimepel_mini():
+    """A small Bimepel: chunked attention with a scaled rotation and routed experts, looped together with a lightning
+    layer, behind a lightning layer without a feed-forward; attention without chunks behind the loop."""
+    rot = {"base": 10000.0, "dims": 32, "scaling": {"factor": 4.0, "original": 256, "fast": 32.0, "slow": 1.0}}
+    attn = {"heads": 6, "kv_heads": 2, "dim": 64, "vdim": 48, "scale": 0.125, "rot": rot}
+    return {"architecture": "Bimepel", "vocab": 1000, "width": 384, "norm": {"eps": 1e-5}, "loop": {"start": 1, "stop": 3, "times": 2},
+            "layers": [
+                {"type": "lightning", "mixer": {"heads": 3, "dim": 32, "vdim": 64, "decay": [0.75, 0.95, 0.995]}, "mlp": None},
+                {"type": "attention", "mixer": dict(attn, mask={"size": 90}),
+                 "mlp": {"kind": "moe", "expert": {"ff": 128}, "router": {"experts": 16, "top": 3, "scale": 1.5}}},
+                {"type": "lightning", "mixer": {"heads": 4, "dim": 64, "vdim": 96, "decay": [0.5, 0.9, 0.98, 0.999]},
+                 "mlp": {"kind": "dense", "ff": 640, "limit": 2.0}},
+                {"type": "attention", "mixer": attn, "mlp": {"kind": "dense", "ff": 640, "limit": 2.0}},
+            ]}
+
+
 PRESETS = {
     # name: (config.json keys, seed, norm jitter); keys with "architecture" go through the registry,
     # the others are those of a Llama dense decoder
@@ -103,6 +119,7 @@ PRESETS = {
     "bifatar-mini": (_bifatar_mini(), 5, 0.1),
     "rivetar-mini": (_rivetar_mini(), 7, 0.1),
     "lobutar-mini": (_lobutar_mini(), 8, 0.1),
+    "bimepel-mini": (_bimepel_mini(), 9, 0.1),
     "tiny-a": (dict(vocab_size=256, hidden_size=64, intermediate_size=172, num_hidden_layers=2,
                     num_attention_heads=4, num_key_value_heads=2, head_dim=16, max_position_embeddings=128,
                     rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=False), 0, 0.0),

@@ -138,7 +138,10 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int
     float* ch = gb + G;                                        // choice scores: -inf once taken
     if (sigmoid_scores) {
       __syncwarp();
-      for (int e = lane; e < E; e += 32) z[e] = 1.f / (1.f + expf(-z[e]));
+      for (int e = lane; e < E; e += 32) {
+        ch[e] = z[e];                                          // (the sigmoid keeps the order; in float it makes large logits equal)
+        z[e] = 1.f / (1.f + expf(-z[e]));
+      }
     } else {
       float m = -INFINITY;
       for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
@@ -149,11 +152,12 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int
       __syncwarp();
       for (int e = lane; e < E; e += 32) z[e] = expf(z[e] - m) / sum;
     }
-    for (int e = lane; e < E; e += 32) ch[e] = z[e] + (correction ? correction[e] : 0.f);
+    const bool limited = G > 1 && keep < G;
+    if (!sigmoid_scores || correction || limited)
+      for (int e = lane; e < E; e += 32) ch[e] = z[e] + (correction ? correction[e] : 0.f);
     if (has_gate && lane == 0) gate_out[row] = 1.f / (1.f + expf(-z[E]));
     __syncwarp();
     const int per = E / G;
-    const bool limited = G > 1 && keep < G;
     if (limited) {
       for (int g = lane; g < G; g += 32) {
         float best = -INFINITY, second = -INFINITY;            // the group's two largest choice scores

@@ -1176,12 +1176,13 @@ SCAN_DELTA, SCAN_DELTA_CHANNEL, SCAN_LINEAR, SCAN_LINEAR_CHANNEL = 0, 1, 2, 3
 
 def state_scan(mode: int, qkv: torch.Tensor, bases, beta: Optional[torch.Tensor], g: Optional[torch.Tensor],
                gd: Optional[torch.Tensor], state: torch.Tensor, ctx, out: torch.Tensor, heads: int, qk_heads: int,
-               dk: int, dv: int, silu: bool = False) -> None:
+               dk: int, dv: int, silu: bool = False, seqs: Optional[int] = None) -> None:
     """The matrix-state recurrences over every request's rows of the step, from and into its state row
     (csrc/cuda/delta_rule.cu).  ``bases`` = where a row's q, k and v start; ``beta`` [T, >= heads] (a view
     with a row stride is fine), ``g`` likewise (one decay per head) or ``gd`` [T, heads*dk] (one per head
     and key channel).  The linear forms take ``beta`` None (it then counts as one) and ``silu``: q, k and v are
-    projections that pass SiLU first.  A row stride of zero in ``g`` gives every row the same decays."""
+    projections that pass SiLU first.  A row stride of zero in ``g`` gives every row the same decays.
+    ``seqs``: only the batch's first entries, which are its single-row ones."""
     _cuda(qkv, beta, g, gd, state, out)
     _need(all(t is None or t.dtype == torch.float32 for t in (qkv, beta, g, gd, state, out)), "state_scan: float32")
     linear = mode in (SCAN_LINEAR, SCAN_LINEAR_CHANNEL)
@@ -1195,8 +1196,35 @@ def state_scan(mode: int, qkv: torch.Tensor, bases, beta: Optional[torch.Tensor]
           and state.shape[1] >= heads * dk * dv and (beta is None or beta.shape[1] >= heads), "state_scan: shapes")
     _check(_lib().kvcm_state_scan(int(mode), _p(qkv), C, qb, kb, vb, _p(beta), beta.stride(0) if beta is not None else 0, _p(g),
                                   g.stride(0) if g is not None else 0, _p(gd), _p(state), _ll(state.stride(0)),
-                                  _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out), qkv.shape[0],
-                                  ctx.seqs, heads, qk_heads, dk, dv, int(bool(silu)), _stream()), "state_scan", f"(mode={mode}, dk={dk}, dv={dv})")
+                                  _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out),
+                                  qkv.shape[0] if seqs is None else int(seqs), ctx.seqs if seqs is None else int(seqs), heads, qk_heads,
+                                  dk, dv, int(bool(silu)), _stream()), "state_scan", f"(mode={mode}, dk={dk}, dv={dv})")
+
+
+def linear_chunk_supported(dk: int) -> bool:
+    return int(dk) <= int(_lib().kvcm_linear_chunk_max_dk())
+
+
+def linear_chunk(qkv: torch.Tensor, bases, decay: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int,
+                 qk_heads: int, dk: int, dv: int, silu: bool = False) -> None:
+    """``state_scan``'s linear form with one constant decay per head (``decay`` float32 [heads]), in chunks of 64 tokens on the
+    tensor cores, for the step's portions of more than one token (csrc/cuda/linear_chunk.cu); rows of single-row
+    entries are left alone.  For a 16-bit model: q, k and v are bfloat16 operands there."""
+    _cuda(qkv, decay, state, out)
+    _need(all(t.dtype == torch.float32 for t in (qkv, decay, state, out)), "linear_chunk: float32")
+    _need(qkv.is_contiguous() and out.is_contiguous() and state.is_contiguous() and decay.is_contiguous() and decay.numel() == heads,
+          "linear_chunk: layout")
+    qb, kb, vb = (int(b) for b in bases)
+    C = qkv.shape[1]
+    _need(max(qb, kb) + qk_heads * dk <= C and vb + heads * dv <= C and out.shape == (qkv.shape[0], heads * dv)
+          and state.shape[1] >= heads * dk * dv and ctx.tile_rows == 64, "linear_chunk: shapes")
+    tiles = ctx.prefill_tiles
+    carry = torch.empty((tiles, heads, dk, dv), dtype=torch.float32, device=qkv.device)
+    _check(_lib().kvcm_linear_chunk(_p(qkv), C, qb, kb, vb, _p(decay), _p(carry), _p(state), _ll(state.stride(0)), _p(ctx.tile_seq),
+                                    _p(ctx.tile_q0), _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out), tiles,
+                                    heads, qk_heads, dk, dv, int(bool(silu)), _stream()), "linear_chunk", f"(dk={dk}, dv={dv})")
+    global _launches
+    _launches += 2                          # outer, carry, read
 
 
 def delta_prepare_channel(qkv: torch.Tensor, b: torch.Tensor, beta: torch.Tensor, a: torch.Tensor, a_log: torch.Tensor,

@@ -10,8 +10,10 @@ by sigmoid(W_g h), and go through the output projection.
 
 State of a request: one float32 row per call site, S of every head.  One product gives q | k | v | g (float32 result).
 The recurrence is the engine's matrix-state scan in its linear form (csrc/cuda/delta_rule.cu) with the same decays for
-every row; it applies SiLU to q, k and v as it stages them.  Everything between the two products is float32 in both
-storage dtypes.
+every row; it applies SiLU to q, k and v as it stages them.  With bfloat16 storage the portions of more than a few
+tokens take the chunked form on the tensor cores instead (csrc/cuda/linear_chunk.cu; ``options['scan']``: 'tokens' forces
+the token-by-token kernel, 'chunks' the chunked one).  Everything between the two products is float32 in both storage
+dtypes, but for the chunked form's q, k and v, which are bfloat16 operands.
 """
 from __future__ import annotations
 
@@ -22,6 +24,9 @@ import torch
 from ..kernels import library as K
 from .base import MIXERS, Mixer, SiteCache, StateSpec, StepContext
 from .linear import Linear
+
+
+CHUNKED_MIN_TOKENS = 32       # portions at least this long take the chunked form
 
 
 @MIXERS.register("lightning")
@@ -53,8 +58,15 @@ class LightningAttention(Mixer):
         n, v0 = H * dv, 2 * H * dk
         proj = self.qkvg.forward(h, ctx, out_dtype=torch.float32)
         o = torch.empty((T, n), dtype=torch.float32, device=h.device)                # (the scan zeroes padding rows)
-        K.state_scan(K.SCAN_LINEAR, proj, (0, H * dk, v0), None, self._decay.expand(T, H), None, site.state, ctx, o, H, H, dk, dv,
-                     silu=True)
+        bases, decay = (0, H * dk, v0), self._decay.expand(T, H)
+        mode = ctx.options.get("scan", "auto")
+        if (mode == "chunks" or (mode == "auto" and h.dtype == torch.bfloat16 and ctx.max_q_len >= CHUNKED_MIN_TOKENS)) \
+                and ctx.prefill_tiles > 0 and K.linear_chunk_supported(dk):
+            if ctx.decode_seqs:                                                      # the single-row entries come first
+                K.state_scan(K.SCAN_LINEAR, proj, bases, None, decay, None, site.state, ctx, o, H, H, dk, dv, silu=True, seqs=ctx.decode_seqs)
+            K.linear_chunk(proj, bases, self._decay, site.state, ctx, o, H, H, dk, dv, silu=True)
+        else:
+            K.state_scan(K.SCAN_LINEAR, proj, bases, None, decay, None, site.state, ctx, o, H, H, dk, dv, silu=True)
         gated = torch.empty((T, n), dtype=h.dtype, device=h.device)
         K.group_rms_gate(o, proj[:, v0 + n:], self._norm, gated, n, self.norm_eps, False, "sigmoid")
         return self.o.forward(gated, ctx, out_dtype=torch.float32)

@@ -118,6 +118,7 @@ class Replayer:
         self.runner, self.kv, self.slots, self.live = (self.session.runner, self.session.kv, self.session.slots,
                                                        self.session.live)
         self.pages_seen: List[int] = []
+        self.pages_seen_of: List[set] = [set() for _ in range(self.runner.num_groups)]      # per layer group
         self.page_owners: Dict[int, set] = {}
 
     def step(self, entries: Sequence[dict], end: Sequence[str] = ()) -> Optional[torch.Tensor]:
@@ -125,6 +126,8 @@ class Replayer:
         for e in entries:
             seq = self.live[e["id"]]
             self.pages_seen.extend(p for p in seq.table(0) if p >= 0)
+            for g, seen in enumerate(self.pages_seen_of):
+                seen.update(p for p in seq.table(g) if p >= 0)
             for p in seq.table(0):
                 if p >= 0:
                     self.page_owners.setdefault(p, set()).add(seq.id)
@@ -133,14 +136,15 @@ class Replayer:
             self.session.release(rid)
         return None if out is None else out.float().cpu()
 
-    def stray_writes(self) -> List[int]:
-        """Pages of the first layer group that no request ever held and that are no longer all
-        zero (pools start zero-filled): a kernel wrote through a wrong page number or slot."""
+    def stray_writes(self, group: int = 0) -> List[int]:
+        """Pages of a layer group that no request was seen to hold after a step and that are no longer all zero
+        (pools start zero-filled): a kernel wrote through a wrong page number or slot.  For groups that keep every
+        key (pages that a window or chunk passes inside one step are never seen)."""
         pools = self.runner.pools
-        never = sorted(set(range(self.kv.num_blocks())) - set(self.pages_seen))
+        never = sorted(set(range(self.kv.num_blocks())) - self.pages_seen_of[group])
         bad = []
         for page in never:
-            if any(bool(t[:, page].count_nonzero()) for t in (pools.k[0], pools.v[0]) if t is not None):
+            if any(bool(t[:, page].count_nonzero()) for t in (pools.k[group], pools.v[group]) if t is not None):
                 bad.append(page)
         return bad
 
