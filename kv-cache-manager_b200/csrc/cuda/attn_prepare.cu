@@ -210,6 +210,127 @@ attn_prepare_kernel(AttnPrepareParams p) {
   }
 }
 
+// The same for mixers whose heads need nothing of one another before the attention (no whole-projection norm, no bias, one
+// map a head, values neither kept, mixed nor turned) and whose heads have at most 128 elements, in quads: a warp takes a
+// head, a lane four neighbouring elements in registers; the partner of a rotate-half pair comes by shuffle.  The loads
+// of up to four heads of a warp are in flight together.
+__device__ __forceinline__ void store_quad(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store_quad(bf16* p, const float (&v)[4]) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  uint2 raw;
+  raw.x = *reinterpret_cast<const uint32_t*>(&a);
+  raw.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+__device__ __forceinline__ float quad_inv_rms(const float (&x)[4], int width, float eps) {
+  const float ss = warp_sum(fmaf(x[0], x[0], fmaf(x[1], x[1], fmaf(x[2], x[2], x[3] * x[3]))));     // (elements beyond the head are zero)
+  return 1.f / sqrtf(ss / float(width) + eps);
+}
+
+constexpr int kHeadBatch = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+attn_prepare_heads_kernel(AttnPrepareParams p) {
+  extern __shared__ __align__(16) float cs_table[];  // cosines, sines of the row's angles
+  pdl_launch_dependents();
+  const int r = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarps = blockDim.x >> 5;
+  const int half = p.rot / 2;
+  if (half > 0) {
+    const float pos = float(p.positions[r]);
+    for (int j = tid; j < half; j += blockDim.x) {
+      float sn, cs;
+      sincosf(pos * p.inv_freq[j], &sn, &cs);
+      cs_table[j] = cs * p.amplitude;
+      cs_table[half + j] = sn * p.amplitude;
+    }
+  }
+  const int slot = p.slot_mapping ? p.slot_mapping[r] : -1;
+  const int page = slot >= 0 ? slot / p.block_size : 0, off = slot >= 0 ? slot - page * p.block_size : 0;
+  const size_t base = (size_t(page) * p.nkv * p.block_size + off) * p.HD;
+  const size_t head_stride = size_t(p.block_size) * p.HD;
+  __syncthreads();
+  pdl_wait();
+  const float* src = p.proj + size_t(r) * p.ldp;
+  const int nqk = p.nh + p.nkv, units = nqk + p.nkv, i = 4 * lane;
+  for (int u0 = warp; u0 < units; u0 += kHeadBatch * nwarps) {
+    float x[kHeadBatch][4];
+#pragma unroll
+    for (int b = 0; b < kHeadBatch; ++b) {
+      const int u = u0 + b * nwarps;
+      x[b][0] = x[b][1] = x[b][2] = x[b][3] = 0.f;
+      if (u < units && i < (u < nqk ? p.dk : p.dv)) {
+        const float4 v = *reinterpret_cast<const float4*>(src + (u < nqk ? u * p.dk : nqk * p.dk + (u - nqk) * p.dv) + i);
+        x[b][0] = v.x; x[b][1] = v.y; x[b][2] = v.z; x[b][3] = v.w;
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < kHeadBatch; ++b) {
+      const int u = u0 + b * nwarps;
+      if (u >= units) break;
+      if (u < nqk) {
+        const bool is_q = u < p.nh;
+        if (p.hq) {
+          const float f = quad_inv_rms(x[b], p.dk, p.eps);
+          if (i < p.dk) {
+            const float4 w = *reinterpret_cast<const float4*>((is_q ? p.hq : p.hk) + i);
+            x[b][0] *= f * w.x; x[b][1] *= f * w.y; x[b][2] *= f * w.z; x[b][3] *= f * w.w;
+          }
+        }
+        if (half > 0 && p.interleaved) {
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const int j = (i + e) / 2;
+            if (j < half) {
+              float ra, rb;
+              rotate_pair(x[b][e], x[b][e + 1], cs_table[j], cs_table[half + j], ra, rb);
+              x[b][e] = ra;
+              x[b][e + 1] = rb;
+            }
+          }
+        } else if (half > 0) {                       // (half % 4 == 0: a quad's partners are one quad)
+          const bool low = i < half, in = i < p.rot;
+          const int from = in ? (low ? lane + half / 4 : lane - half / 4) : lane;
+          float y[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[e] = __shfl_sync(0xffffffffu, x[b][e], from);
+          if (in) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int j = low ? i + e : i + e - half;
+              float ra, rb;
+              rotate_pair(low ? x[b][e] : y[e], low ? y[e] : x[b][e], cs_table[j], cs_table[half + j], ra, rb);
+              x[b][e] = low ? ra : rb;
+            }
+          }
+        }
+        if (p.head_norm) {
+          const float f = quad_inv_rms(x[b], p.dk, p.eps);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[b][e] *= f;
+        }
+        if (i >= p.HD) continue;
+        if (is_q) store_quad(reinterpret_cast<T*>(p.q_out) + (size_t(r) * p.nh + u) * p.HD + i, x[b]);
+        else if (slot >= 0) store_quad(reinterpret_cast<T*>(p.k_cache) + base + (u - p.nh) * head_stride + i, x[b]);
+      } else {
+        if (p.v_norm) {
+          const float f = quad_inv_rms(x[b], p.dv, p.eps);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[b][e] *= f;
+        }
+        if (slot >= 0 && i < p.HD) store_quad(reinterpret_cast<T*>(p.v_cache) + base + (u - nqk) * head_stride + i, x[b]);
+      }
+    }
+  }
+}
+
+static bool heads_are_quads(const AttnPrepareParams& p) {
+  auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  return !p.bias && !p.wq && p.maps == 1 && !p.v_keep && !p.v_first && !p.v_inv_freq && p.HD <= 128 && (p.HD % 4) == 0 &&
+         (p.dk % 4) == 0 && (p.dv % 4) == 0 && (p.ldp % 4) == 0 && (p.interleaved || (p.rot % 8) == 0) && aligned(p.proj) &&
+         aligned(p.hq) && aligned(p.hk) && aligned(p.q_out) && aligned(p.k_cache) && aligned(p.v_cache);
+}
+
 template <typename T>
 int launch_attn_prepare(const AttnPrepareParams& p, int rows, cudaStream_t s) {
   if (rows == 0) return 0;
@@ -222,6 +343,8 @@ int launch_attn_prepare(const AttnPrepareParams& p, int rows, cudaStream_t s) {
     const cudaError_t e = cudaFuncSetAttribute(attn_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     if (e != cudaSuccess) return int(e);
   }
+  if (heads_are_quads(p))
+    return pdl_launch(attn_prepare_heads_kernel<T>, dim3(rows), dim3(256), size_t(p.rot) * sizeof(float), s, p);
   // a row of a few thousand elements is a chain of short passes: more threads, fewer turns each
   const int threads = (p.nh * p.maps + 2 * p.nkv) * p.HD >= 2048 ? 512 : 256;
   return pdl_launch(attn_prepare_kernel<T>, dim3(rows), dim3(threads), smem, s, p);

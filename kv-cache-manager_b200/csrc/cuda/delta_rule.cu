@@ -785,6 +785,56 @@ group_rms_gate_wide_kernel(const float* __restrict__ o, const Z* __restrict__ z,
   }
 }
 
+// The wide form without a skip and with the gate behind the norm, four neighbouring elements a thread (16-byte
+// accesses): a row's values and gates are all asked for before the reduction.
+__device__ __forceinline__ float4 rms_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 rms_load4(const bf16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void rms_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void rms_store4(bf16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<const uint32_t*>(&a);
+  raw.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+template <typename T, typename Z, int NC>      // NC: quads a thread keeps (group <= 256 * 4 * NC)
+__global__ void __launch_bounds__(256)
+group_rms_gate_vec_kernel(const float* __restrict__ o, const Z* __restrict__ z, int ldz, const float* __restrict__ w, int wlen,
+                          T* __restrict__ out, int n, int group, int act, float eps) {
+  __shared__ float scratch[33];
+  const int row = blockIdx.x, i0 = blockIdx.y * group;
+  float4 v[NC], gz[NC];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int j = 4 * (threadIdx.x + c * blockDim.x);
+    if (j >= group) continue;
+    v[c] = rms_load4(o + size_t(row) * n + i0 + j);
+    gz[c] = rms_load4(z + size_t(row) * ldz + i0 + j);
+  }
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int j = 4 * (threadIdx.x + c * blockDim.x);
+    if (j >= group) continue;
+    ss = fmaf(v[c].x, v[c].x, fmaf(v[c].y, v[c].y, fmaf(v[c].z, v[c].z, fmaf(v[c].w, v[c].w, ss))));
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / float(group) + eps);
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int j = 4 * (threadIdx.x + c * blockDim.x);
+    if (j >= group) continue;
+    const float4 ww = rms_load4(w + (wlen == group ? j : (i0 + j) % wlen));            // (wlen % 4 == 0)
+    rms_store4(out + size_t(row) * n + i0 + j,
+               make_float4(v[c].x * inv * ww.x * gate_act(gz[c].x, act), v[c].y * inv * ww.y * gate_act(gz[c].y, act),
+                           v[c].z * inv * ww.z * gate_act(gz[c].z, act), v[c].w * inv * ww.w * gate_act(gz[c].w, act)));
+  }
+}
+
 template <typename T, typename Z>
 static int launch_group_rms_gate(const float* o, const void* z, int ldz, const float* skip, int lds, const float* skip_coef,
                                  int head, const float* w, int wlen, void* out, int rows, int n, int group, int gate_first,
@@ -792,6 +842,19 @@ static int launch_group_rms_gate(const float* o, const void* z, int ldz, const f
   if (rows == 0) return 0;
   if (group < 1 || n % group || wlen < 1 || (skip && head < 1)) return KVCM_ERR_UNSUPPORTED;
   const int groups = n / group;
+  if (group > 256 && groups <= 65535 && !skip && !gate_first && group <= 8192 && (group % 4) == 0 && (n % 4) == 0 && (ldz % 4) == 0 &&
+      (wlen % 4) == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(z) |
+                           reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+    const dim3 grid(rows, groups);
+    const int need = (group / 4 + 255) / 256;
+    if (need <= 2)
+      group_rms_gate_vec_kernel<T, Z, 2><<<grid, 256, 0, s>>>(o, (const Z*)z, ldz, w, wlen, (T*)out, n, group, act, eps);
+    else if (need <= 4)
+      group_rms_gate_vec_kernel<T, Z, 4><<<grid, 256, 0, s>>>(o, (const Z*)z, ldz, w, wlen, (T*)out, n, group, act, eps);
+    else
+      group_rms_gate_vec_kernel<T, Z, 8><<<grid, 256, 0, s>>>(o, (const Z*)z, ldz, w, wlen, (T*)out, n, group, act, eps);
+    return KVCM_LAUNCH_RESULT();
+  }
   if (group > 256 && groups <= 65535) {
     group_rms_gate_wide_kernel<T, Z><<<dim3(rows, groups), 256, 0, s>>>(o, (const Z*)z, ldz, skip, lds, skip_coef, head, w, wlen,
                                                                       (T*)out, n, group, gate_first, act, eps);

@@ -9,9 +9,12 @@
 //     S'  = d^n S + P,   P = sum_j d^(n-1-j) k_j v_j^T
 //
 // so three launches serve every chunk (the batch's tiles of 64 rows) of every request at once:
-//   1. outer : P of every (chunk, head)                                     tensor cores, all chunks side by side
-//   2. carry : per request and element of S, S' along the request's chunks; P's place takes the S a chunk starts with
+//   1. outer : P of every (chunk, head)                                     tensor cores, all chunks side by side;
+//              leaves the activated q, k and v as bfloat16 tiles for the third launch
+//   2. carry : per request and element of S, S' along the request's chunks; leaves the S a chunk starts with, split
 //   3. read  : o of every (chunk, head)                                     tensor cores, all chunks side by side
+// What one launch leaves for the next lies in scratch as whole tiles (key sizes padded to 32, 64 or 128, value sizes to
+// multiples of 64, missing rows and columns zero), so the third launch only copies.
 // No power of the decay is ever divided by: every factor is d^m with m >= 0.
 //
 // Precision: q, k and v (after the optional SiLU) are bfloat16 operands, as the projections of a 16-bit model may be.
@@ -26,43 +29,70 @@ namespace kvcm {
 
 constexpr int kLcRows = 64;                // tokens of a chunk (the batch builder's tile)
 constexpr int kLcCols = 64;                // columns of S per block
-constexpr int kLcThreads = 128;
+constexpr int kLcOuterThreads = 256, kLcReadThreads = 128;
 
 struct LinearChunkParams {
   const float* proj; int ld; int q_base, k_base, v_base;
   const float* decay;                      // [heads]
-  float* carry;                            // [tiles, heads, dk, dv]
+  float* outer;                            // P      [tiles, heads, DK, DVP]
+  bf16* split;                             // S      [tiles, heads, 2 (hi, lo), DK, DVP]
+  bf16* q; bf16* k; bf16* v;               // [tiles, heads, 64, DK] twice, [tiles, heads, 64, DVP]
   float* state; long long state_stride;
   const int* tile_seq; const int* tile_q0; const int* seq_q_start; const int* seq_q_len; const int* seq_state_slot;
   float* out;                              // [rows, heads * dv]
-  int tiles, heads, qk_heads, dk, dv, silu, vec;
+  int tiles, heads, qk_heads, dk, dv, dvp, silu, vec;
 };
 
-__device__ __forceinline__ float lc_act(float z, int silu) { return silu ? z / (1.f + expf(-z)) : z; }
+__device__ __forceinline__ float lc_act(float z) { return z / (1.f + expf(-z)); }
 
 // hi + lo = x up to 2^-17 |x|
-__device__ __forceinline__ void lc_split(float x, bf16& hi, bf16& lo) {
-  hi = __float2bfloat16_rn(x);
-  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
-}
+__device__ __forceinline__ float lc_round(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
 
-// Rows [0, kLcRows) of W neighbouring columns of the projection (activated, zero beyond n rows and `width` columns), each
-// handed to `put(row, column, value)`; 16-byte loads where they are aligned.
+// Rows [0, kLcRows) of W neighbouring columns of the projection (activated, zero beyond n rows and `width` columns), four
+// neighbouring values at a time handed to `put(row, column, values)`; 16-byte loads, eight of a thread in flight
+// together, where they are aligned.
 template <int W, typename Put>
 __device__ __forceinline__ void lc_rows(const float* src, int ld, int n, int width, int silu, int vec, Put put) {
-  if (vec) {
-    for (int i = threadIdx.x; i < kLcRows * (W / 4); i += kLcThreads) {
-      const int r = i / (W / 4), c = (i - r * (W / 4)) * 4;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (r < n && c < width) v = *reinterpret_cast<const float4*>(src + size_t(r) * ld + c);      // (width % 4 == 0)
-      put(r, c, lc_act(v.x, silu)); put(r, c + 1, lc_act(v.y, silu)); put(r, c + 2, lc_act(v.z, silu)); put(r, c + 3, lc_act(v.w, silu));
+  constexpr int kQuads = kLcRows * (W / 4), kTurns = kQuads / kLcOuterThreads, kBatch = kTurns < 8 ? kTurns : 8;
+  static_assert(kQuads % kLcOuterThreads == 0 && kTurns % kBatch == 0, "a thread's turns come in whole batches");
+#pragma unroll 1
+  for (int t = 0; t < kTurns; t += kBatch) {
+    float v[kBatch][4];
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      const int i = threadIdx.x + (t + b) * kLcOuterThreads, r = i / (W / 4), c = (i - r * (W / 4)) * 4;
+      v[b][0] = v[b][1] = v[b][2] = v[b][3] = 0.f;
+      if (r >= n) continue;
+      const float* at = src + size_t(r) * ld + c;
+      if (vec) {
+        if (c < width) {                                       // (width % 4 == 0)
+          const float4 f = *reinterpret_cast<const float4*>(at);
+          v[b][0] = f.x; v[b][1] = f.y; v[b][2] = f.z; v[b][3] = f.w;
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (c + e < width) v[b][e] = at[e];
+      }
     }
-  } else {
-    for (int i = threadIdx.x; i < kLcRows * W; i += kLcThreads) {
-      const int r = i / W, c = i - r * W;
-      put(r, c, r < n && c < width ? lc_act(src[size_t(r) * ld + c], silu) : 0.f);
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      const int i = threadIdx.x + (t + b) * kLcOuterThreads, r = i / (W / 4), c = (i - r * (W / 4)) * 4;
+      if (silu) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[b][e] = lc_act(v[b][e]);
+      }
+      put(r, c, v[b]);
     }
   }
+}
+
+// Four neighbouring bfloat16 values as one 8-byte store (tile rows are an even number of elements wide).
+__device__ __forceinline__ void lc_store4(bf16* dst, float a, float b, float c, float d) {
+  uint2 raw;
+  raw.x = pack_bf16(a, b);
+  raw.y = pack_bf16(c, d);
+  *reinterpret_cast<uint2*>(dst) = raw;
 }
 
 // A fragment (16 x 16) of the transpose of a tile stored [k][m]: the four 8 x 8 matrices transposed as they are loaded.
@@ -71,118 +101,147 @@ __device__ __forceinline__ void lc_frag_trans(uint32_t (&a)[4], const bf16* tile
   ldmatrix_x4_trans(a, tile + ((mi >> 1) * 8 + (lane & 7)) * ldm + (mi & 1) * 8);
 }
 
-template <int DK>
-__global__ void __launch_bounds__(kLcThreads)
+// O (16 x 64) += A (16 x 16) * B (16 x 64), B stored [k][column] at a row stride of ldv.
+__device__ __forceinline__ void lc_pv_64(float (&o)[8][4], const uint32_t (&a)[4], const bf16* tile, int ldv, int lane) {
+  const int row = (lane & 7) + (((lane >> 3) & 1) << 3), col = (lane >> 4) << 3;
+#pragma unroll
+  for (int dd = 0; dd < 4; ++dd) {
+    uint32_t b[4];
+    ldmatrix_x4_trans(b, tile + row * ldv + dd * 16 + col);
+    mma_bf16(o[2 * dd], a, b[0], b[1]);
+    mma_bf16(o[2 * dd + 1], a, b[2], b[3]);
+  }
+}
+
+template <int DK, int DVB>                     // DVB: columns of S a block forms
+__global__ void __launch_bounds__(kLcOuterThreads, 2)
 linear_chunk_outer_kernel(LinearChunkParams p) {
-  constexpr int LDK = DK + 8, LDV = kLcCols + 8;
+  constexpr int LDK = DK + 8, LDV = DVB + 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* khi = reinterpret_cast<bf16*>(smem_raw);             // [64][LDK] d^(n-1-j) k_j
   bf16* klo = khi + kLcRows * LDK;
   bf16* vs = klo + kLcRows * LDK;                             // [64][LDV]
   __shared__ float pw[kLcRows + 1];
   pdl_launch_dependents();
-  const int tile = blockIdx.x, head = blockIdx.y, c0 = blockIdx.z * kLcCols;
+  const int tile = blockIdx.x, head = blockIdx.y, c0 = blockIdx.z * DVB;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile];
   const int row0 = p.seq_q_start[seq] + q0, n = min(kLcRows, p.seq_q_len[seq] - q0);
-  const float d = p.decay[head];
-  if (tid <= kLcRows) pw[tid] = powf(d, float(tid));
+  if (tid <= kLcRows) pw[tid] = powf(p.decay[head], float(tid));
   __syncthreads();
   pdl_wait();
   const float* src = p.proj + size_t(row0) * p.ld;
-  lc_rows<DK>(src + p.k_base + (head / (p.heads / p.qk_heads)) * p.dk, p.ld, n, p.dk, p.silu, p.vec, [&](int r, int c, float x) {
+  const int qk = (head / (p.heads / p.qk_heads)) * p.dk;
+  const size_t th = size_t(tile) * p.heads + head;
+  const bool first = blockIdx.z == 0;                         // leaves q and k too
+  bf16* qg = p.q + th * kLcRows * DK;
+  bf16* kg = p.k + th * kLcRows * DK;
+  bf16* vg = p.v + th * kLcRows * p.dvp + c0;
+  lc_rows<DK>(src + p.k_base + qk, p.ld, n, p.dk, p.silu, p.vec, [&](int r, int c, const float (&x)[4]) {
     // the key as a bfloat16 operand, then times its power of the decay in two parts
-    lc_split(__bfloat162float(__float2bfloat16_rn(x)) * (r < n ? pw[n - 1 - r] : 0.f), khi[r * LDK + c], klo[r * LDK + c]);
-  });
-  lc_rows<kLcCols>(src + p.v_base + head * p.dv + c0, p.ld, n, p.dv - c0, p.silu, p.vec,
-                   [&](int r, int c, float x) { vs[r * LDV + c] = __float2bfloat16_rn(x); });
-  __syncthreads();
-  float* dst = p.carry + (size_t(tile) * p.heads + head) * p.dk * p.dv;
-  const int g = lane >> 2, t4 = lane & 3;
-  for (int mt = warp; mt < DK / 16; mt += kLcThreads / 32) {
-    if (mt * 16 >= p.dk) break;
-    float o[kLcCols / 8][4];
+    const float f = r < n ? pw[n - 1 - r] : 0.f;
+    float y[4], hi[4];
 #pragma unroll
-    for (int i = 0; i < kLcCols / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int e = 0; e < 4; ++e) {
+      y[e] = lc_round(x[e]) * f;
+      hi[e] = lc_round(y[e]);
+    }
+    lc_store4(khi + r * LDK + c, hi[0], hi[1], hi[2], hi[3]);
+    lc_store4(klo + r * LDK + c, y[0] - hi[0], y[1] - hi[1], y[2] - hi[2], y[3] - hi[3]);
+    if (first) lc_store4(kg + r * DK + c, x[0], x[1], x[2], x[3]);
+  });
+  lc_rows<DVB>(src + p.v_base + head * p.dv + c0, p.ld, n, p.dv - c0, p.silu, p.vec, [&](int r, int c, const float (&x)[4]) {
+    lc_store4(vs + r * LDV + c, x[0], x[1], x[2], x[3]);
+    lc_store4(vg + r * p.dvp + c, x[0], x[1], x[2], x[3]);
+  });
+  if (first)
+    lc_rows<DK>(src + p.q_base + qk, p.ld, n, p.dk, p.silu, p.vec,
+                [&](int r, int c, const float (&x)[4]) { lc_store4(qg + r * DK + c, x[0], x[1], x[2], x[3]); });
+  __syncthreads();
+  float* dst = p.outer + th * DK * p.dvp + c0;
+  const int g = lane >> 2, t4 = lane & 3;
+  for (int task = warp; task < (DK / 16) * (DVB / 64); task += kLcOuterThreads / 32) {       // 16 rows x 64 columns of P
+    const int mt = task % (DK / 16), nb = task / (DK / 16) * 64;
+    float o[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
 #pragma unroll
     for (int kk = 0; kk < kLcRows / 16; ++kk) {
-      uint32_t a[4];
+      uint32_t a[4], b[4];
       lc_frag_trans(a, khi + kk * 16 * LDK + mt * 16, LDK, lane);
-      pv_16x16<kLcCols>(o, a, vs + kk * 16 * LDV, lane);
-      lc_frag_trans(a, klo + kk * 16 * LDK + mt * 16, LDK, lane);
-      pv_16x16<kLcCols>(o, a, vs + kk * 16 * LDV, lane);
+      lc_frag_trans(b, klo + kk * 16 * LDK + mt * 16, LDK, lane);
+      lc_pv_64(o, a, vs + kk * 16 * LDV + nb, LDV, lane);
+      lc_pv_64(o, b, vs + kk * 16 * LDV + nb, LDV, lane);
     }
 #pragma unroll
-    for (int i = 0; i < kLcCols / 8; ++i)
+    for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int r = mt * 16 + g + 8 * h, c = c0 + 8 * i + 2 * t4;
-        if (r >= p.dk) continue;
-        float* at = dst + size_t(r) * p.dv + c;
-        if ((p.dv & 1) == 0) {
-          if (c < p.dv) *reinterpret_cast<float2*>(at) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
-        } else {
-          if (c < p.dv) at[0] = o[i][2 * h];
-          if (c + 1 < p.dv) at[1] = o[i][2 * h + 1];
-        }
-      }
+      for (int h = 0; h < 2; ++h)
+        *reinterpret_cast<float2*>(dst + size_t(mt * 16 + g + 8 * h) * p.dvp + nb + 8 * i + 2 * t4) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
   }
 }
 
-// One thread carries V neighbouring elements of one request's S along its chunks.
-template <int V>
+// One thread carries four neighbouring elements of one request's (padded) S along its chunks.
 __global__ void __launch_bounds__(256)
-linear_chunk_carry_kernel(LinearChunkParams p) {
+linear_chunk_carry_kernel(LinearChunkParams p, int DK) {
   pdl_launch_dependents();
   const int tile0 = blockIdx.y;
   if (p.tile_q0[tile0] != 0) return;                          // a request's chunks belong to the block row of its first
   const int seq = p.tile_seq[tile0], len = p.seq_q_len[seq], slot = p.seq_state_slot[seq];
-  const int per = p.dk * p.dv, total = p.heads * per;
-  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  const int per = DK * p.dvp, total = p.heads * per;          // (dvp is a multiple of 64)
+  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (i >= total) return;
-  const float d = p.decay[i / per];                           // (V divides a head's elements)
+  const int head = i / per, in = i - head * per, r = in / p.dvp, c = in - r * p.dvp;
+  const float d = p.decay[head];
   const float whole = powf(d, float(kLcRows));
-  pdl_wait();
-  float S[V];
-  float* st = slot >= 0 ? p.state + slot * p.state_stride + i : nullptr;
-#pragma unroll
-  for (int e = 0; e < V; ++e) S[e] = st ? st[e] : 0.f;
-  float* at = p.carry + size_t(tile0) * total + i;
   const int n_tiles = (len + kLcRows - 1) / kLcRows;
+  const float last = powf(d, float(len - (n_tiles - 1) * kLcRows));
+  const int live = r < p.dk ? min(4, p.dv - c) : 0;           // elements that the state holds
+  float* st = slot >= 0 ? p.state + slot * p.state_stride + (size_t(head) * p.dk + r) * p.dv + c : nullptr;
+  pdl_wait();
+  float S[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int e = 0; e < 4; ++e)
+    if (st && e < live) S[e] = st[e];
+  const float* src = p.outer + size_t(tile0) * total + i;
+  bf16* dst = p.split + 2 * (size_t(tile0) * total + size_t(head) * per) + in;
   constexpr int AHEAD = 8;                                    // chunks whose P is asked for together
   for (int t0 = 0; t0 < n_tiles; t0 += AHEAD) {
-    float P[AHEAD][V];
+    float4 P[AHEAD];
 #pragma unroll
-    for (int j = 0; j < AHEAD; ++j) {
-      if (t0 + j >= n_tiles) break;
-      const float* src = at + size_t(t0 + j) * total;
-      if constexpr (V == 4) {
-        const float4 v = *reinterpret_cast<const float4*>(src);
-        P[j][0] = v.x; P[j][1] = v.y; P[j][2] = v.z; P[j][3] = v.w;
-      } else {
-        P[j][0] = src[0];
-      }
-    }
+    for (int j = 0; j < AHEAD; ++j)
+      if (t0 + j < n_tiles) P[j] = *reinterpret_cast<const float4*>(src + size_t(t0 + j) * total);
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j) {
       const int t = t0 + j;
       if (t >= n_tiles) break;
-      float* dst = at + size_t(t) * total;
-      if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(S[0], S[1], S[2], S[3]);
-      else dst[0] = S[0];
-      const float f = t + 1 < n_tiles ? whole : powf(d, float(len - t * kLcRows));
+      float hi[4];
 #pragma unroll
-      for (int e = 0; e < V; ++e) S[e] = fmaf(f, S[e], P[j][e]);
+      for (int e = 0; e < 4; ++e) hi[e] = lc_round(S[e]);
+      bf16* at = dst + 2 * size_t(t) * total;
+      lc_store4(at, hi[0], hi[1], hi[2], hi[3]);
+      lc_store4(at + per, S[0] - hi[0], S[1] - hi[1], S[2] - hi[2], S[3] - hi[3]);
+      const float f = t + 1 < n_tiles ? whole : last;
+      S[0] = fmaf(f, S[0], P[j].x); S[1] = fmaf(f, S[1], P[j].y); S[2] = fmaf(f, S[2], P[j].z); S[3] = fmaf(f, S[3], P[j].w);
     }
   }
-  if (st) {
 #pragma unroll
-    for (int e = 0; e < V; ++e) st[e] = S[e];
+  for (int e = 0; e < 4; ++e)
+    if (st && e < live) st[e] = S[e];
+}
+
+// Copies a [rows][W] bfloat16 tile (row stride lds elements in memory) to shared memory rows of W + 8 elements.
+template <int W>
+__device__ __forceinline__ void lc_copy_tile(bf16* dst, const bf16* src, int rows, int lds) {
+  constexpr int CH = W / 8;
+  for (int i = threadIdx.x; i < rows * CH; i += kLcReadThreads) {
+    const int r = i / CH, c = (i - r * CH) * 8;
+    cp_async16(dst + r * (W + 8) + c, src + size_t(r) * lds + c);
   }
 }
 
 template <int DK>
-__global__ void __launch_bounds__(kLcThreads)
+__global__ void __launch_bounds__(kLcReadThreads)
 linear_chunk_read_kernel(LinearChunkParams p) {
   constexpr int LDK = DK + 8, LDV = kLcCols + 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -199,34 +258,17 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   const int row0 = p.seq_q_start[seq] + q0, n = min(kLcRows, p.seq_q_len[seq] - q0);
   if (tid <= kLcRows) pw[tid] = powf(p.decay[head], float(tid));
   pdl_wait();
-  const float* src = p.proj + size_t(row0) * p.ld;
-  const int qk = (head / (p.heads / p.qk_heads)) * p.dk;
-  lc_rows<DK>(src + p.q_base + qk, p.ld, n, p.dk, p.silu, p.vec, [&](int r, int c, float x) { qs[r * LDK + c] = __float2bfloat16_rn(x); });
-  lc_rows<DK>(src + p.k_base + qk, p.ld, n, p.dk, p.silu, p.vec, [&](int r, int c, float x) { ks[r * LDK + c] = __float2bfloat16_rn(x); });
-  lc_rows<kLcCols>(src + p.v_base + head * p.dv + c0, p.ld, n, p.dv - c0, p.silu, p.vec,
-                   [&](int r, int c, float x) { vs[r * LDV + c] = __float2bfloat16_rn(x); });
-  const float* S = p.carry + (size_t(tile) * p.heads + head) * p.dk * p.dv + c0;
-  const bool svec = p.vec != 0;                               // (dv % 4 == 0)
-  for (int i = tid; i < DK * (kLcCols / 4); i += kLcThreads) {
-    const int r = i / (kLcCols / 4), c = (i - r * (kLcCols / 4)) * 4;
-    float v[4] = {0.f, 0.f, 0.f, 0.f};
-    if (r < p.dk) {
-      if (svec) {
-        if (c0 + c < p.dv) {
-          const float4 a = *reinterpret_cast<const float4*>(S + size_t(r) * p.dv + c);
-          v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-        }
-      } else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (c0 + c + e < p.dv) v[e] = S[size_t(r) * p.dv + c + e];
-      }
-    }
-#pragma unroll
-    for (int e = 0; e < 4; ++e) lc_split(v[e], shi[r * LDV + c + e], slo[r * LDV + c + e]);
-  }
+  const size_t th = size_t(tile) * p.heads + head;
+  const bf16* S = p.split + 2 * th * DK * p.dvp + c0;
+  lc_copy_tile<DK>(qs, p.q + th * kLcRows * DK, kLcRows, DK);
+  lc_copy_tile<kLcCols>(shi, S, DK, p.dvp);
+  lc_copy_tile<kLcCols>(slo, S + size_t(DK) * p.dvp, DK, p.dvp);
+  cp_async_commit();
+  lc_copy_tile<DK>(ks, p.k + th * kLcRows * DK, kLcRows, DK);
+  lc_copy_tile<kLcCols>(vs, p.v + th * kLcRows * p.dvp + c0, kLcRows, p.dvp);
+  cp_async_commit();
+  cp_async_wait<1>();
   __syncthreads();
-  if (warp * 16 >= n) return;
   const int g = lane >> 2, t4 = lane & 3;
   uint32_t qa[DK / 16][4];
   load_q_frags<DK>(qa, qs + warp * 16 * LDK, lane);
@@ -238,6 +280,9 @@ linear_chunk_read_kernel(LinearChunkParams p) {
     pv_16x16<kLcCols>(o, qa[kk], shi + kk * 16 * LDV, lane);
     pv_16x16<kLcCols>(o, qa[kk], slo + kk * 16 * LDV, lane);
   }
+  cp_async_wait<0>();
+  __syncthreads();                                             // every thread's share of k and v is there
+  if (warp * 16 >= n) return;
   const int row[2] = {warp * 16 + g, warp * 16 + g + 8};      // this thread's rows of the chunk
 #pragma unroll
   for (int i = 0; i < kLcCols / 8; ++i)
@@ -253,7 +298,7 @@ linear_chunk_read_kernel(LinearChunkParams p) {
       for (int j = 0; j < 4; ++j) {
         const int dist = row[j >> 1] - (kb * 16 + 8 * h + 2 * t4 + (j & 1));
         const float x = dist >= 0 ? s[h][j] * pw[dist] : 0.f;
-        const float hi = __bfloat162float(__float2bfloat16_rn(x));
+        const float hi = lc_round(x);
         s[h][j] = hi;
         lo[h][j] = x - hi;
       }
@@ -279,28 +324,49 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   }
 }
 
-template <int DK>
-static int launch_linear_chunk(const LinearChunkParams& p, cudaStream_t s) {
-  constexpr int LDK = DK + 8, LDV = kLcCols + 8;
-  constexpr size_t smem_outer = size_t(2 * kLcRows * LDK + kLcRows * LDV) * sizeof(bf16);
-  constexpr size_t smem_read = size_t(2 * kLcRows * LDK + kLcRows * LDV + 2 * DK * LDV) * sizeof(bf16);
+// Scratch of a launch, in bytes from a 16-byte aligned start: P, then S split, q, k, v (every part a multiple of 16).
+struct LinearChunkScratch { long long outer, split, q, k, v, total; };
+static LinearChunkScratch linear_chunk_scratch(int tiles, int heads, int DK, int dvp) {
+  const long long th = (long long)tiles * heads;
+  LinearChunkScratch s;
+  s.outer = 0;
+  s.split = s.outer + th * DK * dvp * 4;
+  s.q = s.split + th * DK * dvp * 4;
+  s.k = s.q + th * kLcRows * DK * 2;
+  s.v = s.k + th * kLcRows * DK * 2;
+  s.total = s.v + th * kLcRows * dvp * 2;
+  return s;
+}
+static int linear_chunk_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : 128; }
+static int linear_chunk_dvp(int dv) { return (dv + 63) / 64 * 64; }
+
+template <int DK, int DVB>
+static int launch_linear_outer(const LinearChunkParams& p, cudaStream_t s) {
+  constexpr size_t smem = size_t(2 * kLcRows * (DK + 8) + kLcRows * (DVB + 8)) * sizeof(bf16);
   static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(linear_chunk_outer_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_outer));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_chunk_read_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_read));
+  if (!configured && smem > 40 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(linear_chunk_outer_kernel<DK, DVB>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     if (e != cudaSuccess) return int(e);
     configured = true;
   }
-  const dim3 grid(p.tiles, p.heads, (p.dv + kLcCols - 1) / kLcCols);
-  int rc = pdl_launch(linear_chunk_outer_kernel<DK>, grid, dim3(kLcThreads), smem_outer, s, p);
+  return pdl_launch(linear_chunk_outer_kernel<DK, DVB>, dim3(p.tiles, p.heads, p.dvp / DVB), dim3(kLcOuterThreads), smem, s, p);
+}
+
+template <int DK>
+static int launch_linear_chunk(const LinearChunkParams& p, cudaStream_t s) {
+  constexpr size_t smem = size_t(2 * kLcRows * (DK + 8) + kLcRows * (kLcCols + 8) + 2 * DK * (kLcCols + 8)) * sizeof(bf16);
+  static bool configured = false;
+  if (!configured && smem > 40 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(linear_chunk_read_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    if (e != cudaSuccess) return int(e);
+    configured = true;
+  }
+  int rc = (p.dvp % 128) == 0 ? launch_linear_outer<DK, 128>(p, s) : launch_linear_outer<DK, 64>(p, s);
   if (rc) return rc;
-  const long long total = (long long)p.heads * p.dk * p.dv;
-  if (((p.dk * p.dv) % 4) == 0 && (reinterpret_cast<uintptr_t>(p.carry) & 15) == 0)
-    rc = pdl_launch(linear_chunk_carry_kernel<4>, dim3(unsigned((total / 4 + 255) / 256), p.tiles), dim3(256), 0, s, p);
-  else
-    rc = pdl_launch(linear_chunk_carry_kernel<1>, dim3(unsigned((total + 255) / 256), p.tiles), dim3(256), 0, s, p);
+  const long long quads = (long long)p.heads * DK * p.dvp / 4;
+  rc = pdl_launch(linear_chunk_carry_kernel, dim3(unsigned((quads + 255) / 256), p.tiles), dim3(256), 0, s, p, DK);
   if (rc) return rc;
-  return pdl_launch(linear_chunk_read_kernel<DK>, grid, dim3(kLcThreads), smem_read, s, p);
+  return pdl_launch(linear_chunk_read_kernel<DK>, dim3(p.tiles, p.heads, p.dvp / kLcCols), dim3(kLcReadThreads), smem, s, p);
 }
 
 }  // namespace kvcm
@@ -310,22 +376,33 @@ using namespace kvcm;
 // Largest key size of the chunked form.
 KVCM_API int kvcm_linear_chunk_max_dk(void) { return 128; }
 
+// Bytes of scratch for a step of `tiles` chunks.
+KVCM_API long long kvcm_linear_chunk_scratch_bytes(int tiles, int heads, int dk, int dv) {
+  return linear_chunk_scratch(tiles, heads, linear_chunk_dk(dk), linear_chunk_dvp(dv)).total;
+}
+
 // Runs the recurrence over the rows of every portion of more than one token (the step's tiles of 64 rows); single-row
-// entries are not touched.  proj: float rows of `ld` elements with q, k, v at the given bases; decay [heads]; carry: float
-// scratch [tiles, heads, dk, dv]; out: float [rows, heads * dv].
-KVCM_API int kvcm_linear_chunk(const float* proj, int ld, int q_base, int k_base, int v_base, const float* decay, float* carry,
+// entries are not touched.  proj: float rows of `ld` elements with q, k, v at the given bases; decay [heads]; scratch:
+// kvcm_linear_chunk_scratch_bytes(), 16-byte aligned; out: float [rows, heads * dv].
+KVCM_API int kvcm_linear_chunk(const float* proj, int ld, int q_base, int k_base, int v_base, const float* decay, void* scratch,
                                float* state, long long state_stride, const int* tile_seq, const int* tile_q0,
                                const int* seq_q_start, const int* seq_q_len, const int* seq_state_slot, float* out, int tiles,
                                int heads, int qk_heads, int dk, int dv, int silu, void* stream) {
   if (tiles == 0) return 0;
-  if (dk < 1 || dk > 128 || dv < 1 || qk_heads < 1 || heads % qk_heads || tiles > 65535) return KVCM_ERR_UNSUPPORTED;
+  if (dk < 1 || dk > 128 || dv < 1 || qk_heads < 1 || heads % qk_heads || tiles > 65535 || heads > 65535 ||
+      (reinterpret_cast<uintptr_t>(scratch) & 15))
+    return KVCM_ERR_UNSUPPORTED;
   LinearChunkParams p;
-  p.proj = proj; p.ld = ld; p.q_base = q_base; p.k_base = k_base; p.v_base = v_base; p.decay = decay; p.carry = carry;
+  p.proj = proj; p.ld = ld; p.q_base = q_base; p.k_base = k_base; p.v_base = v_base; p.decay = decay;
   p.state = state; p.state_stride = state_stride; p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.seq_q_start = seq_q_start;
   p.seq_q_len = seq_q_len; p.seq_state_slot = seq_state_slot; p.out = out; p.tiles = tiles; p.heads = heads;
-  p.qk_heads = qk_heads; p.dk = dk; p.dv = dv; p.silu = silu;
+  p.qk_heads = qk_heads; p.dk = dk; p.dv = dv; p.dvp = linear_chunk_dvp(dv); p.silu = silu;
+  const LinearChunkScratch at = linear_chunk_scratch(tiles, heads, linear_chunk_dk(dk), p.dvp);
+  char* base = static_cast<char*>(scratch);
+  p.outer = reinterpret_cast<float*>(base + at.outer); p.split = reinterpret_cast<bf16*>(base + at.split);
+  p.q = reinterpret_cast<bf16*>(base + at.q); p.k = reinterpret_cast<bf16*>(base + at.k); p.v = reinterpret_cast<bf16*>(base + at.v);
   p.vec = (dk % 4) == 0 && (dv % 4) == 0 && (ld % 4) == 0 && (q_base % 4) == 0 && (k_base % 4) == 0 && (v_base % 4) == 0 &&
-          ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(carry)) & 15) == 0;
+          (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
   cudaStream_t s = (cudaStream_t)stream;
   if (dk <= 32) return launch_linear_chunk<32>(p, s);
   if (dk <= 64) return launch_linear_chunk<64>(p, s);

@@ -1,7 +1,7 @@
 // A feed-forward made of many small gated experts of which every row uses a few.
 //
-//   route    router logits in float (one warp a row), softmax over all experts, optionally only the
-//            experts of the best `keep` of `groups` equal groups of neighbours may be chosen (a
+//   route    router logits in float (bfloat16 rows and router: products on the tensor cores, float sums),
+//            softmax over all experts, optionally only the experts of the best `keep` of `groups` equal groups of neighbours may be chosen (a
 //            group's score is its largest expert score), the `top` largest scores win; a row's
 //            weights are its chosen scores times `scale`, not renormalised.  An extra row of the
 //            router matrix, if present, is a per-row gate: sigmoid of its logit.  Options: scores
@@ -39,6 +39,12 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
+// Unsigned integers in the order of the floats (larger float, larger key; every key is above zero).
+__device__ __forceinline__ unsigned route_key(float v) {
+  const unsigned u = __float_as_uint(v);
+  return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+}
+
 // ------------------------------------------------------------------------------------ route
 // One block of eight warps for RB rows: the rows of h are staged in shared memory as floats, the
 // warps share out the experts (each logit one warp's sum over the width, float FMAs, 16-byte loads
@@ -63,14 +69,123 @@ __device__ __forceinline__ void route_load(const bf16* p, float (&v)[8]) {
   for (int i = 0; i < 4; ++i) { v[2 * i] = __bfloat162float(h2[i].x); v[2 * i + 1] = __bfloat162float(h2[i].y); }
 }
 
+// One warp's choice for one row.  `z`: the row's E logits (and the gate's behind them) in shared memory, then room for the
+// groups' scores and the choice scores.
+struct RouteChoice {
+  int E, G, keep, top, has_gate, sigmoid_scores, group_top, renorm;
+  float scale;
+  const float* correction;
+  int* idx; float* wt; float* gate_out;
+};
+__device__ __forceinline__ void route_choose(const RouteChoice& c, float* z, int row, int lane) {
+  const int E = c.E, G = c.G, keep = c.keep, top = c.top, has_gate = c.has_gate, sigmoid_scores = c.sigmoid_scores,
+            group_top = c.group_top, renorm = c.renorm;
+  const float scale = c.scale;
+  const float* correction = c.correction;
+  int* idx = c.idx;
+  float* wt = c.wt;
+  float* gate_out = c.gate_out;
+  float* gb = z + E + 1;
+  float* ch = gb + G;                                        // choice scores: -inf once taken
+  if (sigmoid_scores) {
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) {
+      ch[e] = z[e];                                          // (the sigmoid keeps the order; in float it makes large logits equal)
+      z[e] = 1.f / (1.f + expf(-z[e]));
+    }
+  } else {
+    float m = -INFINITY;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - m);
+    sum = warp_sum(sum);
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) z[e] = expf(z[e] - m) / sum;
+  }
+  const bool limited = G > 1 && keep < G;
+  if (!sigmoid_scores || correction || limited)
+    for (int e = lane; e < E; e += 32) ch[e] = z[e] + (correction ? correction[e] : 0.f);
+  if (has_gate && lane == 0) gate_out[row] = 1.f / (1.f + expf(-z[E]));
+  __syncwarp();
+  const int per = E / G;
+  if (limited) {
+    for (int g = lane; g < G; g += 32) {
+      float best = -INFINITY, second = -INFINITY;            // the group's two largest choice scores
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float cs = ch[e];
+        if (cs > best) { second = best; best = cs; }
+        else if (cs > second) second = cs;
+      }
+      gb[g] = (group_top >= 2 && per >= 2) ? best + second : best;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+      float bv = -INFINITY;
+      int bi = 0x7fffffff;
+      for (int g = lane; g < G; g += 32) {
+        const float cs = gb[g];
+        if (cs != INFINITY && (bi == 0x7fffffff || cs > bv)) { bv = cs; bi = g; }
+      }
+      warp_argmax(bv, bi);
+      __syncwarp();
+      if (lane == 0 && bi < G) gb[bi] = INFINITY;           // kept
+      __syncwarp();
+    }
+  }
+  // Every lane keeps the best of its own experts at hand; a choice is one maximum over the warp (and the lowest index
+  // among equals), after which only the lane that owned it looks through its experts again.
+  auto best_of_mine = [&](float& bv, int& bi) {
+    bv = -INFINITY;
+    bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const bool allowed = !limited || gb[e / per] == INFINITY;
+      const float cs = ch[e];
+      if (allowed && cs != -INFINITY && (bi == 0x7fffffff || cs > bv)) { bv = cs; bi = e; }
+    }
+  };
+  float bv;
+  int bi;
+  best_of_mine(bv, bi);
+  float chosen = 0.f, mine = 0.f;                            // sum of the chosen scores, in the order of choice
+  int my_expert = 0;                                         // lane k % 32 keeps choice k until it is stored
+  for (int k = 0; k < top; ++k) {
+    const unsigned key = route_key(bv);
+    const unsigned most = __reduce_max_sync(0xffffffffu, bi < E ? key : 0u);
+    const int win = int(__reduce_min_sync(0xffffffffu, bi < E && key == most ? unsigned(bi) : 0x7fffffffu));
+    const bool ok = win < E;
+    const float score = ok ? z[win] : 0.f;
+    chosen += score;
+    if (lane == (k & 31)) { mine = score; my_expert = ok ? win : 0; }
+    if (bi == win && ok) {                                   // this lane's: taken
+      ch[win] = -INFINITY;
+      best_of_mine(bv, bi);
+    }
+    if ((k & 31) == 31 || k + 1 == top) {                    // a batch of up to 32 choices
+      const int at = (k & ~31) + lane;
+      if (at <= k) {
+        idx[size_t(row) * top + at] = my_expert;
+        wt[size_t(row) * top + at] = mine * scale;
+      }
+    }
+  }
+  if (renorm) {
+    if (top <= 32) {
+      if (lane < top) wt[size_t(row) * top + lane] = mine / (chosen + 1e-20f) * scale;
+    } else {
+      __syncwarp();
+      for (int k = lane; k < top; k += 32) wt[size_t(row) * top + k] /= chosen + 1e-20f;
+    }
+  }
+}
+
 template <typename T, typename W, int RB>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int rows, int D, int E, int G, int keep,
-                 int top, float scale, int has_gate, int vec_ok, int sigmoid_scores, const float* __restrict__ correction,
-                 int group_top, int renorm, int* __restrict__ idx, float* __restrict__ wt, float* __restrict__ gate_out) {
+moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int rows, int D, int vec_ok, RouteChoice choice) {
   extern __shared__ float route_smem[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row0 = blockIdx.x * RB;
+  const int E = choice.E, G = choice.G, has_gate = choice.has_gate;
   const int zstride = (2 * E + 1 + G + 3) & ~3;             // per row: scores, the gate's logit, the groups' scores, choice scores
   float* hs = route_smem + RB * zstride;                    // RB rows of h (16-byte aligned)
   for (int rr = 0; rr < RB; ++rr) {
@@ -133,77 +248,77 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const W* __restrict__ wr, int
   for (int rr = warp; rr < RB; rr += ROUTE_WARPS) {
     const int row = row0 + rr;
     if (row >= rows) break;
-    float* z = route_smem + rr * zstride;
-    float* gb = z + E + 1;
-    float* ch = gb + G;                                        // choice scores: -inf once taken
-    if (sigmoid_scores) {
-      __syncwarp();
-      for (int e = lane; e < E; e += 32) {
-        ch[e] = z[e];                                          // (the sigmoid keeps the order; in float it makes large logits equal)
-        z[e] = 1.f / (1.f + expf(-z[e]));
+    route_choose(choice, route_smem + rr * zstride, row, lane);
+  }
+}
+
+// bfloat16 rows and router on the tensor cores: sixteen rows a block, the width split over its eight warps (blocks of 32
+// columns; a thread's 16 bytes of a row and of a router row are the same columns, so two products take them in any
+// order of columns), float sums, added over the warps in warp order.  The products of two bfloat16 numbers are exact in
+// float: the logits are float sums as above.
+constexpr int ROUTE_MMA_ROWS = 16;
+
+__device__ __forceinline__ void route_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int NT>                                           // 8 * NT experts at a time
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+moe_route_mma_kernel(const bf16* __restrict__ h, int ldh, const bf16* __restrict__ wr, int rows, int D, RouteChoice choice) {
+  constexpr int NP = 8 * NT;
+  extern __shared__ float route_smem[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t4 = lane & 3;
+  const int row0 = blockIdx.x * ROUTE_MMA_ROWS;
+  const int E = choice.E, outs = E + (choice.has_gate ? 1 : 0);
+  const int zstride = (2 * E + 1 + choice.G + 3) & ~3;
+  float* part = route_smem + ROUTE_MMA_ROWS * zstride;      // [warps][16][NP]
+  // (rows and experts beyond the last read the last: their sums are never used)
+  const bf16* ra = h + size_t(min(row0 + g, rows - 1)) * ldh + t4 * 8;
+  const bf16* rb = h + size_t(min(row0 + g + 8, rows - 1)) * ldh + t4 * 8;
+  for (int n0 = 0; n0 < outs; n0 += NP) {
+    float acc[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    const bf16* we[NT];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) we[i] = wr + size_t(min(n0 + 8 * i + g, outs - 1)) * D + t4 * 8;
+    auto step = [&](int kb, bool in) {                      // `in`: this thread's eight columns lie within the row (D % 8 == 0)
+      const uint4 none = make_uint4(0u, 0u, 0u, 0u);
+      const uint4 a = in ? *reinterpret_cast<const uint4*>(ra + kb) : none, b = in ? *reinterpret_cast<const uint4*>(rb + kb) : none;
+      uint4 w[NT];
+#pragma unroll
+      for (int i = 0; i < NT; ++i) w[i] = in ? *reinterpret_cast<const uint4*>(we[i] + kb) : none;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        route_mma(acc[i], a.x, b.x, a.y, b.y, w[i].x, w[i].y);
+        route_mma(acc[i], a.z, b.z, a.w, b.w, w[i].z, w[i].w);
       }
-    } else {
-      float m = -INFINITY;
-      for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
-      m = warp_max(m);
-      float sum = 0.f;
-      for (int e = lane; e < E; e += 32) sum += expf(z[e] - m);
-      sum = warp_sum(sum);
-      __syncwarp();
-      for (int e = lane; e < E; e += 32) z[e] = expf(z[e] - m) / sum;
+    };
+    const int whole = D & ~31;
+#pragma unroll (NT == 4 ? 4 : 2)
+    for (int kb = warp * 32; kb < whole; kb += ROUTE_WARPS * 32) step(kb, true);
+    if (whole < D && ((whole >> 5) % ROUTE_WARPS) == warp) step(whole, whole + t4 * 8 < D);
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      float* at = part + (warp * ROUTE_MMA_ROWS + g) * NP + 8 * i + 2 * t4;
+      at[0] = acc[i][0]; at[1] = acc[i][1];
+      at[8 * NP] = acc[i][2]; at[8 * NP + 1] = acc[i][3];
     }
-    const bool limited = G > 1 && keep < G;
-    if (!sigmoid_scores || correction || limited)
-      for (int e = lane; e < E; e += 32) ch[e] = z[e] + (correction ? correction[e] : 0.f);
-    if (has_gate && lane == 0) gate_out[row] = 1.f / (1.f + expf(-z[E]));
-    __syncwarp();
-    const int per = E / G;
-    if (limited) {
-      for (int g = lane; g < G; g += 32) {
-        float best = -INFINITY, second = -INFINITY;            // the group's two largest choice scores
-        for (int e = g * per; e < (g + 1) * per; ++e) {
-          const float c = ch[e];
-          if (c > best) { second = best; best = c; }
-          else if (c > second) second = c;
-        }
-        gb[g] = (group_top >= 2 && per >= 2) ? best + second : best;
-      }
-      __syncwarp();
-      for (int k = 0; k < keep; ++k) {
-        float bv = -INFINITY;
-        int bi = 0x7fffffff;
-        for (int g = lane; g < G; g += 32) {
-          const float c = gb[g];
-          if (c != INFINITY && (bi == 0x7fffffff || c > bv)) { bv = c; bi = g; }
-        }
-        warp_argmax(bv, bi);
-        __syncwarp();
-        if (lane == 0 && bi < G) gb[bi] = INFINITY;           // kept
-        __syncwarp();
-      }
+    __syncthreads();
+    for (int i = threadIdx.x; i < ROUTE_MMA_ROWS * NP; i += ROUTE_WARPS * 32) {
+      const int r = i / NP, e = n0 + i % NP;
+      if (e >= outs) continue;
+      float z = 0.f;
+#pragma unroll
+      for (int w = 0; w < ROUTE_WARPS; ++w) z += part[w * ROUTE_MMA_ROWS * NP + i];
+      route_smem[r * zstride + e] = z;
     }
-    float chosen = 0.f;                                        // sum of the chosen scores, in the order of choice
-    for (int k = 0; k < top; ++k) {
-      float bv = -INFINITY;
-      int bi = 0x7fffffff;
-      for (int e = lane; e < E; e += 32) {
-        const bool allowed = !limited || gb[e / per] == INFINITY;
-        const float c = ch[e];
-        if (allowed && c != -INFINITY && (bi == 0x7fffffff || c > bv)) { bv = c; bi = e; }
-      }
-      warp_argmax(bv, bi);
-      __syncwarp();
-      if (bi < E) chosen += z[bi];
-      if (lane == 0) {
-        const bool ok = bi < E;
-        idx[size_t(row) * top + k] = ok ? bi : 0;
-        wt[size_t(row) * top + k] = ok ? z[bi] * scale : 0.f;
-        if (ok) ch[bi] = -INFINITY;                            // taken
-      }
-      __syncwarp();
-    }
-    if (renorm && lane == 0)
-      for (int k = 0; k < top; ++k) wt[size_t(row) * top + k] = wt[size_t(row) * top + k] / (chosen + 1e-20f);
+    __syncthreads();
+  }
+  for (int rr = warp; rr < ROUTE_MMA_ROWS; rr += ROUTE_WARPS) {
+    const int row = row0 + rr;
+    if (row < rows) route_choose(choice, route_smem + rr * zstride, row, lane);
   }
 }
 
@@ -392,6 +507,19 @@ int launch_moe_route(const void* h, int ldh, const void* wr, int w_f32, int rows
   while (rb > 1 && (rb * (zstride + D)) * sizeof(float) > 160 * 1024) rb /= 2;
   const size_t smem = rb * (zstride + D) * sizeof(float);
   if (smem > 200 * 1024) return KVCM_ERR_UNSUPPORTED;
+  const RouteChoice choice = {E, G, keep, top, has_gate, sigmoid_scores, group_top, renorm, scale, correction, idx, wt, gate_out};
+  if constexpr (sizeof(T) == 2) {
+    const int outs = E + (has_gate ? 1 : 0), np = outs <= 32 ? 32 : 64;
+    const size_t mma_smem = ROUTE_MMA_ROWS * (zstride + ROUTE_WARPS * np) * sizeof(float);
+    if (!w_f32 && (D % 8) == 0 && (ldh % 8) == 0 && ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(wr)) & 15) == 0 &&
+        mma_smem <= 200 * 1024) {
+      const dim3 grid((rows + ROUTE_MMA_ROWS - 1) / ROUTE_MMA_ROWS);
+      auto kernel = np == 32 ? moe_route_mma_kernel<4> : moe_route_mma_kernel<8>;
+      if (mma_smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mma_smem);
+      kernel<<<grid, ROUTE_WARPS * 32, mma_smem, s>>>((const bf16*)h, ldh, (const bf16*)wr, rows, D, choice);
+      return KVCM_LAUNCH_RESULT();
+    }
+  }
   const int vec = w_f32 ? 4 : RouteVec<T>::N;
   const int vec_ok = (D % vec) == 0 && (reinterpret_cast<uintptr_t>(wr) & 15) == 0;
 #define KVCM_ROUTE(W, RB)                                                                                             \
@@ -399,8 +527,7 @@ int launch_moe_route(const void* h, int ldh, const void* wr, int w_f32, int rows
     if (smem > 48 * 1024)                                                                                             \
       cudaFuncSetAttribute(moe_route_kernel<T, W, RB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
     moe_route_kernel<T, W, RB><<<(rows + RB - 1) / RB, ROUTE_WARPS * 32, smem, s>>>(                                  \
-        (const T*)h, ldh, (const W*)wr, rows, D, E, G, keep, top, scale, has_gate, vec_ok, sigmoid_scores, correction, \
-        group_top, renorm, idx, wt, gate_out);                                                                                \
+        (const T*)h, ldh, (const W*)wr, rows, D, vec_ok, choice);                                                     \
   } while (0)
 #define KVCM_ROUTE_RB(W)                                                                                              \
   do {                                                                                                                \

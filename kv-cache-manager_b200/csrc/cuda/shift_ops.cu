@@ -64,7 +64,7 @@ constexpr int kNormPairMaxRows = 4;
 // Slots of a block: 0 = the row before its first (when a shift needs it), 1..R = its rows, R + 1 = the last row of a
 // request that starts in this block and ends in a later one (its h becomes the request's state).
 template <typename T, int V, int R>
-__global__ void __launch_bounds__(kNormPairThreads)
+__global__ void __launch_bounds__(kNormPairThreads, 2)
 norm_pair_kernel(NormPairParams p) {
   constexpr int S = R + 2;
   extern __shared__ __align__(16) float vals[];      // [S][D], then (with experts) S * top weights and S * top places
@@ -131,11 +131,6 @@ norm_pair_kernel(NormPairParams p) {
     if (p.p1) add(p.p1, p.s1);
     if (p.p2) add(p.p2, p.s2);
     if (p.ey) {
-      float sum[S][V];
-#pragma unroll
-      for (int j = 0; j < S; ++j)
-#pragma unroll
-        for (int e = 0; e < V; ++e) sum[j][e] = 0.f;
       for (int k = 0; k < p.top; ++k)
 #pragma unroll
         for (int j = 0; j < S; ++j) {
@@ -143,14 +138,8 @@ norm_pair_kernel(NormPairParams p) {
           const Cols<V> a = Cols<V>::load(p.ey + size_t(eplace[j * p.top + k]) * D + i);
           const float w = ewt[j * p.top + k];
 #pragma unroll
-          for (int e = 0; e < V; ++e) sum[j][e] = fmaf(w, a.v[e], sum[j][e]);
+          for (int e = 0; e < V; ++e) c[j].v[e] = fmaf(w, a.v[e], c[j].v[e]);
         }
-#pragma unroll
-      for (int j = 0; j < S; ++j) {
-        if (src[j] < 0) continue;
-#pragma unroll
-        for (int e = 0; e < V; ++e) c[j].v[e] += sum[j][e];
-      }
     }
 #pragma unroll
     for (int j = 0; j < S; ++j) {

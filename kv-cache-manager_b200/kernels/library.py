@@ -1219,8 +1219,9 @@ def linear_chunk(qkv: torch.Tensor, bases, decay: torch.Tensor, state: torch.Ten
     _need(max(qb, kb) + qk_heads * dk <= C and vb + heads * dv <= C and out.shape == (qkv.shape[0], heads * dv)
           and state.shape[1] >= heads * dk * dv and ctx.tile_rows == 64, "linear_chunk: shapes")
     tiles = ctx.prefill_tiles
-    carry = torch.empty((tiles, heads, dk, dv), dtype=torch.float32, device=qkv.device)
-    _check(_lib().kvcm_linear_chunk(_p(qkv), C, qb, kb, vb, _p(decay), _p(carry), _p(state), _ll(state.stride(0)), _p(ctx.tile_seq),
+    _lib().kvcm_linear_chunk_scratch_bytes.restype = ctypes.c_longlong
+    scratch = torch.empty((int(_lib().kvcm_linear_chunk_scratch_bytes(tiles, heads, dk, dv)),), dtype=torch.uint8, device=qkv.device)
+    _check(_lib().kvcm_linear_chunk(_p(qkv), C, qb, kb, vb, _p(decay), _p(scratch), _p(state), _ll(state.stride(0)), _p(ctx.tile_seq),
                                     _p(ctx.tile_q0), _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out), tiles,
                                     heads, qk_heads, dk, dv, int(bool(silu)), _stream()), "linear_chunk", f"(dk={dk}, dv={dv})")
     global _launches
