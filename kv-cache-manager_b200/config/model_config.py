@@ -310,6 +310,23 @@ def _check_heads(m: Dict[str, Any], where: str) -> None:
         raise ConfigError(f"{where}: heads ({m['heads']}) must be a multiple of kv_heads ({m['kv_heads']})")
 
 
+def _check_rot_scaling(m: Dict[str, Any], where: str) -> None:
+    scaling = _section(m.get("rot") or {}, "scaling", where + " rot", optional=True)
+    if scaling:
+        for k in ("factor", "original", "fast", "slow"):
+            if not (_require(scaling, k, float, where + " rot.scaling") > 0):
+                raise ConfigError(f"{where}: rot.scaling.{k} must be positive")
+        if m["rot"]["base"] <= 1:
+            raise ConfigError(f"{where}: a scaled rotation needs a base above 1")
+
+
+def _check_decay(m: Dict[str, Any], where: str) -> None:
+    decay = m.get("decay")
+    if not isinstance(decay, list) or len(decay) != m["heads"] or \
+            any(isinstance(v, bool) or not isinstance(v, (int, float)) for v in decay):
+        raise ConfigError(f"{where}: decay must list one number for each of the {m['heads']} heads, got {decay!r}")
+
+
 @dataclass(frozen=True)
 class BifatarConfig(ModelConfig):
     """Bifatar: a decoder whose layers are listed one by one; every layer is a parallel block
@@ -675,22 +692,13 @@ class BimepelConfig(ModelConfig):
                 _check_heads(m, mw)
                 _require(m, "scale", float, mw)
                 _check_rot(m, mw)
-                scaling = _section(m.get("rot") or {}, "scaling", mw + " rot", optional=True)
-                if scaling:
-                    for k in ("factor", "original", "fast", "slow"):
-                        if not (_require(scaling, k, float, mw + " rot.scaling") > 0):
-                            raise ConfigError(f"{mw}: rot.scaling.{k} must be positive")
-                    if m["rot"]["base"] <= 1:
-                        raise ConfigError(f"{mw}: a scaled rotation needs a base above 1")
+                _check_rot_scaling(m, mw)
                 mask = _section(m, "mask", mw, optional=True)
                 if mask is not None and _require(mask, "size", int, mw + " mask") <= 0:
                     raise ConfigError(f"{mw}: mask.size must be positive")
             elif kind == "lightning":
                 _positive_ints(m, ("heads", "dim", "vdim"), mw)
-                decay = m.get("decay")
-                if not isinstance(decay, list) or len(decay) != m["heads"] or \
-                        any(isinstance(v, bool) or not isinstance(v, (int, float)) for v in decay):
-                    raise ConfigError(f"{mw}: decay must list one number for each of the {m['heads']} heads, got {decay!r}")
+                _check_decay(m, mw)
             else:
                 raise ConfigError(f"{lw}: unknown type {kind!r} (known: attention, lightning)")
             mlp = layer.get("mlp")
@@ -718,3 +726,85 @@ class BimepelConfig(ModelConfig):
         if self.has_loop:
             d["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
         return d
+
+
+# ------------------------------------------------------------------------------------ Pemorax
+
+@dataclass(frozen=True)
+class PemoraxConfig(ModelConfig):
+    """Pemorax: a decoder whose layers are listed one by one, every sublayer normalised on both sides and every mixer made of
+    two side by side, windowed attention and retention.
+
+    Top level: ``vocab``, ``width``, ``norm.eps`` and ``layers``: a list of {type, mixer, mlp}.  ``type`` "parallel": mixer {left
+    {heads, kv_heads, dim, vdim, scale, conv (taps; optional), rot {base, dims, scaling {factor, original, fast, slow}
+    (optional)} (optional), mask {size, keep_first (optional)} (optional), softcap (optional)}, right {heads, dim, vdim, decay
+    (one number per head), rot {base, dims} (optional)}}.  ``mlp`` is null, {kind: "dense", ff} or {kind: "moe", expert {ff},
+    router {experts, top}}.  ``layers`` is kept as the parsed JSON after validation; the builder reads every size from it."""
+    vocab: int = 0
+    width: int = 0
+    norm_eps: float = 1e-6
+    layers: tuple = ()
+
+    @classmethod
+    def from_json_dict(cls, d: Dict[str, Any]) -> "PemoraxConfig":
+        w = "config.json (Pemorax)"
+        norm = _section(d, "norm", w)
+        layers = d.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError(f"{w}: 'layers' must be a non-empty list")
+        cfg = cls(architecture="Pemorax", vocab=_require(d, "vocab", int, w), width=_require(d, "width", int, w),
+                  norm_eps=_require(norm, "eps", float, w + " norm"), layers=tuple(json.loads(json.dumps(layers))))
+        cfg.validate()
+        return cfg
+
+    def validate(self) -> None:
+        w = "PemoraxConfig"
+        if self.vocab <= 0 or self.width <= 0:
+            raise ConfigError(f"{w}: 'vocab' and 'width' must be positive")
+        if not (self.norm_eps > 0):
+            raise ConfigError(f"{w}: norm.eps must be positive, got {self.norm_eps}")
+        for i, layer in enumerate(self.layers):
+            lw = f"{w}: layer {i}"
+            if not isinstance(layer, dict):
+                raise ConfigError(f"{lw} must be an object")
+            if layer.get("type") != "parallel":
+                raise ConfigError(f"{lw}: unknown type {layer.get('type')!r} (known: parallel)")
+            m = _section(layer, "mixer", lw)
+            left, right = _section(m, "left", lw + " mixer"), _section(m, "right", lw + " mixer")
+            mw = lw + " mixer.left"
+            _check_heads(left, mw)
+            _require(left, "scale", float, mw)
+            _check_rot(left, mw)
+            _check_rot_scaling(left, mw)
+            if left.get("conv") is not None:
+                _positive_ints(left, ("conv",), mw)
+            if left.get("softcap") is not None and not (_require(left, "softcap", float, mw) > 0):
+                raise ConfigError(f"{mw}: softcap must be positive")
+            mask = _section(left, "mask", mw, optional=True)
+            if mask is not None:
+                _positive_ints(mask, ("size",), mw + " mask")
+                if mask.get("keep_first") is not None and _require(mask, "keep_first", int, mw + " mask") < 0:
+                    raise ConfigError(f"{mw}: mask.keep_first must not be negative")
+            mw = lw + " mixer.right"
+            _positive_ints(right, ("heads", "dim", "vdim"), mw)
+            _check_decay(right, mw)
+            _check_rot(right, mw)
+            _check_rot_scaling(right, mw)
+            mlp = layer.get("mlp")
+            if mlp is None:
+                continue
+            pw = lw + " mlp"
+            if not isinstance(mlp, dict) or mlp.get("kind") not in ("dense", "moe"):
+                raise ConfigError(f"{lw}: mlp must be null or of kind 'dense' or 'moe', got {mlp!r}")
+            if mlp["kind"] == "dense":
+                _positive_ints(mlp, ("ff",), pw)
+                continue
+            _positive_ints(_section(mlp, "expert", pw), ("ff",), pw + " expert")
+            r = _section(mlp, "router", pw)
+            _positive_ints(r, ("experts", "top"), pw + " router")
+            if r["top"] > r["experts"]:
+                raise ConfigError(f"{pw}: router cannot choose {r['top']} of {r['experts']} experts")
+
+    def to_json_dict(self) -> Dict[str, Any]:
+        return {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+                "layers": json.loads(json.dumps(list(self.layers)))}

@@ -11,8 +11,8 @@
 //           a second kernel.  With one partition the block writes the result itself (v1).
 // (Portions of more than one token: attention_tcgen05.cu and attention_prefill_mma.cu.)
 // Any head_dim that is a multiple of 16 up to 256, any page size, any number of heads and groups,
-// optional window (keys t > position - window) or chunk (keys of the position's own chunk; the partitions then
-// split the chunk's part of the context, not all of it).  Scores are scaled in float after the product;
+// optional window (keys t > position - window, and with it a request's first keys) or chunk (keys of the position's own
+// chunk); the partitions then split the window's or the chunk's part of the context, not all of it.  Scores are scaled in float after the product;
 // softmax by exp2 with log2(e) folded into the scale; probabilities are rounded to bfloat16 for
 // the P*V product, sums stay float.
 #include <cooperative_groups.h>
@@ -143,12 +143,12 @@ attn_decode_kernel(DecodeParams p) {
 
   const int ctx = p.seq_ctx_len[seq];
   const int lo = ctx > 0 ? first_visible(ctx - 1, p.window, p.chunk) : 0;
-  const int pbeg = (p.chunk > 0 ? lo / kKeyTile * kKeyTile : 0) + part * p.part_size;
+  const int pbeg = (p.chunk > 0 || p.window > 0 ? lo / kKeyTile * kKeyTile : 0) + part * p.part_size;
   const int begin = max(lo, pbeg);
   const int end = min(ctx, pbeg + p.part_size);
-  // Kept first keys that lie below the window: [pbeg, kend) of this partition (kend <= lo <= begin).
-  const int kend = p.keep_first > 0 ? min(min(p.keep_first, lo), end) : 0;
-  const bool has_kept = kend > pbeg;
+  // Kept first keys that lie below the window, [0, kend) with kend <= lo: the first partition's.
+  const int kend = p.keep_first > 0 && part == 0 ? min(p.keep_first, lo) : 0;
+  const bool has_kept = kend > 0;
   float* mo = reinterpret_cast<float*>(kbuf);                       // [4][16][HD]   (after the key loop)
   float* mm = mo + 4 * 16 * HD;                                     // [4][16]
   float* mlsum = mm + 4 * 16;                                       // [4][16]
@@ -179,7 +179,7 @@ attn_decode_kernel(DecodeParams p) {
   // here instead of one inside every round of the key loop.
   const int* table = p.block_tables + size_t(seq) * p.max_blocks;
   {
-    const int first_page = (has_kept ? pbeg : begin) / p.block_size;
+    const int first_page = (has_kept ? 0 : begin) / p.block_size;
     const int n_pages = ((begin < end ? end : kend) - 1) / p.block_size - first_page + 1;
     if (n_pages <= kTabMax) {
       for (int j = tid; j < n_pages; j += kAttnThreads) stab[j] = table[first_page + j];
@@ -191,11 +191,11 @@ attn_decode_kernel(DecodeParams p) {
   // Tiles: those of the kept first keys that start below the window's first tile, then the window's.
   const int t_first = (begin / kKeyTile) * kKeyTile;
   const int n_win = begin < end ? (end - t_first + kKeyTile - 1) / kKeyTile : 0;
-  int n_kept = has_kept ? (kend - pbeg + kKeyTile - 1) / kKeyTile : 0;
-  if (n_win > 0) n_kept = min(n_kept, (t_first - pbeg) / kKeyTile);
+  int n_kept = has_kept ? (kend + kKeyTile - 1) / kKeyTile : 0;
+  if (n_win > 0) n_kept = min(n_kept, t_first / kKeyTile);
   const int n_tiles = n_kept + n_win;
-  const int load_lo = has_kept ? pbeg : begin;
-  auto tile_start = [&](int i) { return i < n_kept ? pbeg + i * kKeyTile : t_first + (i - n_kept) * kKeyTile; };
+  const int load_lo = has_kept ? 0 : begin;
+  auto tile_start = [&](int i) { return i < n_kept ? i * kKeyTile : t_first + (i - n_kept) * kKeyTile; };
   auto load_stage = [&](int i) {                                   // tile i -> ring slot i % stages
     const int sl = i % kKVStages;
     if (i < n_tiles) {
@@ -468,8 +468,8 @@ KVCM_API int kvcm_attention_decode_cluster_parts(void) { return kMaxClusterParts
 // `softcap` > 0: scaled scores are capped as cap * tanh(score / cap); `sink` (per head, optional): exp(sink)
 // joins the softmax's denominator.
 // `keep_first` > 0 (with a window): the first keep_first keys of every request stay visible.  `chunk` > 0: a row sees
-// only its own chunk of positions, and the num_parts partitions of part_size keys cover [chunk's first key rounded down
-// to a tile of 64, context).
+// only its own chunk of positions.  With a window or a chunk the num_parts partitions of part_size keys cover [its first key
+// rounded down to a tile of 64, context).
 KVCM_API int kvcm_attention_decode_keep_bf16(const void* q, int q_stride, void* out, int out_stride,
                                              const void* k_cache, const void* v_cache, const int* block_tables,
                                              int max_blocks, const int* seq_ctx_len, int seqs, int nh, int nkv,

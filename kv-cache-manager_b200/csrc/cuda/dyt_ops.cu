@@ -5,10 +5,10 @@
 //              any of them absent), then  out = tanh(alpha * x) * w + b  in the storage type.
 //              The norm takes no statistics of the row; alpha is one number read from device memory.
 //              With `rows` the output rows are gathered from the listed input rows and x is left as it is.
-//   relu_sq:   out = max(x, 0)^2, the activation of an ungated feed-forward.
+//   unary_act: out = act(x), the activation of an ungated feed-forward (UnaryKind, gated_act.cuh).
 //
 // The stream, the sum and the tanh are float in both storage types.
-#include "common.cuh"
+#include "gated_act.cuh"
 #include "pdl.cuh"
 
 namespace kvcm {
@@ -72,18 +72,17 @@ dyt_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ p0, float s
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-relu_sq_kernel(const T* in, T* out, long long n) {
+unary_act_kernel(const T* in, T* out, long long n, int kind) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    const float v = fmaxf(ldf(in + i), 0.f);
-    stf(out + i, v * v);
+    stf(out + i, unary_act(kind, ldf(in + i)));
   }
 }
 
 // bfloat16, eight elements a thread (16-byte accesses): n % 8 == 0 and aligned pointers.
 __global__ void __launch_bounds__(256)
-relu_sq_vec_kernel(const uint4* in, uint4* out, long long n8) {
+unary_act_vec_kernel(const uint4* in, uint4* out, long long n8, int kind) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n8; i += (long long)gridDim.x * blockDim.x) {
@@ -92,8 +91,7 @@ relu_sq_vec_kernel(const uint4* in, uint4* out, long long n8) {
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       float2 f = __bfloat1622float2(h[k]);
-      f.x = fmaxf(f.x, 0.f); f.y = fmaxf(f.y, 0.f);
-      h[k] = __floats2bfloat162_rn(f.x * f.x, f.y * f.y);
+      h[k] = __floats2bfloat162_rn(unary_act(kind, f.x), unary_act(kind, f.y));
     }
     out[i] = v;
   }
@@ -124,17 +122,20 @@ KVCM_API int kvcm_dyt_norm_bf16(float* x, const float* p0, float s0, const float
   return launch_dyt_norm<bf16>(x, p0, s0, p1, s1, p2, s2, w, b, alpha, (bf16*)out, rows, n_rows, hidden, (cudaStream_t)stream);
 }
 
-KVCM_API int kvcm_relu_sq_f32(const void* in, void* out, long long n, void* stream) {
+// kind: UnaryKind.
+KVCM_API int kvcm_unary_act_f32(const void* in, void* out, long long n, int kind, void* stream) {
   if (n == 0) return 0;
+  if (kind < kUnaryReluSq || kind > kUnaryGeluTanh) return KVCM_ERR_UNSUPPORTED;
   const int blocks = int(min((n + 255) / 256, (long long)148 * 16));
-  return pdl_launch(relu_sq_kernel<float>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const float*)in, (float*)out, n);
+  return pdl_launch(unary_act_kernel<float>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const float*)in, (float*)out, n, kind);
 }
-KVCM_API int kvcm_relu_sq_bf16(const void* in, void* out, long long n, void* stream) {
+KVCM_API int kvcm_unary_act_bf16(const void* in, void* out, long long n, int kind, void* stream) {
   if (n == 0) return 0;
+  if (kind < kUnaryReluSq || kind > kUnaryGeluTanh) return KVCM_ERR_UNSUPPORTED;
   if (n % 8 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
     const int vblocks = int(min((n / 8 + 255) / 256, (long long)148 * 16));
-    return pdl_launch(relu_sq_vec_kernel, dim3(vblocks), dim3(256), 0, (cudaStream_t)stream, (const uint4*)in, (uint4*)out, n / 8);
+    return pdl_launch(unary_act_vec_kernel, dim3(vblocks), dim3(256), 0, (cudaStream_t)stream, (const uint4*)in, (uint4*)out, n / 8, kind);
   }
   const int blocks = int(min((n + 255) / 256, (long long)148 * 16));
-  return pdl_launch(relu_sq_kernel<bf16>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const bf16*)in, (bf16*)out, n);
+  return pdl_launch(unary_act_kernel<bf16>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const bf16*)in, (bf16*)out, n, kind);
 }

@@ -459,7 +459,7 @@ using namespace kvcm;
                                           float limit, float alpha, void* stream) {                   \
     if (rows == 0) return 0;                                                                          \
     return launch_gated_act<T, kGatedClamped>((const T*)gate_up, (T*)out, rows, inter,                \
-                                              GatedAct{limit, alpha}, (cudaStream_t)stream);          \
+                                              GatedAct{limit, alpha, 0}, (cudaStream_t)stream);          \
   }                                                                                                   \
   KVCM_API int kvcm_gather_rows_##SUFFIX(const void* src, const int* rows, void* dst, int n,          \
                                          int width, void* stream) {                                   \

@@ -104,8 +104,8 @@ struct StreamParams {
   // SCALED: the sums of row m are multiplied by rsqrt(sum over t of ss_in[t][m] / K + eps) before the
   // epilogue (ss_in [ss_tiles][kNormRows] as kResidual leaves it)
   const float* ss_in; int ss_tiles; float eps;
-  // kStore: 1 = the stored value is max(y, 0)^2 of the rounded sum y (an ungated feed-forward's activation)
-  int relu_sq;
+  // kStore: UnaryKind of what is stored of the rounded sum (an ungated feed-forward's activation)
+  int unary;
   // kSiluMul: which activation joins gate and up (GatedKind; 0 counts as SiLU)
   int gate_kind; GatedAct gate_act;
 };
@@ -493,10 +493,7 @@ gemm_stream_kernel(StreamParams p) {
         const int n = row_in(base, r);
         if (n < p.N && m < p.M) {
           float v = total_of(r, m);
-          if (p.relu_sq) {                                       // as the separate kernel: round, clamp, square
-            v = fmaxf(Store<OutT>::round(v), 0.f);
-            v *= v;
-          }
+          if (p.unary) v = unary_act(p.unary, Store<OutT>::round(v));   // as the separate kernel: of the rounded sum
           stf(Y + size_t(m) * p.ldy + n, v);
         }
       }
@@ -645,15 +642,15 @@ KVCM_API int kvcm_gemm_stream_bf16(const void* X, const void* W, void* Y, int M,
   return out_f32 ? launch_stream<2, float, kStore>(p, sm_count, s) : launch_stream<2, bf16, kStore>(p, sm_count, s);
 }
 
-// The plain product with the squared ReLU applied to the rounded sums: Y = bfloat16(max(bfloat16(X * W^T), 0)^2).
-KVCM_API int kvcm_gemm_stream_relu_sq_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int ldx,
-                                           int ldw, int ldy, int sm_count, void* stream) {
+// The plain product with an activation applied to the rounded sums: Y = bfloat16(act(bfloat16(X * W^T))), act a UnaryKind.
+KVCM_API int kvcm_gemm_stream_act_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int ldx,
+                                           int ldw, int ldy, int kind, int sm_count, void* stream) {
   if (M == 0 || N == 0) return 0;
-  if (!stream_ok(M, N, K, sm_count, true) || (ldw % 8) || (ldx % 8)) return KVCM_ERR_UNSUPPORTED;
+  if (!stream_ok(M, N, K, sm_count, true) || (ldw % 8) || (ldx % 8) || kind < kUnaryReluSq || kind > kUnaryGeluTanh) return KVCM_ERR_UNSUPPORTED;
   if ((reinterpret_cast<uintptr_t>(W) & 15) || (reinterpret_cast<uintptr_t>(X) & 15)) return KVCM_ERR_UNSUPPORTED;
   StreamParams p = {};
   p.W = (const bf16*)W; p.N = N; p.K = K; p.ldw = ldw; p.X = (const bf16*)X; p.ldx = ldx; p.M = M;
-  p.Y = Y; p.ldy = ldy; p.relu_sq = 1;
+  p.Y = Y; p.ldy = ldy; p.unary = kind;
   p.pair_blocks = 1; p.group_stride = 16; p.pair_offset = 8;
   cudaStream_t s = (cudaStream_t)stream;
   return M <= 8 ? launch_stream<1, bf16, kStore>(p, sm_count, s) : launch_stream<2, bf16, kStore>(p, sm_count, s);
@@ -741,7 +738,7 @@ KVCM_API int kvcm_gate_up_silu_scaled_bf16(const void* X, const float* ss_in, in
 // The same with the clamped activation (no row scale).
 KVCM_API int kvcm_gate_up_clamped_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw, int ldy,
                                        float limit, float alpha, int sm_count, void* stream) {
-  return gate_up_stream(X, nullptr, 0, 0.f, W, Y, M, I, K, ldx, ldw, ldy, sm_count, kGatedClamped, GatedAct{limit, alpha}, stream);
+  return gate_up_stream(X, nullptr, 0, 0.f, W, Y, M, I, K, ldx, ldw, ldy, sm_count, kGatedClamped, GatedAct{limit, alpha, 0}, stream);
 }
 
 KVCM_API int kvcm_gate_up_silu_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw,

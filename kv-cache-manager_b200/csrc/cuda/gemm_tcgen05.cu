@@ -32,7 +32,7 @@ __device__ int g_tcgen05_error = 0;
 // n0..n0+127 and the 128 up columns N+n0.., and the epilogue stores
 // y[m][n] = round(round(silu(round(gate))) * round(up)) -- the roundings of the separate product
 // and activation kernels -- so the [M, 2N] intermediate never goes to memory.  (GATED is a GatedKind: SiLU or the
-// clamped activation, gated_act.cuh.)
+// clamped activation, gated_act.cuh.)  Ungated with a bfloat16 result: `act.unary` is applied to the rounded sums.
 template <typename OutT, int BN, int GATED>
 __global__ void __launch_bounds__(kTcThreads)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
@@ -209,6 +209,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
               __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(packed);
 #pragma unroll
               for (int i = 0; i < 16; ++i) h2[i] = __floats2bfloat162_rn(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1]));
+              if (act.unary) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                  const float2 f = __bfloat1622float2(h2[i]);
+                  h2[i] = __floats2bfloat162_rn(unary_act(act.unary, f.x), unary_act(act.unary, f.y));
+                }
+              }
 #pragma unroll
               for (int i = 0; i < 4; ++i) reinterpret_cast<uint4*>(dst)[i] = packed[i];
             } else {
@@ -219,7 +226,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
           } else {
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              if (col0 + i < N) stf(dst + i, __uint_as_float(v[i]));
+              if (col0 + i < N) {
+                  const float f = __uint_as_float(v[i]);
+                  stf(dst + i, act.unary ? unary_act(act.unary, Store<OutT>::round(f)) : f);
+                }
           }
         }
       }
@@ -266,7 +276,7 @@ int launch_tcgen05_bn(const void* X, const void* W, void* Y, int M, int N, int K
 
 template <typename OutT>
 int launch_tcgen05(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                   cudaStream_t s) {
+                   cudaStream_t s, GatedAct act = GatedAct{}) {
   static int sm_count = 0;
   if (sm_count == 0) {
     int dev = 0;
@@ -278,8 +288,8 @@ int launch_tcgen05(const void* X, const void* W, void* Y, int M, int N, int K, i
   const long long m_tiles = (M + kTcBM - 1) / kTcBM;
   const long long t256 = m_tiles * ((N + 255) / 256), t128 = m_tiles * ((N + 127) / 128);
   const long long cost256 = ((t256 + sm_count - 1) / sm_count) * 256, cost128 = ((t128 + sm_count - 1) / sm_count) * 128;
-  if (cost128 * 3 < cost256 * 2) return launch_tcgen05_bn<OutT, 128>(X, W, Y, M, N, K, ldx, ldw, ldy, sm_count, s);
-  return launch_tcgen05_bn<OutT, 256>(X, W, Y, M, N, K, ldx, ldw, ldy, sm_count, s);
+  if (cost128 * 3 < cost256 * 2) return launch_tcgen05_bn<OutT, 128>(X, W, Y, M, N, K, ldx, ldw, ldy, sm_count, s, act);
+  return launch_tcgen05_bn<OutT, 256>(X, W, Y, M, N, K, ldx, ldw, ldy, sm_count, s, act);
 }
 
 }  // namespace kvcm
@@ -307,7 +317,7 @@ KVCM_API int kvcm_gate_up_silu_tcgen05_bf16(const void* X, const void* W, void* 
 // The same with the clamped activation.
 KVCM_API int kvcm_gate_up_clamped_tcgen05_bf16(const void* X, const void* W, void* Y, int M, int I, int K, int ldx, int ldw,
                                                int ldy, float limit, float alpha, void* stream) {
-  return gate_up_tcgen05<kGatedClamped>(X, W, Y, M, I, K, ldx, ldw, ldy, GatedAct{limit, alpha}, stream);
+  return gate_up_tcgen05<kGatedClamped>(X, W, Y, M, I, K, ldx, ldw, ldy, GatedAct{limit, alpha, 0}, stream);
 }
 
 KVCM_API int kvcm_gemm_tcgen05_supports(int M, int N, int K, int ldx, int ldw) {
@@ -323,6 +333,15 @@ KVCM_API int kvcm_gemm_tcgen05_bf16(const void* X, const void* W, void* Y, int M
   cudaStream_t s = (cudaStream_t)stream;
   return out_f32 ? launch_tcgen05<float>(X, W, Y, M, N, K, ldx, ldw, ldy, s)
                  : launch_tcgen05<bf16>(X, W, Y, M, N, K, ldx, ldw, ldy, s);
+}
+
+// Y = bfloat16(act(bfloat16(X * W^T))), act a UnaryKind: an ungated feed-forward's up product with its activation.
+KVCM_API int kvcm_gemm_tcgen05_act_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
+                                        int kind, void* stream) {
+  if (M == 0 || N == 0) return 0;
+  if (!kvcm_gemm_tcgen05_supports(M, N, K, ldx, ldw) || kind < kUnaryReluSq || kind > kUnaryGeluTanh) return KVCM_ERR_UNSUPPORTED;
+  if ((reinterpret_cast<uintptr_t>(X) & 15) || (reinterpret_cast<uintptr_t>(W) & 15)) return KVCM_ERR_UNSUPPORTED;
+  return launch_tcgen05<bf16>(X, W, Y, M, N, K, ldx, ldw, ldy, (cudaStream_t)stream, GatedAct{0.f, 0.f, kind});
 }
 
 // Device address of the error word (the sampling kernels copy it out with the step's tokens).

@@ -20,7 +20,8 @@
 // Precision: q, k and v (after the optional SiLU) are bfloat16 operands, as the projections of a 16-bit model may be.
 // Whatever belongs to the recurrence is kept to more than float's 16 leading bits: operands that hold a decay or the state
 // (d^m k, S, the decayed scores) are split into two bfloat16 parts, x = hi + lo with |x - hi - lo| <= 2^-17 |x|, and
-// multiplied in two products; all sums, P and S are float.
+// multiplied in two products; all sums, P and S are float.  With `exact` the queries and keys are no plain projections
+// (rotated, scaled) and are split the same way (products of two low parts, 2^-18 of a term, are left out).
 // (Portions of one token, float storage and key sizes beyond 128 stay with the token-by-token kernel.)
 #include "attention_mma.cuh"
 #include "pdl.cuh"
@@ -37,6 +38,7 @@ struct LinearChunkParams {
   float* outer;                            // P      [tiles, heads, DK, DVP]
   bf16* split;                             // S      [tiles, heads, 2 (hi, lo), DK, DVP]
   bf16* q; bf16* k; bf16* v;               // [tiles, heads, 64, DK] twice, [tiles, heads, 64, DVP]
+  bf16* q_lo; bf16* k_lo;                  // exact: the low parts of q and k, like them; else null
   float* state; long long state_stride;
   const int* tile_seq; const int* tile_q0; const int* seq_q_start; const int* seq_q_len; const int* seq_state_slot;
   float* out;                              // [rows, heads * dv]
@@ -143,12 +145,15 @@ linear_chunk_outer_kernel(LinearChunkParams p) {
     float y[4], hi[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      y[e] = lc_round(x[e]) * f;
+      y[e] = (p.k_lo ? x[e] : lc_round(x[e])) * f;
       hi[e] = lc_round(y[e]);
     }
     lc_store4(khi + r * LDK + c, hi[0], hi[1], hi[2], hi[3]);
     lc_store4(klo + r * LDK + c, y[0] - hi[0], y[1] - hi[1], y[2] - hi[2], y[3] - hi[3]);
-    if (first) lc_store4(kg + r * DK + c, x[0], x[1], x[2], x[3]);
+    if (first) {
+      lc_store4(kg + r * DK + c, x[0], x[1], x[2], x[3]);
+      if (p.k_lo) lc_store4(p.k_lo + th * kLcRows * DK + r * DK + c, x[0] - lc_round(x[0]), x[1] - lc_round(x[1]), x[2] - lc_round(x[2]), x[3] - lc_round(x[3]));
+    }
   });
   lc_rows<DVB>(src + p.v_base + head * p.dv + c0, p.ld, n, p.dv - c0, p.silu, p.vec, [&](int r, int c, const float (&x)[4]) {
     lc_store4(vs + r * LDV + c, x[0], x[1], x[2], x[3]);
@@ -156,7 +161,10 @@ linear_chunk_outer_kernel(LinearChunkParams p) {
   });
   if (first)
     lc_rows<DK>(src + p.q_base + qk, p.ld, n, p.dk, p.silu, p.vec,
-                [&](int r, int c, const float (&x)[4]) { lc_store4(qg + r * DK + c, x[0], x[1], x[2], x[3]); });
+                [&](int r, int c, const float (&x)[4]) {
+                  lc_store4(qg + r * DK + c, x[0], x[1], x[2], x[3]);
+                  if (p.q_lo) lc_store4(p.q_lo + th * kLcRows * DK + r * DK + c, x[0] - lc_round(x[0]), x[1] - lc_round(x[1]), x[2] - lc_round(x[2]), x[3] - lc_round(x[3]));
+                });
   __syncthreads();
   float* dst = p.outer + th * DK * p.dvp + c0;
   const int g = lane >> 2, t4 = lane & 3;
@@ -240,7 +248,8 @@ __device__ __forceinline__ void lc_copy_tile(bf16* dst, const bf16* src, int row
   }
 }
 
-template <int DK>
+// EXACT: q and k in two parts each; the low part of q waits behind S, that of k takes the place of q once q is in registers.
+template <int DK, bool EXACT>
 __global__ void __launch_bounds__(kLcReadThreads)
 linear_chunk_read_kernel(LinearChunkParams p) {
   constexpr int LDK = DK + 8, LDV = kLcCols + 8;
@@ -250,6 +259,7 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   bf16* vs = ks + kLcRows * LDK;                              // [64][LDV]
   bf16* shi = vs + kLcRows * LDV;                             // [DK][LDV]
   bf16* slo = shi + DK * LDV;
+  bf16* qls = slo + DK * LDV;                                 // EXACT: [64][LDK]
   __shared__ float pw[kLcRows + 1];
   pdl_launch_dependents();
   const int tile = blockIdx.x, head = blockIdx.y, c0 = blockIdx.z * kLcCols;
@@ -261,6 +271,7 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   const size_t th = size_t(tile) * p.heads + head;
   const bf16* S = p.split + 2 * th * DK * p.dvp + c0;
   lc_copy_tile<DK>(qs, p.q + th * kLcRows * DK, kLcRows, DK);
+  if constexpr (EXACT) lc_copy_tile<DK>(qls, p.q_lo + th * kLcRows * DK, kLcRows, DK);
   lc_copy_tile<kLcCols>(shi, S, DK, p.dvp);
   lc_copy_tile<kLcCols>(slo, S + size_t(DK) * p.dvp, DK, p.dvp);
   cp_async_commit();
@@ -272,6 +283,13 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   const int g = lane >> 2, t4 = lane & 3;
   uint32_t qa[DK / 16][4];
   load_q_frags<DK>(qa, qs + warp * 16 * LDK, lane);
+  uint32_t ql[EXACT ? DK / 16 : 1][4];
+  if constexpr (EXACT) {
+    load_q_frags<DK>(reinterpret_cast<uint32_t(&)[DK / 16][4]>(ql), qls + warp * 16 * LDK, lane);
+    __syncthreads();                                           // every warp has its rows of q
+    lc_copy_tile<DK>(qs, p.k_lo + th * kLcRows * DK, kLcRows, DK);
+    cp_async_commit();
+  }
   float o[kLcCols / 8][4];
 #pragma unroll
   for (int i = 0; i < kLcCols / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -279,6 +297,7 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   for (int kk = 0; kk < DK / 16; ++kk) {
     pv_16x16<kLcCols>(o, qa[kk], shi + kk * 16 * LDV, lane);
     pv_16x16<kLcCols>(o, qa[kk], slo + kk * 16 * LDV, lane);
+    if constexpr (EXACT) pv_16x16<kLcCols>(o, ql[kk], shi + kk * 16 * LDV, lane);
   }
   cp_async_wait<0>();
   __syncthreads();                                             // every thread's share of k and v is there
@@ -291,6 +310,15 @@ linear_chunk_read_kernel(LinearChunkParams p) {
   for (int kb = 0; kb <= warp; ++kb) {                         // sixteen keys at a time, up to the rows' own
     float s[2][4];
     qk_16x16<DK>(s, qa, ks + kb * 16 * LDK, lane);
+    if constexpr (EXACT) {
+      float a[2][4], b[2][4];
+      qk_16x16<DK>(a, reinterpret_cast<const uint32_t(&)[DK / 16][4]>(ql), ks + kb * 16 * LDK, lane);
+      qk_16x16<DK>(b, qa, qs + kb * 16 * LDK, lane);
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[h][j] += a[h][j] + b[h][j];
+    }
     float lo[2][4];
 #pragma unroll
     for (int h = 0; h < 2; ++h)
@@ -325,8 +353,8 @@ linear_chunk_read_kernel(LinearChunkParams p) {
 }
 
 // Scratch of a launch, in bytes from a 16-byte aligned start: P, then S split, q, k, v (every part a multiple of 16).
-struct LinearChunkScratch { long long outer, split, q, k, v, total; };
-static LinearChunkScratch linear_chunk_scratch(int tiles, int heads, int DK, int dvp) {
+struct LinearChunkScratch { long long outer, split, q, k, v, q_lo, k_lo, total; };
+static LinearChunkScratch linear_chunk_scratch(int tiles, int heads, int DK, int dvp, int exact) {
   const long long th = (long long)tiles * heads;
   LinearChunkScratch s;
   s.outer = 0;
@@ -334,7 +362,9 @@ static LinearChunkScratch linear_chunk_scratch(int tiles, int heads, int DK, int
   s.q = s.split + th * DK * dvp * 4;
   s.k = s.q + th * kLcRows * DK * 2;
   s.v = s.k + th * kLcRows * DK * 2;
-  s.total = s.v + th * kLcRows * dvp * 2;
+  s.q_lo = s.v + th * kLcRows * dvp * 2;
+  s.k_lo = s.q_lo + (exact ? th * kLcRows * DK * 2 : 0);
+  s.total = s.k_lo + (exact ? th * kLcRows * DK * 2 : 0);
   return s;
 }
 static int linear_chunk_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : 128; }
@@ -352,12 +382,12 @@ static int launch_linear_outer(const LinearChunkParams& p, cudaStream_t s) {
   return pdl_launch(linear_chunk_outer_kernel<DK, DVB>, dim3(p.tiles, p.heads, p.dvp / DVB), dim3(kLcOuterThreads), smem, s, p);
 }
 
-template <int DK>
-static int launch_linear_chunk(const LinearChunkParams& p, cudaStream_t s) {
-  constexpr size_t smem = size_t(2 * kLcRows * (DK + 8) + kLcRows * (kLcCols + 8) + 2 * DK * (kLcCols + 8)) * sizeof(bf16);
+template <int DK, bool EXACT>
+static int launch_linear_chunk_as(const LinearChunkParams& p, cudaStream_t s) {
+  constexpr size_t smem = size_t((EXACT ? 3 : 2) * kLcRows * (DK + 8) + kLcRows * (kLcCols + 8) + 2 * DK * (kLcCols + 8)) * sizeof(bf16);
   static bool configured = false;
   if (!configured && smem > 40 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(linear_chunk_read_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    const cudaError_t e = cudaFuncSetAttribute(linear_chunk_read_kernel<DK, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     if (e != cudaSuccess) return int(e);
     configured = true;
   }
@@ -366,7 +396,11 @@ static int launch_linear_chunk(const LinearChunkParams& p, cudaStream_t s) {
   const long long quads = (long long)p.heads * DK * p.dvp / 4;
   rc = pdl_launch(linear_chunk_carry_kernel, dim3(unsigned((quads + 255) / 256), p.tiles), dim3(256), 0, s, p, DK);
   if (rc) return rc;
-  return pdl_launch(linear_chunk_read_kernel<DK>, dim3(p.tiles, p.heads, p.dvp / kLcCols), dim3(kLcReadThreads), smem, s, p);
+  return pdl_launch(linear_chunk_read_kernel<DK, EXACT>, dim3(p.tiles, p.heads, p.dvp / kLcCols), dim3(kLcReadThreads), smem, s, p);
+}
+template <int DK>
+static int launch_linear_chunk(const LinearChunkParams& p, cudaStream_t s) {
+  return p.q_lo ? launch_linear_chunk_as<DK, true>(p, s) : launch_linear_chunk_as<DK, false>(p, s);
 }
 
 }  // namespace kvcm
@@ -377,8 +411,8 @@ using namespace kvcm;
 KVCM_API int kvcm_linear_chunk_max_dk(void) { return 128; }
 
 // Bytes of scratch for a step of `tiles` chunks.
-KVCM_API long long kvcm_linear_chunk_scratch_bytes(int tiles, int heads, int dk, int dv) {
-  return linear_chunk_scratch(tiles, heads, linear_chunk_dk(dk), linear_chunk_dvp(dv)).total;
+KVCM_API long long kvcm_linear_chunk_scratch_bytes(int tiles, int heads, int dk, int dv, int exact) {
+  return linear_chunk_scratch(tiles, heads, linear_chunk_dk(dk), linear_chunk_dvp(dv), exact).total;
 }
 
 // Runs the recurrence over the rows of every portion of more than one token (the step's tiles of 64 rows); single-row
@@ -387,7 +421,7 @@ KVCM_API long long kvcm_linear_chunk_scratch_bytes(int tiles, int heads, int dk,
 KVCM_API int kvcm_linear_chunk(const float* proj, int ld, int q_base, int k_base, int v_base, const float* decay, void* scratch,
                                float* state, long long state_stride, const int* tile_seq, const int* tile_q0,
                                const int* seq_q_start, const int* seq_q_len, const int* seq_state_slot, float* out, int tiles,
-                               int heads, int qk_heads, int dk, int dv, int silu, void* stream) {
+                               int heads, int qk_heads, int dk, int dv, int silu, int exact, void* stream) {
   if (tiles == 0) return 0;
   if (dk < 1 || dk > 128 || dv < 1 || qk_heads < 1 || heads % qk_heads || tiles > 65535 || heads > 65535 ||
       (reinterpret_cast<uintptr_t>(scratch) & 15))
@@ -397,10 +431,11 @@ KVCM_API int kvcm_linear_chunk(const float* proj, int ld, int q_base, int k_base
   p.state = state; p.state_stride = state_stride; p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.seq_q_start = seq_q_start;
   p.seq_q_len = seq_q_len; p.seq_state_slot = seq_state_slot; p.out = out; p.tiles = tiles; p.heads = heads;
   p.qk_heads = qk_heads; p.dk = dk; p.dv = dv; p.dvp = linear_chunk_dvp(dv); p.silu = silu;
-  const LinearChunkScratch at = linear_chunk_scratch(tiles, heads, linear_chunk_dk(dk), p.dvp);
+  const LinearChunkScratch at = linear_chunk_scratch(tiles, heads, linear_chunk_dk(dk), p.dvp, exact);
   char* base = static_cast<char*>(scratch);
   p.outer = reinterpret_cast<float*>(base + at.outer); p.split = reinterpret_cast<bf16*>(base + at.split);
   p.q = reinterpret_cast<bf16*>(base + at.q); p.k = reinterpret_cast<bf16*>(base + at.k); p.v = reinterpret_cast<bf16*>(base + at.v);
+  p.q_lo = exact ? reinterpret_cast<bf16*>(base + at.q_lo) : nullptr; p.k_lo = exact ? reinterpret_cast<bf16*>(base + at.k_lo) : nullptr;
   p.vec = (dk % 4) == 0 && (dv % 4) == 0 && (ld % 4) == 0 && (q_base % 4) == 0 && (k_base % 4) == 0 && (v_base % 4) == 0 &&
           (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
   cudaStream_t s = (cudaStream_t)stream;

@@ -8,7 +8,8 @@
 //            sigmoid(z) instead of the softmax; a `correction` per expert that is added to the scores
 //            for the choice only (choice scores may then be negative; the weights use the scores
 //            themselves); a group's score as the sum of its two largest choice scores; the chosen scores divided by
-//            their sum before the scale (`renorm`).
+//            their sum before the scale (`renorm`); a `bias` per expert that joins the logits; weights that are the
+//            softmax over the chosen logits only (the largest logits win).
 //   sort     the (row, choice) pairs ordered by expert, cut into tiles of 64 pairs of one expert.
 //   gate_up  act[pair] = silu(h[row] Wg_e^T) * (h[row] Wu_e^T)      per tile, float accumulation
 //   down     y[pair]   = act[pair] Wd_e^T                           per tile, float results
@@ -72,14 +73,15 @@ __device__ __forceinline__ void route_load(const bf16* p, float (&v)[8]) {
 // One warp's choice for one row.  `z`: the row's E logits (and the gate's behind them) in shared memory, then room for the
 // groups' scores and the choice scores.
 struct RouteChoice {
-  int E, G, keep, top, has_gate, sigmoid_scores, group_top, renorm;
+  int E, G, keep, top, has_gate, scores, group_top, renorm;      // scores: 0 softmax, 1 sigmoid, 2 softmax over the chosen logits only
   float scale;
   const float* correction;
+  const float* bias;                                         // [E], joins the logits; or null
   int* idx; float* wt; float* gate_out;
 };
 __device__ __forceinline__ void route_choose(const RouteChoice& c, float* z, int row, int lane) {
-  const int E = c.E, G = c.G, keep = c.keep, top = c.top, has_gate = c.has_gate, sigmoid_scores = c.sigmoid_scores,
-            group_top = c.group_top, renorm = c.renorm;
+  const int E = c.E, G = c.G, keep = c.keep, top = c.top, has_gate = c.has_gate, group_top = c.group_top, renorm = c.renorm;
+  const bool sigmoid_scores = c.scores == 1, chosen_softmax = c.scores == 2;
   const float scale = c.scale;
   const float* correction = c.correction;
   int* idx = c.idx;
@@ -87,7 +89,13 @@ __device__ __forceinline__ void route_choose(const RouteChoice& c, float* z, int
   float* gate_out = c.gate_out;
   float* gb = z + E + 1;
   float* ch = gb + G;                                        // choice scores: -inf once taken
-  if (sigmoid_scores) {
+  if (c.bias) {                                              // (lane by lane: the element an expert's lane reads below)
+    for (int e = lane; e < E; e += 32) z[e] += c.bias[e];
+  }
+  if (chosen_softmax) {
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) ch[e] = z[e];         // the logits choose; the chosen ones become weights at the end
+  } else if (sigmoid_scores) {
     __syncwarp();
     for (int e = lane; e < E; e += 32) {
       ch[e] = z[e];                                          // (the sigmoid keeps the order; in float it makes large logits equal)
@@ -104,7 +112,7 @@ __device__ __forceinline__ void route_choose(const RouteChoice& c, float* z, int
     for (int e = lane; e < E; e += 32) z[e] = expf(z[e] - m) / sum;
   }
   const bool limited = G > 1 && keep < G;
-  if (!sigmoid_scores || correction || limited)
+  if (!(sigmoid_scores || chosen_softmax) || correction || limited)
     for (int e = lane; e < E; e += 32) ch[e] = z[e] + (correction ? correction[e] : 0.f);
   if (has_gate && lane == 0) gate_out[row] = 1.f / (1.f + expf(-z[E]));
   __syncwarp();
@@ -165,11 +173,27 @@ __device__ __forceinline__ void route_choose(const RouteChoice& c, float* z, int
       const int at = (k & ~31) + lane;
       if (at <= k) {
         idx[size_t(row) * top + at] = my_expert;
-        wt[size_t(row) * top + at] = mine * scale;
+        wt[size_t(row) * top + at] = chosen_softmax ? mine : mine * scale;
       }
     }
   }
-  if (renorm) {
+  if (chosen_softmax) {
+    float* w = wt + size_t(row) * top;
+    if (top <= 32) {
+      const float m = warp_max(lane < top ? mine : -INFINITY);
+      const float e = lane < top ? expf(mine - m) : 0.f;
+      const float sum = warp_sum(e);
+      if (lane < top) w[lane] = e / sum * scale;
+    } else {
+      __syncwarp();
+      float m = -INFINITY, sum = 0.f;
+      for (int k = lane; k < top; k += 32) m = fmaxf(m, w[k]);
+      m = warp_max(m);
+      for (int k = lane; k < top; k += 32) sum += expf(w[k] - m);
+      sum = warp_sum(sum);
+      for (int k = lane; k < top; k += 32) w[k] = expf(w[k] - m) / sum * scale;
+    }
+  } else if (renorm) {
     if (top <= 32) {
       if (lane < top) wt[size_t(row) * top + lane] = mine / (chosen + 1e-20f) * scale;
     } else {
@@ -497,17 +521,17 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place_of
 
 template <typename T>
 int launch_moe_route(const void* h, int ldh, const void* wr, int w_f32, int rows, int D, int E, int G, int keep, int top,
-                     float scale, int has_gate, int sigmoid_scores, const float* correction, int group_top, int renorm, int* idx,
+                     float scale, int has_gate, int scores, const float* bias, const float* correction, int group_top, int renorm, int* idx,
                      float* wt, float* gate_out, cudaStream_t s) {
   if (rows == 0) return 0;
-  if (E < 1 || G < 1 || E % G || keep < 1 || keep > G || top < 1 || top > (E / G) * keep || group_top < 1 || group_top > 2)
+  if (E < 1 || G < 1 || E % G || keep < 1 || keep > G || top < 1 || top > (E / G) * keep || group_top < 1 || group_top > 2 || scores < 0 || scores > 2)
     return KVCM_ERR_UNSUPPORTED;
   const size_t zstride = (size_t(2 * E + 1 + G) + 3) & ~size_t(3);
   int rb = rows >= 512 ? 8 : 1;                                       // many rows: read the router once for 8 of them
   while (rb > 1 && (rb * (zstride + D)) * sizeof(float) > 160 * 1024) rb /= 2;
   const size_t smem = rb * (zstride + D) * sizeof(float);
   if (smem > 200 * 1024) return KVCM_ERR_UNSUPPORTED;
-  const RouteChoice choice = {E, G, keep, top, has_gate, sigmoid_scores, group_top, renorm, scale, correction, idx, wt, gate_out};
+  const RouteChoice choice = {E, G, keep, top, has_gate, scores, group_top, renorm, scale, correction, bias, idx, wt, gate_out};
   if constexpr (sizeof(T) == 2) {
     const int outs = E + (has_gate ? 1 : 0), np = outs <= 32 ? 32 : 64;
     const size_t mma_smem = ROUTE_MMA_ROWS * (zstride + ROUTE_WARPS * np) * sizeof(float);
@@ -618,10 +642,10 @@ KVCM_API int kvcm_moe_experts_tc_bf16(const void* h, int ldh, const void* wgu, c
 
 #define KVCM_MOE(SUFFIX, T)                                                                                          \
   KVCM_API int kvcm_moe_route_##SUFFIX(const void* h, int ldh, const void* wr, int w_f32, int rows, int D, int E,    \
-                                       int G, int keep, int top, float scale, int has_gate, int sigmoid_scores,      \
-                                       const float* correction, int group_top, int renorm, int* idx, float* wt,      \
+                                       int G, int keep, int top, float scale, int has_gate, int scores,              \
+                                       const float* bias, const float* correction, int group_top, int renorm, int* idx, float* wt, \
                                        float* gate_out, void* stream) {                                              \
-    return launch_moe_route<T>(h, ldh, wr, w_f32, rows, D, E, G, keep, top, scale, has_gate, sigmoid_scores,         \
+    return launch_moe_route<T>(h, ldh, wr, w_f32, rows, D, E, G, keep, top, scale, has_gate, scores, bias,           \
                                correction, group_top, renorm, idx, wt, gate_out, (cudaStream_t)stream);              \
   }                                                                                                                  \
   KVCM_API int kvcm_moe_experts_##SUFFIX(const void* h, int ldh, const void* wgu, const void* wd, const int* idx,    \

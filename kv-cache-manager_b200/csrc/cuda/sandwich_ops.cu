@@ -4,7 +4,8 @@
 //
 //   embed_scaled    x[t] = table[id[t]] * scale (and a copy for parts that read the embedding later)
 //   norm_post_pre   x += wb * y / rms(y)   (if y);   out = T(wn * x / rms(x))   (if out; optionally of gathered rows)
-//                   -- the norm that closes one sublayer and the norm that opens the next in one pass
+//                   -- the norm that closes one sublayer and the norm that opens the next in one pass; y is a float row, the
+//                   sum of two normalised branches, or the weighted sum over a row's experts, formed in the same pass
 //   poly_norm_act   out = T(a N(z) + b N(z^2) + c N(z^3) + e), N(v) = v / rms(v) over a row, powers element-wise
 //   concat_cast     out[t] = [T(a[t]) | T(b[t])]
 //   add_bias_rows   x[t] += bias
@@ -35,53 +36,6 @@ embed_scaled_kernel(const int* __restrict__ ids, const T* __restrict__ table, fl
   }
 }
 
-// One block a row; the row's new value stays in shared memory between the two passes.
-template <typename T>
-__global__ void __launch_bounds__(256)
-norm_post_pre_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ wb,
-                     const float* __restrict__ wn, T* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
-  extern __shared__ __align__(16) float row[];
-  __shared__ float scratch[33];
-  pdl_launch_dependents();
-  pdl_wait();
-  const int r = rows ? rows[blockIdx.x] : blockIdx.x;
-  float* xr = x + size_t(r) * H;
-  if (y) {
-    const float* yr = y + size_t(r) * H;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float v = yr[i];
-      row[i] = v;
-      ss = fmaf(v, v, ss);
-    }
-    ss = block_sum(ss, scratch);
-    const float inv = 1.f / sqrtf(ss / float(H) + eps);
-    float s2 = 0.f;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float v = xr[i] + wb[i] * (row[i] * inv);
-      row[i] = v;
-      if (!rows) xr[i] = v;
-      s2 = fmaf(v, v, s2);
-    }
-    if (!out) return;
-    s2 = block_sum(s2, scratch);
-    const float inv2 = 1.f / sqrtf(s2 / float(H) + eps);
-    T* o = out + size_t(blockIdx.x) * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) stf(o + i, wn[i] * (row[i] * inv2));
-  } else {
-    float s2 = 0.f;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float v = xr[i];
-      row[i] = v;
-      s2 = fmaf(v, v, s2);
-    }
-    s2 = block_sum(s2, scratch);
-    const float inv2 = 1.f / sqrtf(s2 / float(H) + eps);
-    T* o = out + size_t(blockIdx.x) * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) stf(o + i, wn[i] * (row[i] * inv2));
-  }
-}
-
 // Four values a thread and access (H % 4 == 0 and 16-byte aligned rows); as many threads as a row has float4s, at most 512.
 __device__ __forceinline__ void st4(float* p, float a, float b, float c, float d) {
   *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
@@ -94,50 +48,136 @@ __device__ __forceinline__ void st4(bf16* p, float a, float b, float c, float d)
   *reinterpret_cast<uint2*>(p) = u;
 }
 
-template <typename T>
+// What a sublayer returned, y:
+//   kYNone     nothing is pending
+//   kYDense    one float row
+//   kYJoined   the sum of two branches, each first divided by its own root mean square: w0 * y0 / rms(y0) + w1 * y1 / rms(y1)
+//   kYExperts  the weighted sum over a row's experts, sum_k wt[row, k] y[place of (row, k)]
+enum { kYNone = 0, kYDense = 1, kYJoined = 2, kYExperts = 3 };
+struct NormPostPreParams {
+  float* x;
+  const float* y; const float* y1; const float* w0; const float* w1; float eps_join;
+  const int* place; const float* wt; int top;
+  const float* wb; const float* wn; void* out; const int* rows;
+  int H; float eps;
+};
+
+__device__ __forceinline__ void load_cols(float (&v)[4], const float* p) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void load_cols(float (&v)[1], const float* p) { v[0] = *p; }
+template <typename T> __device__ __forceinline__ void store_cols(T* p, const float (&v)[4]) { st4(p, v[0], v[1], v[2], v[3]); }
+template <typename T> __device__ __forceinline__ void store_cols(T* p, const float (&v)[1]) { stf(p, v[0]); }
+
+// Two block-wide sums at once.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if (lane == 0) scratch[warp] = make_float2(a, b);
+  __syncthreads();
+  float2 t = lane < nwarps ? scratch[lane] : make_float2(0.f, 0.f);
+  t.x = warp_sum(t.x);
+  t.y = warp_sum(t.y);
+  return t;
+}
+
+// One block a row, V neighbouring values a thread and access (V = 4: H % 4 == 0 and 16-byte aligned rows); every global
+// load of the row is asked for before the first sum, and the values wait in shared memory ([y | x], joined: [y0 | x | y1]).
+template <typename T, int V, int MODE>
 __global__ void __launch_bounds__(512)
-norm_post_pre_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ wb,
-                         const float* __restrict__ wn, T* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
+norm_post_pre_kernel(NormPostPreParams p) {
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[33];
+  __shared__ float2 scratch2[32];
   pdl_launch_dependents();
+  const int H = p.H, tid = V * threadIdx.x, step = V * blockDim.x;
+  const int r = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+  float* xs = row + H;
+  float* ys = row + 2 * H;
+  float* xr = p.x + size_t(r) * H;
   pdl_wait();
-  const int r = rows ? rows[blockIdx.x] : blockIdx.x;
-  float* xr = x + size_t(r) * H;
-  float s2 = 0.f;
-  if (y) {
-    const float* yr = y + size_t(r) * H;
-    float ss = 0.f;
-    for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
-      const float4 v = *reinterpret_cast<const float4*>(yr + i);
-      *reinterpret_cast<float4*>(row + i) = v;
-      ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+  float sa = 0.f, sb = 0.f;
+  for (int i = tid; i < H; i += step) {
+    float x[V], y[V];
+    load_cols(x, xr + i);
+    if constexpr (MODE == kYNone) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) sb = fmaf(x[e], x[e], sb);
+    } else if constexpr (MODE == kYExperts) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = 0.f;
+      for (int k = 0; k < p.top; ++k) {
+        float a[V];
+        load_cols(a, p.y + size_t(p.place[size_t(r) * p.top + k]) * H + i);
+        const float w = p.wt[size_t(r) * p.top + k];
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = fmaf(w, a[e], y[e]);
+      }
+    } else {
+      load_cols(y, p.y + size_t(r) * H + i);
     }
-    ss = block_sum(ss, scratch);
-    const float inv = 1.f / sqrtf(ss / float(H) + eps);
-    for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
-      const float4 xv = *reinterpret_cast<const float4*>(xr + i), w = *reinterpret_cast<const float4*>(wb + i);
-      float4 v = *reinterpret_cast<const float4*>(row + i);
-      v.x = xv.x + w.x * (v.x * inv); v.y = xv.y + w.y * (v.y * inv);
-      v.z = xv.z + w.z * (v.z * inv); v.w = xv.w + w.w * (v.w * inv);
-      *reinterpret_cast<float4*>(row + i) = v;
-      if (!rows) *reinterpret_cast<float4*>(xr + i) = v;
-      s2 = fmaf(v.x, v.x, s2); s2 = fmaf(v.y, v.y, s2); s2 = fmaf(v.z, v.z, s2); s2 = fmaf(v.w, v.w, s2);
+    if constexpr (MODE == kYJoined) {
+      float z[V];
+      load_cols(z, p.y1 + size_t(r) * H + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) sb = fmaf(z[e], z[e], sb);
+      store_cols(ys + i, z);
     }
-    if (!out) return;
-  } else {
-    for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
-      const float4 v = *reinterpret_cast<const float4*>(xr + i);
-      *reinterpret_cast<float4*>(row + i) = v;
-      s2 = fmaf(v.x, v.x, s2); s2 = fmaf(v.y, v.y, s2); s2 = fmaf(v.z, v.z, s2); s2 = fmaf(v.w, v.w, s2);
+    if constexpr (MODE != kYNone) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) sa = fmaf(y[e], y[e], sa);
+      store_cols(row + i, y);
     }
+    store_cols(xs + i, x);
   }
-  s2 = block_sum(s2, scratch);
-  const float inv2 = 1.f / sqrtf(s2 / float(H) + eps);
-  T* o = out + size_t(blockIdx.x) * H;
-  for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
-    const float4 v = *reinterpret_cast<const float4*>(row + i), w = *reinterpret_cast<const float4*>(wn + i);
-    st4(o + i, w.x * (v.x * inv2), w.y * (v.y * inv2), w.z * (v.z * inv2), w.w * (v.w * inv2));
+  float s2 = sb;
+  if constexpr (MODE != kYNone) {
+    if constexpr (MODE == kYJoined) {
+      const float2 t = block_sum2(sa, sb, scratch2);
+      const float i0 = 1.f / sqrtf(t.x / float(H) + p.eps_join), i1 = 1.f / sqrtf(t.y / float(H) + p.eps_join);
+      sa = 0.f;
+      for (int i = tid; i < H; i += step) {
+        float y[V], z[V], w0[V], w1[V];
+        load_cols(w0, p.w0 + i);
+        load_cols(w1, p.w1 + i);
+        load_cols(y, row + i);
+        load_cols(z, ys + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          y[e] = w0[e] * (y[e] * i0) + w1[e] * (z[e] * i1);
+          sa = fmaf(y[e], y[e], sa);
+        }
+        store_cols(row + i, y);
+      }
+    }
+    const float inv = 1.f / sqrtf(block_sum(sa, scratch) / float(H) + p.eps);
+    s2 = 0.f;
+    for (int i = tid; i < H; i += step) {
+      float x[V], y[V], w[V];
+      load_cols(w, p.wb + i);
+      load_cols(x, xs + i);
+      load_cols(y, row + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        x[e] = x[e] + w[e] * (y[e] * inv);
+        s2 = fmaf(x[e], x[e], s2);
+      }
+      store_cols(xs + i, x);
+      if (!p.rows) store_cols(xr + i, x);
+    }
+    if (!p.out) return;
+  }
+  const float inv2 = 1.f / sqrtf(block_sum(s2, scratch) / float(H) + p.eps);
+  T* o = reinterpret_cast<T*>(p.out) + size_t(blockIdx.x) * H;
+  for (int i = tid; i < H; i += step) {
+    float x[V], w[V];
+    load_cols(w, p.wn + i);
+    load_cols(x, xs + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = w[e] * (x[e] * inv2);
+    store_cols(o + i, x);
   }
 }
 
@@ -306,32 +346,47 @@ KVCM_API int kvcm_embed_scaled_bf16(KVCM_EMBED_SCALED_ARGS) {
                     keep, H, vocab, scale);
 }
 
-template <typename T>
-static int launch_norm_post_pre(float* x, const float* y, const float* wb, const float* wn, void* out, const int* rows_idx,
-                                int rows, int H, float eps, cudaStream_t s) {
-  if (rows == 0) return 0;
-  if ((y && !wb) || (out && !wn) || (!y && !out) || (rows_idx && !out)) return KVCM_ERR_UNSUPPORTED;
-  const size_t smem = size_t(H) * sizeof(float);
+template <typename T, int V, int MODE>
+static int launch_norm_post_pre_as(const NormPostPreParams& p, int rows, cudaStream_t s) {
+  const size_t smem = size_t(p.H) * (MODE == kYJoined ? 3 : 2) * sizeof(float);
   if (smem > 200 * 1024) return KVCM_ERR_UNSUPPORTED;
-  if (H % 4 == 0 && aligned16(x, y, wb, wn, out)) {
-    if (smem > 40 * 1024) {
-      const cudaError_t e = cudaFuncSetAttribute(norm_post_pre_vec_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-      if (e != cudaSuccess) return int(e);
-    }
-    return pdl_launch(norm_post_pre_vec_kernel<T>, dim3(rows), dim3(vec_threads(H)), smem, s, x, y, wb, wn, (T*)out, rows_idx, H, eps);
-  }
-  if (smem > 40 * 1024) {                               // (the kernel's static shared memory counts against the 48 KB too)
-    const cudaError_t e = cudaFuncSetAttribute(norm_post_pre_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+  static size_t configured = 0;
+  if (smem > 40 * 1024 && smem > configured) {          // (the kernel's static shared memory counts against the 48 KB too)
+    const cudaError_t e = cudaFuncSetAttribute(norm_post_pre_kernel<T, V, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     if (e != cudaSuccess) return int(e);
+    configured = smem;
   }
-  return pdl_launch(norm_post_pre_kernel<T>, dim3(rows), dim3(256), smem, s, x, y, wb, wn, (T*)out, rows_idx, H, eps);
+  return pdl_launch(norm_post_pre_kernel<T, V, MODE>, dim3(rows), dim3(V == 4 ? vec_threads(p.H) : 256), smem, s, p);
 }
-#define KVCM_NORM_POST_PRE_ARGS float *x, const float *y, const float *wb, const float *wn, void *out, const int *rows_idx, int rows, int H, float eps, void *stream
+template <typename T>
+static int launch_norm_post_pre(const NormPostPreParams& p, int rows, cudaStream_t s) {
+  if (rows == 0) return 0;
+  const bool joined = p.y1 != nullptr, experts = p.place != nullptr;
+  if ((p.y && !p.wb) || (p.out && !p.wn) || (!p.y && (!p.out || joined || experts)) || (p.rows && !p.out) || (joined && (experts || !p.w0 || !p.w1)) ||
+      (experts && (!p.wt || p.top < 1)))
+    return KVCM_ERR_UNSUPPORTED;
+  const bool vec = p.H % 4 == 0 && aligned16(p.x, p.y, p.y1, p.w0, p.w1, p.wb, p.wn) && aligned16(static_cast<const char*>(p.out));
+#define KVCM_NORM_MODE(MODE) return vec ? launch_norm_post_pre_as<T, 4, MODE>(p, rows, s) : launch_norm_post_pre_as<T, 1, MODE>(p, rows, s)
+  if (!p.y) KVCM_NORM_MODE(kYNone);
+  if (joined) KVCM_NORM_MODE(kYJoined);
+  if (experts) KVCM_NORM_MODE(kYExperts);
+  KVCM_NORM_MODE(kYDense);
+#undef KVCM_NORM_MODE
+}
+// y1 (with w0, w1, eps_join): y is the first of two branches that are normalised and summed; place, wt, top: y holds the
+// experts' outputs in the order of the sorted pairs.
+#define KVCM_NORM_POST_PRE_ARGS                                                                                           \
+  float *x, const float *y, const float *y1, const float *w0, const float *w1, float eps_join, const int *place,          \
+      const float *wt, int top, const float *wb, const float *wn, void *out, const int *rows_idx, int rows, int H, float eps, void *stream
+static NormPostPreParams norm_post_pre_params(KVCM_NORM_POST_PRE_ARGS) {
+  (void)rows; (void)stream;
+  return NormPostPreParams{x, y, y1, w0, w1, eps_join, place, wt, top, wb, wn, out, rows_idx, H, eps};
+}
 KVCM_API int kvcm_norm_post_pre_f32(KVCM_NORM_POST_PRE_ARGS) {
-  return launch_norm_post_pre<float>(x, y, wb, wn, out, rows_idx, rows, H, eps, (cudaStream_t)stream);
+  return launch_norm_post_pre<float>(norm_post_pre_params(x, y, y1, w0, w1, eps_join, place, wt, top, wb, wn, out, rows_idx, rows, H, eps, stream), rows, (cudaStream_t)stream);
 }
 KVCM_API int kvcm_norm_post_pre_bf16(KVCM_NORM_POST_PRE_ARGS) {
-  return launch_norm_post_pre<bf16>(x, y, wb, wn, out, rows_idx, rows, H, eps, (cudaStream_t)stream);
+  return launch_norm_post_pre<bf16>(norm_post_pre_params(x, y, y1, w0, w1, eps_join, place, wt, top, wb, wn, out, rows_idx, rows, H, eps, stream), rows, (cudaStream_t)stream);
 }
 
 template <typename T>

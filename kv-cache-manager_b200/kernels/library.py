@@ -483,8 +483,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
                      window: int = 0, softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
                      keep_first: int = 0, chunk: int = 0) -> None:
     """Single-row entries: q/out hold one row per request, in the order of the batch's entries.
-    ``softcap`` / ``sink`` / ``chunk`` as in ``attention_plain``; with chunks the partitions split the longest
-    part of a context that a chunk can hold (and the tile its start lies in)."""
+    ``softcap`` / ``sink`` / ``chunk`` as in ``attention_plain``; with a window or
+    chunks the partitions split the longest part of a context that one can hold (and the tile its start lies in)."""
     _cuda(q, out, k_cache, v_cache, block_tables, sink)
     _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh),
           "attention_decode: sink float32 [heads]")
@@ -494,7 +494,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
     _need(q.stride(1) == 1 and out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous(),
           "attention_decode: layout")
     _need(q.data_ptr() % 16 == 0 and (q.stride(0) * 2) % 16 == 0, "attention_decode: q rows must be 16-byte aligned")
-    span = ctx.max_decode_ctx if chunk <= 0 else min(ctx.max_decode_ctx, int(chunk) + KEY_TILE - 1)
+    reach = chunk if chunk > 0 else window
+    span = ctx.max_decode_ctx if reach <= 0 else min(ctx.max_decode_ctx, int(reach) + KEY_TILE - 1)
     size, parts = decode_partitions(S, nh, nkv, hd, span, q.device,
                                     ctx.options.get("attn_version", "auto"), int(ctx.options.get("attn_parts", 0)))
     scratch = None
@@ -583,17 +584,31 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor) -> None:
     _check(rc, "gemm_stream", f"(M={M}, N={N}, K={K})")
 
 
-def gemm_stream_relu_sq(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor) -> None:
-    """y = max(bfloat16(x @ w^T), 0)^2 in bfloat16: the streaming product of ``gemm_stream`` with the
-    activation of an ungated feed-forward in its epilogue (the same roundings as product, then ``relu_sq``)."""
+UNARY_KINDS = {"relu2": 1, "gelu_tanh": 2}        # csrc/cuda/gated_act.cuh: UnaryKind
+
+
+def gemm_stream_act(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, act: str) -> None:
+    """y = act(bfloat16(x @ w^T)) in bfloat16: the streaming product of ``gemm_stream`` with the activation of an
+    ungated feed-forward ("relu2" | "gelu_tanh") in its epilogue (the same roundings as product, then ``unary_act``)."""
     _cuda(x, w, y)
     M, K = x.shape
     N = w.shape[0]
     _need(w.shape[1] == K and y.shape == (M, N) and x.dtype == w.dtype == y.dtype == torch.bfloat16
-          and x.stride(1) == 1 and w.stride(1) == 1 and y.stride(1) == 1, "gemm_stream_relu_sq: bfloat16 [M,K] x [N,K]")
-    rc = _lib().kvcm_gemm_stream_relu_sq_bf16(_p(x), _p(w), _p(y), M, N, K, x.stride(0), w.stride(0), y.stride(0),
-                                              sm_count(x.device), _stream())
-    _check(rc, "gemm_stream", f"(M={M}, N={N}, K={K}, relu_sq)")
+          and x.stride(1) == 1 and w.stride(1) == 1 and y.stride(1) == 1, "gemm_stream_act: bfloat16 [M,K] x [N,K]")
+    rc = _lib().kvcm_gemm_stream_act_bf16(_p(x), _p(w), _p(y), M, N, K, x.stride(0), w.stride(0), y.stride(0), UNARY_KINDS[act],
+                                          sm_count(x.device), _stream())
+    _check(rc, "gemm_stream", f"(M={M}, N={N}, K={K}, {act})")
+
+
+def gemm_tcgen05_act(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, act: str) -> None:
+    """The same for many rows: the tiled tcgen05 product with the activation in its epilogue."""
+    _cuda(x, w, y)
+    M, K = x.shape
+    N = w.shape[0]
+    _need(w.shape[1] == K and y.shape == (M, N) and x.dtype == w.dtype == y.dtype == torch.bfloat16
+          and x.stride(1) == 1 and w.stride(1) == 1 and y.stride(1) == 1, "gemm_tcgen05_act: bfloat16 [M,K] x [N,K]")
+    _check(_lib().kvcm_gemm_tcgen05_act_bf16(_p(x), _p(w), _p(y), M, N, K, x.stride(0), w.stride(0), y.stride(0), UNARY_KINDS[act],
+                                             _stream()), "gemm_tcgen05", f"(M={M}, N={N}, K={K}, {act})")
 
 
 def stream_test_hooks(wait_limit_ns: int = 0, skip_stage: int = -1) -> None:
@@ -1084,17 +1099,23 @@ def latent_norm_cache(v: torch.Tensor, weight: torch.Tensor, slot_mapping: torch
 
 # ---------------------------------------------------------------------------- routed experts
 
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
+
+
 def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, groups: int, keep: int, top: int, scale: float,
               idx: torch.Tensor, wt: torch.Tensor, gate: Optional[torch.Tensor], scores: str = "softmax",
-              correction: Optional[torch.Tensor] = None, group_top: int = 1, renorm: bool = False) -> None:
-    """Per row: float32 router logits, scores (``scores``: "softmax" over all experts or "sigmoid" of each
-    logit), group-limited choice of ``top`` experts; ``idx`` int32 [T, top], ``wt`` float32 [T, top] =
+              correction: Optional[torch.Tensor] = None, group_top: int = 1, renorm: bool = False,
+              bias: Optional[torch.Tensor] = None) -> None:
+    """Per row: float32 router logits (plus ``bias``, float32 [experts]), scores (``scores``: "softmax" over all experts, "sigmoid" of
+    each logit, or "softmax_chosen": the largest logits are chosen and their softmax among themselves are the weights), group-limited choice of ``top`` experts; ``idx`` int32 [T, top], ``wt`` float32 [T, top] =
     score * scale; ``gate`` float32 [T] = sigmoid of the logit of the router matrix's extra row (row
     ``experts``).  ``correction`` (float32 [experts]) is added to the scores for the choice only;
     ``group_top``: a group's score is the sum of its 1 or 2 largest choice scores; ``renorm``: the chosen scores are
     divided by their sum (+ 1e-20) before the scale."""
     _cuda(h, router, idx, wt, gate, correction)
-    _need(scores in ("softmax", "sigmoid") and group_top in (1, 2), "moe_route: scores 'softmax' | 'sigmoid', group_top 1 | 2")
+    _need(scores in ROUTE_SCORES and group_top in (1, 2), "moe_route: scores 'softmax' | 'sigmoid' | 'softmax_chosen', group_top 1 | 2")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == experts and bias.is_cuda),
+          "moe_route: bias float32 [experts]")
     _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == experts),
           "moe_route: correction float32 [experts]")
     T, D = h.shape
@@ -1105,7 +1126,7 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, groups: int, 
     _need(gate is None or (gate.dtype == torch.float32 and gate.numel() >= T), "moe_route: gate float32 [T]")
     fn = getattr(_lib(), "kvcm_moe_route_" + _suffix(h))
     _check(fn(_p(h), h.stride(0), _p(router), int(router.dtype == torch.float32), T, D, experts, groups, keep, top,
-              ctypes.c_float(scale), int(gate is not None), int(scores == "sigmoid"), _p(correction), int(group_top),
+              ctypes.c_float(scale), int(gate is not None), ROUTE_SCORES[scores], _p(bias), _p(correction), int(group_top),
               int(bool(renorm)), _p(idx), _p(wt), _p(gate), _stream()), "moe_route",
            f"(experts={experts}, groups={groups}, keep={keep}, top={top})")
 
@@ -1187,7 +1208,7 @@ def state_scan(mode: int, qkv: torch.Tensor, bases, beta: Optional[torch.Tensor]
     _need(all(t is None or t.dtype == torch.float32 for t in (qkv, beta, g, gd, state, out)), "state_scan: float32")
     linear = mode in (SCAN_LINEAR, SCAN_LINEAR_CHANNEL)
     _need(linear or (beta is not None and not silu), "state_scan: beta")
-    _need(qkv.is_contiguous() and out.is_contiguous() and state.is_contiguous() and (beta is None or beta.stride(1) == 1)
+    _need(qkv.is_contiguous() and out.is_contiguous() and state.dim() == 2 and state.stride(1) == 1 and (beta is None or beta.stride(1) == 1)
           and (g is None or g.stride(1) == 1) and (gd is None or (gd.is_contiguous() and gd.shape == (qkv.shape[0], heads * dk))),
           "state_scan: layout")
     qb, kb, vb = (int(b) for b in bases)
@@ -1206,13 +1227,14 @@ def linear_chunk_supported(dk: int) -> bool:
 
 
 def linear_chunk(qkv: torch.Tensor, bases, decay: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int,
-                 qk_heads: int, dk: int, dv: int, silu: bool = False) -> None:
+                 qk_heads: int, dk: int, dv: int, silu: bool = False, exact: bool = False) -> None:
     """``state_scan``'s linear form with one constant decay per head (``decay`` float32 [heads]), in chunks of 64 tokens on the
     tensor cores, for the step's portions of more than one token (csrc/cuda/linear_chunk.cu); rows of single-row
-    entries are left alone.  For a 16-bit model: q, k and v are bfloat16 operands there."""
+    entries are left alone.  For a 16-bit model: v, and without ``exact`` q and k too, are bfloat16 operands there; with it
+    q and k keep 16 leading bits (they are no plain projections: rotated, scaled)."""
     _cuda(qkv, decay, state, out)
     _need(all(t.dtype == torch.float32 for t in (qkv, decay, state, out)), "linear_chunk: float32")
-    _need(qkv.is_contiguous() and out.is_contiguous() and state.is_contiguous() and decay.is_contiguous() and decay.numel() == heads,
+    _need(qkv.is_contiguous() and out.is_contiguous() and state.dim() == 2 and state.stride(1) == 1 and decay.is_contiguous() and decay.numel() == heads,
           "linear_chunk: layout")
     qb, kb, vb = (int(b) for b in bases)
     C = qkv.shape[1]
@@ -1220,10 +1242,10 @@ def linear_chunk(qkv: torch.Tensor, bases, decay: torch.Tensor, state: torch.Ten
           and state.shape[1] >= heads * dk * dv and ctx.tile_rows == 64, "linear_chunk: shapes")
     tiles = ctx.prefill_tiles
     _lib().kvcm_linear_chunk_scratch_bytes.restype = ctypes.c_longlong
-    scratch = torch.empty((int(_lib().kvcm_linear_chunk_scratch_bytes(tiles, heads, dk, dv)),), dtype=torch.uint8, device=qkv.device)
+    scratch = torch.empty((int(_lib().kvcm_linear_chunk_scratch_bytes(tiles, heads, dk, dv, int(bool(exact)))),), dtype=torch.uint8, device=qkv.device)
     _check(_lib().kvcm_linear_chunk(_p(qkv), C, qb, kb, vb, _p(decay), _p(scratch), _p(state), _ll(state.stride(0)), _p(ctx.tile_seq),
                                     _p(ctx.tile_q0), _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out), tiles,
-                                    heads, qk_heads, dk, dv, int(bool(silu)), _stream()), "linear_chunk", f"(dk={dk}, dv={dv})")
+                                    heads, qk_heads, dk, dv, int(bool(silu)), int(bool(exact)), _stream()), "linear_chunk", f"(dk={dk}, dv={dv})")
     global _launches
     _launches += 2                          # outer, carry, read
 
@@ -1305,12 +1327,12 @@ def dyt_norm(x: torch.Tensor, pending, weight: torch.Tensor, bias: torch.Tensor,
               _stream()), "dyt_norm")
 
 
-def relu_sq(x: torch.Tensor, out: torch.Tensor) -> None:
-    """out = max(x, 0)^2, elementwise, in the storage dtype."""
+def unary_act(x: torch.Tensor, out: torch.Tensor, act: str) -> None:
+    """out = act(x), elementwise, in the storage dtype: "relu2" = max(x, 0)^2, "gelu_tanh" = the tanh form of gelu."""
     _cuda(x, out)
-    _need(x.is_contiguous() and out.is_contiguous() and x.shape == out.shape and x.dtype == out.dtype, "relu_sq: layout")
-    fn = getattr(_lib(), "kvcm_relu_sq_" + _suffix(x))
-    _check(fn(_p(x), _p(out), _ll(x.numel()), _stream()), "relu_sq")
+    _need(x.is_contiguous() and out.is_contiguous() and x.shape == out.shape and x.dtype == out.dtype, "unary_act: layout")
+    fn = getattr(_lib(), "kvcm_unary_act_" + _suffix(x))
+    _check(fn(_p(x), _p(out), _ll(x.numel()), UNARY_KINDS[act], _stream()), "unary_act")
 
 
 def attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: Optional[torch.Tensor], wk: Optional[torch.Tensor],
@@ -1370,20 +1392,35 @@ def embed_scaled(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, keep: 
     _check(fn(_p(ids), _p(table), _p(x), _p(keep), T, H, table.shape[0], ctypes.c_float(scale), _stream()), "embed_scaled")
 
 
-def norm_post_pre(x: torch.Tensor, y: Optional[torch.Tensor], post_w: Optional[torch.Tensor], pre_w: Optional[torch.Tensor],
+def norm_post_pre(x: torch.Tensor, y, post_w: Optional[torch.Tensor], pre_w: Optional[torch.Tensor],
                   out: Optional[torch.Tensor], eps: float, rows: Optional[torch.Tensor] = None) -> None:
     """The norm that closes a sublayer and the norm that opens the next one, in one pass over a row:
-    x += post_w * y / rms(y) (when ``y`` is given; float32 like x), then out = pre_w * x / rms(x) (when ``out`` is
-    given; storage dtype).  Weights are the multipliers themselves, float32 [H].  ``rows`` gathers: the norms are
-    formed for rows[i] only, ``out`` has one row per index and x is left as it is."""
-    _cuda(x, y, post_w, pre_w, out, rows)
+    x += post_w * y / rms(y) (when ``y`` is given), then out = pre_w * x / rms(x) (when ``out`` is given; storage
+    dtype).  ``y`` is float32 like x, or what a sublayer left unformed and this pass forms: a parts.base.NormedSum (two
+    branches, each normalised with multipliers of its own) or a parts.base.ExpertSum (the weighted sum over a row's
+    experts).  Weights are the multipliers themselves, float32 [H].  ``rows`` gathers: the norms are formed for rows[i]
+    only, ``out`` has one row per index and x is left as it is."""
     T, H = x.shape
+    y0 = y1 = w0 = w1 = place = wt = None
+    top, eps_join = 0, 0.0
+    if hasattr(y, "place"):                             # ExpertSum
+        y0, wt, top = y.y, y.wt, y.wt.shape[1]
+        _need(y0.dtype == wt.dtype == torch.float32 and y0.is_contiguous() and wt.is_contiguous() and y0.shape == (T * top, H)
+              and wt.shape == (T, top), "norm_post_pre: the experts' outputs")
+        place = y.place()
+    elif hasattr(y, "branches"):                        # NormedSum
+        (y0, w0), (y1, w1) = y.branches
+        eps_join = y.eps
+        _need(all(t.dtype == torch.float32 and t.is_contiguous() and t.shape == x.shape for t in (y0, y1)), "norm_post_pre: branches float32 like x")
+    elif y is not None:
+        y0 = y
+        _need(y.dtype == torch.float32 and y.is_contiguous() and y.shape == x.shape, "norm_post_pre: y float32 like x")
+    _cuda(x, y0, y1, w0, w1, wt, post_w, pre_w, out, rows)
     _need(x.dtype == torch.float32 and x.is_contiguous(), "norm_post_pre: x float32 [T, H]")
-    _need(y is None or (y.dtype == torch.float32 and y.is_contiguous() and y.shape == x.shape and post_w is not None),
-          "norm_post_pre: y float32 like x, with its weight")
-    for w in (post_w, pre_w):
+    _need(y0 is None or post_w is not None, "norm_post_pre: y comes with its weight")
+    for w in (post_w, pre_w, w0, w1):
         _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == H), "norm_post_pre: weights float32 [H]")
-    _need(out is not None or y is not None, "norm_post_pre: nothing to do")
+    _need(out is not None or y0 is not None, "norm_post_pre: nothing to do")
     _need(out is None or (out.is_contiguous() and out.shape[1] == H and pre_w is not None), "norm_post_pre: out")
     n = T
     if rows is not None:
@@ -1393,8 +1430,8 @@ def norm_post_pre(x: torch.Tensor, y: Optional[torch.Tensor], post_w: Optional[t
         _need(out.shape[0] == T, "norm_post_pre: out rows != x rows")
     store = out.dtype if out is not None else torch.float32
     fn = getattr(_lib(), "kvcm_norm_post_pre_" + _SUFFIX[store])
-    _check(fn(_p(x), _p(y), _p(post_w), _p(pre_w), _p(out), _p(rows), n, H, ctypes.c_float(eps), _stream()), "norm_post_pre",
-           f"(hidden={H})")
+    _check(fn(_p(x), _p(y0), _p(y1), _p(w0), _p(w1), ctypes.c_float(eps_join), place, _p(wt), top, _p(post_w), _p(pre_w), _p(out),
+              _p(rows), n, H, ctypes.c_float(eps), _stream()), "norm_post_pre", f"(hidden={H})")
 
 
 def poly_norm_act(z: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, eps: float) -> None:
@@ -1609,7 +1646,7 @@ def norm_pair(x: torch.Tensor, pending, experts, w1: torch.Tensor, eps1: float, 
         _need(e.y.dtype == e.wt.dtype == torch.float32 and e.y.is_contiguous() and e.wt.is_contiguous() and e.y.shape == (T * top, D)
               and e.wt.shape == (T, top) and e.work.dtype == _I32, "norm_pair: the experts' outputs")
         ey, wt = _p(e.y), _p(e.wt)
-        place = ctypes.c_void_p(e.work.data_ptr() + 4 * (e.experts + 2 + T * top))      # as the experts' sort leaves it
+        place = e.place()
     pend += [(None, 0.0)] * (3 - len(pend))
     rs, qs, ql, sl = (ctx.row_seq, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_state_slot) if shift is not None else (None,) * 4
     fn = getattr(_lib(), "kvcm_norm_pair_" + _suffix(out1))
@@ -1617,3 +1654,161 @@ def norm_pair(x: torch.Tensor, pending, experts, w1: torch.Tensor, eps1: float, 
               _p(pend[2][0]), ctypes.c_float(pend[2][1]), ey, place, wt, top, _p(w1), ctypes.c_float(eps1), _p(out1), _p(w2),
               ctypes.c_float(eps2), _p(out2), _p(shift), _p(state), _ll(state.stride(0) if state is not None else 0), _p(rs), _p(qs),
               _p(ql), _p(sl), _p(rows), n, D, _stream()), "norm_pair", f"(width={D})")
+
+
+# ---------------------------------------------------- heads in front of and behind mixers, several mixers a launch
+
+class _HeadSegment(ctypes.Structure):
+    _fields_ = [("out", ctypes.c_void_p), ("ld", ctypes.c_longlong), ("units", ctypes.c_int), ("dim", ctypes.c_int), ("HD", ctypes.c_int),
+                ("src", ctypes.c_int), ("conv", ctypes.c_int), ("table", ctypes.c_int), ("interleaved", ctypes.c_int),
+                ("dest", ctypes.c_int), ("scale", ctypes.c_float), ("items", ctypes.c_int)]
+
+
+_HEAD_SEGMENTS, _GATE_SEGMENTS = 6, 4
+
+
+class _HeadPrepareParams(ctypes.Structure):
+    _fields_ = [("proj", ctypes.c_void_p), ("ldp", ctypes.c_longlong), ("positions", ctypes.c_void_p), ("inv_freq", ctypes.c_void_p * 2),
+                ("half", ctypes.c_int * 2), ("amplitude", ctypes.c_float * 2), ("conv_w", ctypes.c_void_p), ("state", ctypes.c_void_p),
+                ("state_stride", ctypes.c_longlong), ("taps", ctypes.c_int), ("channels", ctypes.c_int), ("conv_col", ctypes.c_int),
+                ("write_state", ctypes.c_int), ("row_seq", ctypes.c_void_p), ("seq_q_start", ctypes.c_void_p), ("seq_q_len", ctypes.c_void_p),
+                ("seq_state_slot", ctypes.c_void_p), ("slot_mapping", ctypes.c_void_p), ("block_size", ctypes.c_int), ("rows", ctypes.c_int),
+                ("seqs", ctypes.c_int), ("segments", ctypes.c_int), ("items", ctypes.c_int), ("seg", _HeadSegment * _HEAD_SEGMENTS)]
+
+
+class _GateSegment(ctypes.Structure):
+    _fields_ = [("x", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldx", ctypes.c_longlong), ("ldo", ctypes.c_longlong),
+                ("x_float", ctypes.c_int), ("heads", ctypes.c_int), ("dv", ctypes.c_int), ("HD", ctypes.c_int), ("gate", ctypes.c_int),
+                ("norm", ctypes.c_int), ("silu", ctypes.c_int), ("eps", ctypes.c_float)]
+
+
+class _HeadGateParams(ctypes.Structure):
+    _fields_ = [("gates", ctypes.c_void_p), ("ldg", ctypes.c_longlong), ("rows", ctypes.c_int),
+                ("segments", ctypes.c_int), ("heads", ctypes.c_int), ("vec", ctypes.c_int), ("seg", _GateSegment * _GATE_SEGMENTS)]
+
+
+def head_layouts_match() -> bool:
+    """The parameter blocks above are laid out as the library's."""
+    lib = _lib()
+    return (int(lib.kvcm_head_prepare_params_bytes()) == ctypes.sizeof(_HeadPrepareParams)
+            and int(lib.kvcm_head_gate_params_bytes()) == ctypes.sizeof(_HeadGateParams))
+
+
+class HeadSegment:
+    """``units`` neighbouring heads of ``dim`` elements, the first at column ``src`` of the projection, and what becomes of
+    them: ``conv`` (first channel of the step's short convolution), rotation by ``inv_freq`` (float32 [pairs]; None: none) with
+    ``amplitude`` and the pairing, ``scale``, and where they go: ``dest`` "rows" (out [T, units * HD] in the storage dtype,
+    padded with zeros), "pages" (out [pages, units, page, HD]) or "float" (out float32 rows, column of the first head
+    ``out_col``; may be the projection itself)."""
+    __slots__ = ("units", "dim", "src", "conv", "inv_freq", "amplitude", "interleaved", "scale", "dest", "out", "out_col")
+
+    def __init__(self, units: int, dim: int, src: int, dest: str, out: torch.Tensor, conv: Optional[int] = None,
+                 inv_freq: Optional[torch.Tensor] = None, amplitude: float = 1.0, interleaved: bool = False, scale: float = 1.0,
+                 out_col: int = 0) -> None:
+        self.units, self.dim, self.src, self.dest, self.out, self.conv = units, dim, src, dest, out, conv
+        self.inv_freq, self.amplitude, self.interleaved, self.scale, self.out_col = inv_freq, amplitude, interleaved, scale, out_col
+
+
+class HeadConv:
+    """The short convolution of a ``prepare_heads`` launch: ``weight`` float32 [channels, taps] over the projection's columns
+    from ``col`` on; ``state`` float32 [slots, >= (taps - 1) * channels] (row stride free)."""
+    __slots__ = ("weight", "state", "col")
+
+    def __init__(self, weight: torch.Tensor, state: Optional[torch.Tensor], col: int) -> None:
+        self.weight, self.state, self.col = weight, state, col
+
+
+def prepare_heads(proj: torch.Tensor, segments, ctx, dtype: torch.dtype, conv: Optional[HeadConv] = None,
+                  slot_mapping: Optional[torch.Tensor] = None, block_size: int = 1) -> None:
+    """What lies between a step's float32 projection [T, columns] and the kernels of one or several mixers, for all their
+    heads in one launch (csrc/cuda/head_prepare.cu): short convolution from and into the requests' state, rotation,
+    scale, and the store in rows, page slots or float rows."""
+    T, W = proj.shape
+    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.is_cuda, "prepare_heads: proj float32 [T, columns]")
+    _need(1 <= len(segments) <= _HEAD_SEGMENTS, "prepare_heads: one to six segments")
+    p = _HeadPrepareParams()
+    p.proj, p.ldp, p.positions = proj.data_ptr(), proj.stride(0), ctx.positions.data_ptr()
+    p.rows, p.seqs, p.segments, p.block_size = T, ctx.seqs, len(segments), int(block_size)
+    p.row_seq, p.seq_q_start, p.seq_q_len = ctx.row_seq.data_ptr(), ctx.seq_q_start.data_ptr(), ctx.seq_q_len.data_ptr()
+    p.seq_state_slot = ctx.seq_state_slot.data_ptr()
+    p.amplitude[0] = p.amplitude[1] = 1.0
+    if slot_mapping is not None:
+        _need(slot_mapping.dtype == _I32 and slot_mapping.numel() >= T and slot_mapping.is_cuda, "prepare_heads: slot_mapping int32 [T]")
+        p.slot_mapping = slot_mapping.data_ptr()
+    channels = 0
+    if conv is not None:
+        channels, taps = conv.weight.shape
+        _need(conv.weight.dtype == torch.float32 and conv.weight.is_contiguous() and conv.weight.is_cuda and 0 <= conv.col and conv.col + channels <= W,
+              "prepare_heads: convolution float32 [channels, taps] over the projection's columns")
+        p.conv_w, p.taps, p.channels, p.conv_col = conv.weight.data_ptr(), taps, channels, conv.col
+        if taps > 1:
+            _need(conv.state is not None and conv.state.dtype == torch.float32 and conv.state.dim() == 2 and conv.state.stride(1) == 1
+                  and conv.state.shape[1] >= (taps - 1) * channels and conv.state.is_cuda, "prepare_heads: state rows too short")
+            p.state, p.state_stride = conv.state.data_ptr(), conv.state.stride(0)
+    tables: list = []
+    for i, g in enumerate(segments):
+        s = p.seg[i]
+        s.units, s.dim, s.src, s.scale, s.interleaved = g.units, g.dim, g.src, g.scale, int(bool(g.interleaved))
+        s.conv = -1 if g.conv is None else g.conv
+        _need(g.src >= 0 and g.src + g.units * g.dim <= W and g.out.is_cuda, "prepare_heads: columns of a segment")
+        _need(g.conv is None or (conv is not None and 0 <= g.conv and g.conv + g.units * g.dim <= channels and g.src == conv.col + g.conv),
+              "prepare_heads: convolved columns and channels go together")
+        s.table = -1
+        if g.inv_freq is not None:
+            _need(g.inv_freq.dtype == torch.float32 and g.inv_freq.is_contiguous() and g.inv_freq.is_cuda and 2 * g.inv_freq.numel() <= g.dim,
+                  "prepare_heads: inv_freq float32, at most half a head")
+            key = (g.inv_freq.data_ptr(), g.inv_freq.numel(), g.amplitude)
+            if key not in tables:
+                tables.append(key)
+                _need(len(tables) <= 2, "prepare_heads: at most two rotations")
+                t = len(tables) - 1
+                p.inv_freq[t], p.half[t], p.amplitude[t] = key
+            s.table = tables.index(key)
+        if g.dest == "pages":
+            _need(slot_mapping is not None and g.out.dtype == dtype and g.out.is_contiguous() and g.out.dim() == 4 and g.out.shape[1] == g.units
+                  and g.out.shape[2] == block_size and g.out.shape[3] >= g.dim, "prepare_heads: pages [pages, heads, page, HD]")
+            s.dest, s.HD, s.ld, s.out = 1, g.out.shape[3], 0, g.out.data_ptr()
+        elif g.dest == "rows":
+            _need(g.out.dtype == dtype and g.out.stride(1) == 1 and g.out.shape[0] == T and g.out.shape[1] % g.units == 0
+                  and g.out.shape[1] // g.units >= g.dim, "prepare_heads: rows [T, heads * HD]")
+            s.dest, s.HD, s.ld, s.out = 0, g.out.shape[1] // g.units, g.out.stride(0), g.out.data_ptr()
+        else:
+            _need(g.dest == "float" and g.out.dtype == torch.float32 and g.out.stride(1) == 1 and g.out.shape[0] == T
+                  and g.out_col + g.units * g.dim <= g.out.shape[1] and (g.conv is None or g.out.data_ptr() != proj.data_ptr()),
+                  "prepare_heads: float rows")
+            s.dest, s.HD, s.ld, s.out = 2, g.dim, g.out.stride(0), g.out.data_ptr() + 4 * g.out_col
+    fn = getattr(_lib(), "kvcm_head_prepare_" + _SUFFIX[dtype])
+    _check(fn(ctypes.byref(p), _stream()), "head_prepare", f"(segments={len(segments)})")
+    if conv is not None and p.taps > 1 and T != ctx.seqs:
+        global _launches
+        _launches += 1                      # the state update (a launch of its own unless every request brings one row)
+
+
+class GateSegment:
+    """``heads`` heads of ``dv`` elements on their way to an output product: ``x`` [T, heads * HD] (a recurrence's float32 rows or
+    the attention kernel's padded heads), the first gate column, whether each head is divided by its root mean square (``norm``: the
+    epsilon under its root, or None), the gate's activation ("sigmoid" | "silu"), and ``out`` [T, heads * dv] in the storage dtype."""
+    __slots__ = ("x", "out", "heads", "dv", "gate", "norm", "act")
+
+    def __init__(self, x: torch.Tensor, out: torch.Tensor, heads: int, dv: int, gate: int, norm: Optional[float], act: str) -> None:
+        self.x, self.out, self.heads, self.dv, self.gate, self.norm, self.act = x, out, heads, dv, gate, norm, act
+
+
+def gate_heads(gates: torch.Tensor, segments) -> None:
+    """out = x [/ rms of its head] * act(gate) for all heads of one or several mixers in one launch; ``gates`` are the float32
+    projection's rows (csrc/cuda/head_prepare.cu)."""
+    T, W = gates.shape
+    _need(gates.dtype == torch.float32 and gates.stride(1) == 1 and gates.is_cuda and 1 <= len(segments) <= _GATE_SEGMENTS, "gate_heads: gates float32")
+    p = _HeadGateParams()
+    p.gates, p.ldg, p.rows, p.segments = gates.data_ptr(), gates.stride(0), T, len(segments)
+    store = segments[0].out.dtype
+    for i, g in enumerate(segments):
+        s = p.seg[i]
+        _need(g.x.is_cuda and g.out.is_cuda and g.x.dtype in (torch.float32, store) and g.out.dtype == store and g.x.stride(1) == 1 and g.out.stride(1) == 1
+              and g.x.shape[0] == T and g.out.shape == (T, g.heads * g.dv) and g.x.shape[1] % g.heads == 0 and g.x.shape[1] >= g.heads * g.dv
+              and 0 <= g.gate and g.gate + g.heads * g.dv <= W and g.act in ("sigmoid", "silu"), "gate_heads: layout")
+        s.x, s.out, s.ldx, s.ldo = g.x.data_ptr(), g.out.data_ptr(), g.x.stride(0), g.out.stride(0)
+        s.x_float, s.heads, s.dv, s.HD = int(g.x.dtype == torch.float32), g.heads, g.dv, g.x.shape[1] // g.heads
+        s.gate, s.norm, s.silu, s.eps = g.gate, int(g.norm is not None), int(g.act == "silu"), g.norm or 0.0
+    fn = getattr(_lib(), "kvcm_head_gate_" + _SUFFIX[store])
+    _check(fn(ctypes.byref(p), _stream()), "head_gate", f"(segments={len(segments)})")

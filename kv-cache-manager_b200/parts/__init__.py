@@ -6,11 +6,13 @@ from .linear import Linear, matmul_nt
 from .norm import DynamicTanh, Float32RMSNorm, OffsetRMSNorm, OutputRMSNorm, RMSNorm
 from .rope import NoPositionEncoding, RotaryEmbedding
 from .attention import GeneralAttention, PagedAttention
-from .delta import ChannelDecayDeltaMixer, GatedDeltaMixer, SideBySideMixer
+from .delta import ChannelDecayDeltaMixer, GatedDeltaMixer
+from .side_by_side import SideBySideMixer
 from .ssm import Mamba2Mixer
 from .latent_attention import LatentAttention, LatentRopeAttention
 from .gla import GatedLinearAttention
 from .lightning import LightningAttention
+from .retention import Retention
 from .loop import LoopEntry
 from .mlp import DenseMLP, GatedMLP
 from .moe import RoutedExperts
@@ -26,5 +28,5 @@ __all__ = [
     "LatentAttention", "RoutedExperts", "DynamicTanh", "GeneralAttention", "ChannelDecayDeltaMixer",
     "SideBySideMixer", "Mamba2Mixer", "DenseMLP", "ParallelBlock", "StreamPart", "OffsetRMSNorm", "LatentRopeAttention",
     "GatedLinearAttention", "LoopEntry", "ScaledEmbedding", "SandwichBlock",
-    "Float32RMSNorm", "LightningAttention", "ParallelNormsBlock",
+    "Float32RMSNorm", "LightningAttention", "ParallelNormsBlock", "Retention",
 ]

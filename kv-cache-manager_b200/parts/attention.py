@@ -15,7 +15,7 @@ from typing import Optional
 import torch
 
 from ..kernels import library as K
-from .base import CacheSpec, MIXERS, Mixer, PositionEncoding, SiteCache, StepContext
+from .base import CacheSpec, MIXERS, Mixer, PositionEncoding, SiteCache, StagedWork, StateSpec, StepContext
 from .linear import Linear, matmul_nt
 
 
@@ -101,6 +101,10 @@ class GeneralAttention(Mixer):
       dv (no weight) before it is cached;
     * ``chunk``: row i sees keys j <= i with j // chunk == i // chunk only (its page group gives passed chunks back);
     * ``gate``: the concatenated heads multiplied element by element by sigmoid(W_g h), in front of the output product;
+    * ``taps`` > 0: q, k and v pass a short causal convolution over time, channel by channel (weight ``conv`` [q|k|v channels,
+      taps], no bias, no activation), between projection and rotation; the last taps - 1 projected values of a request are
+      its state.  Such a mixer is a staged one (see ``parts.base.Mixer``), has a gate and goes without the options that
+      change q, k or v in other ways;
     * ``head_norm``: q and k of every head scaled to unit root mean square (no weights), after the
       rotation;
     * ``softcap``: score <- cap * tanh(score / cap) after the scale;
@@ -108,7 +112,8 @@ class GeneralAttention(Mixer):
       (j <= i), at its true position.  Such a mixer asks for pages that are never given back: the cache
       manager's windows release pages from the front, where the kept keys lie;
     * ``sink``: a learned number per head whose exponential joins the softmax's denominator (no key, no
-      value, not scaled, not capped);
+      value, not scaled, not capped); ``sink_score`` is the same with one fixed number for every head (0: the denominator
+      is 1 + sum exp(score));
     * ``value_mix``: "source" leaves this layer's values (as projected) in ``ctx.shared[mix_key]`` for later
       layers of the same step; "mix" replaces v by v + lambda (v_source - v) before it is cached.
 
@@ -120,7 +125,7 @@ class GeneralAttention(Mixer):
                  sink: bool = False, bias: bool = False, proj_norm: bool = False, head_norm: bool = False,
                  norm_eps: float = 1e-6, value_mix: Optional[str] = None, mix_key: str = "v_first",
                  rotate_values: bool = False, keep_first: int = 0, qk_norm: bool = False, value_norm: bool = False,
-                 chunk: int = 0, gate: bool = False) -> None:
+                 chunk: int = 0, gate: bool = False, taps: int = 0, sink_score: Optional[float] = None) -> None:
         super().__init__()
         if num_kv_heads < 1 or num_heads % num_kv_heads:
             raise ValueError(f"attention: {num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
@@ -139,6 +144,13 @@ class GeneralAttention(Mixer):
         if self.chunk > 0 and self.keep_first > 0:
             raise ValueError("attention_general: chunks do not keep first keys")
         self._v_inv_freq = None
+        self.taps = int(taps or 0)
+        self.staged = bool(gate) and not (bias or proj_norm or head_norm or value_mix or rotate_values or qk_norm or value_norm)
+        if self.taps > 0 and not self.staged:
+            raise ValueError("attention_general: the convolution goes with a gate and without biases, norms, value mixing and turned values")
+        if sink and sink_score is not None:
+            raise ValueError("attention_general: the sink is either learned or fixed")
+        self.sink_score = None if sink_score is None else float(sink_score)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(dk)
         self.has_sink, self.has_bias, self.proj_norm, self.head_norm = bool(sink), bool(bias), bool(proj_norm), bool(head_norm)
         self.norm_eps, self.value_mix, self.mix_key = float(norm_eps), value_mix, mix_key
@@ -159,8 +171,19 @@ class GeneralAttention(Mixer):
             self.declare("sink", (num_heads,), ("normal", 1.0), "vector")
         if value_mix is not None:
             self.declare("vmix", (), ("normal", 0.3), "vector")       # read by "mix" layers only
+        if self.taps:
+            self.declare("conv", (nq + nk + nv, self.taps), ("normal", 0.5), "vector")
         self._f32 = {}
-        self._o_weight = None
+        self._o_weight = self._sink = None
+
+    @property
+    def projection(self) -> Linear:
+        return self.qkv
+
+    def state_spec(self) -> Optional[StateSpec]:
+        if self.taps < 2:
+            return None
+        return StateSpec(((self.taps - 1) * ((self.nh + self.nkv) * self.dk + self.nkv * self.dv),), torch.float32)
 
     def cache_spec(self) -> CacheSpec:
         return CacheSpec(self.nkv, self.hd, 0 if self.keep_first > 0 else self.window, chunk=self.chunk)
@@ -169,6 +192,11 @@ class GeneralAttention(Mixer):
         super().prepare(device, dtype)
         self._f32 = {n: self.param(n).to(device=device, dtype=torch.float32).reshape(-1).contiguous()
                      for n in self.param_specs()}
+        if self.taps:
+            self._f32["conv"] = self._f32["conv"].view(-1, self.taps)
+        self._sink = self._f32.get("sink")
+        if self.sink_score is not None:
+            self._sink = torch.full((self.nh,), self.sink_score, dtype=torch.float32, device=device)
         if self.rotate_values:
             m = torch.arange(self.dv // 2, dtype=torch.float64)
             self._v_inv_freq = (1.0 / torch.pow(torch.tensor(self.position.theta, dtype=torch.float64),
@@ -180,7 +208,35 @@ class GeneralAttention(Mixer):
             w = wide.view(self.hidden, self.nh * self.hd)
         self._o_weight = w
 
+    def begin(self, proj: torch.Tensor, base: int, dtype: torch.dtype, ctx: StepContext, site: SiteCache) -> StagedWork:
+        work, pos, g = StagedWork(proj, base, dtype, ctx, site), self.position, ctx.groups[site.group]
+        nq, nk = self.nh * self.dk, self.nkv * self.dk
+        work.q = torch.empty((proj.shape[0], self.nh * self.hd), dtype=dtype, device=proj.device)
+        at = (0, nq, nq + nk) if self.taps else (None, None, None)
+        turn = dict(inv_freq=pos.inv_freq, amplitude=pos.amplitude, interleaved=pos.interleaved)
+        work.segments.append(K.HeadSegment(self.nh, self.dk, base, "rows", work.q, conv=at[0], **turn))
+        if site.writes:
+            work.slot_mapping, work.block_size = g.slot_mapping, g.block_size
+            work.segments += [K.HeadSegment(self.nkv, self.dk, base + nq, "pages", site.k, conv=at[1], **turn),
+                              K.HeadSegment(self.nkv, self.dv, base + nq + nk, "pages", site.v, conv=at[2])]
+        if self.taps:
+            work.conv = K.HeadConv(self._f32["conv"], site.state, base)
+        return work
+
+    def mix(self, work: StagedWork) -> K.GateSegment:
+        T, g, site = work.proj.shape[0], work.ctx.groups[work.site.group], work.site
+        o = torch.empty((T, self.nh * self.hd), dtype=work.dtype, device=work.proj.device)
+        K.paged_attention(work.q, o, site.k, site.v, g.block_tables, work.ctx, self.nh, self.nkv, self.hd, self.scale, self.window,
+                          self.softcap, self._sink, self.keep_first, self.chunk)
+        work.out = torch.empty((T, self.nh * self.dv), dtype=work.dtype, device=work.proj.device)
+        return K.GateSegment(o, work.out, self.nh, self.dv, work.base + self.qkv.out_features - self.nh * self.dv, None, "sigmoid")
+
+    def finish(self, work: StagedWork) -> torch.Tensor:
+        return matmul_nt(work.out, self._o_weight, torch.float32, work.ctx.options)
+
     def forward(self, h: torch.Tensor, ctx: StepContext, site: SiteCache) -> torch.Tensor:
+        if self.taps:
+            return self.forward_staged(h, ctx, site)
         g = ctx.groups[site.group]
         pos, f = self.position, self._f32
         T = h.shape[0]
@@ -199,7 +255,7 @@ class GeneralAttention(Mixer):
                        amplitude=getattr(pos, "amplitude", 1.0))
         out = torch.empty((T, self.nh * self.hd), dtype=h.dtype, device=h.device)
         K.paged_attention(q, out, site.k, site.v, g.block_tables, ctx, self.nh, self.nkv, self.hd, self.scale,
-                          self.window, self.softcap, f.get("sink"), self.keep_first, self.chunk)
+                          self.window, self.softcap, self._sink, self.keep_first, self.chunk)
         if self.rotate_values:
             K.rotate_heads(out, ctx.positions, self._v_inv_freq, self.nh, self.hd, bool(getattr(pos, "interleaved", False)), -1.0)
         if self.has_gate:

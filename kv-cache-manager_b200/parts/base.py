@@ -20,6 +20,7 @@ Interfaces
 """
 from __future__ import annotations
 
+import ctypes
 from dataclasses import dataclass, field
 from typing import Any, Callable, Dict, List, Optional, Sequence, Tuple
 
@@ -225,6 +226,25 @@ BLOCKS = Registry("block")
 
 
 class Mixer(Part):
+    """``forward(h, ctx, site)`` does the whole of it.  A mixer whose work falls into the stages below sets ``staged``: two
+    such mixers that read the same rows can share the launches of the first, second and fourth (``side_by_side``), and
+    ``forward_staged`` is the mixer alone.
+
+        projection        the ``Linear`` whose float32 rows hold all it needs of h
+        begin(proj, base, dtype, ctx, site) -> work     ``work.segments`` (``kernels.library.HeadSegment``s, columns from ``base``
+                          on), ``work.conv`` (a ``HeadConv`` or None): what one ``prepare_heads`` launch has to do
+        mix(work)         -> ``kernels.library.GateSegment``: attention or recurrence; what a ``gate_heads`` launch has to do
+        finish(work)      -> the output product of the gated heads, float32"""
+    staged = False
+
+    def forward_staged(self, h: torch.Tensor, ctx: StepContext, site: SiteCache) -> torch.Tensor:
+        from ..kernels import library as K
+        proj = self.projection.forward(h, ctx, out_dtype=torch.float32)
+        work = self.begin(proj, 0, h.dtype, ctx, site)
+        run_prepare(proj, [work], h.dtype, ctx)
+        K.gate_heads(proj, [self.mix(work)])
+        return self.finish(work)
+
     def cache_spec(self) -> Optional[CacheSpec]:
         return None
 
@@ -233,6 +253,27 @@ class Mixer(Part):
 
     def forward(self, h: torch.Tensor, ctx: StepContext, site: SiteCache) -> torch.Tensor:
         raise NotImplementedError
+
+
+class StagedWork:
+    """What a staged mixer keeps of one call (see ``Mixer``); ``block_size`` and ``slot_mapping`` are those of its page group."""
+
+    def __init__(self, proj: torch.Tensor, base: int, dtype: torch.dtype, ctx: StepContext, site: SiteCache) -> None:
+        self.proj, self.base, self.dtype, self.ctx, self.site = proj, base, dtype, ctx, site
+        self.segments: List[Any] = []
+        self.conv: Any = None
+        self.slot_mapping: Optional[torch.Tensor] = None
+        self.block_size = 1
+        self.out: Optional[torch.Tensor] = None          # the gated heads
+
+
+def run_prepare(proj: torch.Tensor, works, dtype: torch.dtype, ctx: StepContext) -> None:
+    """One ``prepare_heads`` launch for the given mixers (at most one of them convolves, at most one writes pages)."""
+    from ..kernels import library as K
+    conv = next((w.conv for w in works if w.conv is not None), None)
+    paged = next((w for w in works if w.slot_mapping is not None), None)
+    K.prepare_heads(proj, [s for w in works for s in w.segments], ctx, dtype, conv, paged.slot_mapping if paged else None,
+                    paged.block_size if paged else 1)
 
 
 class FeedForward(Part):
@@ -251,13 +292,30 @@ class PositionEncoding(Part):
 
 
 class ClosingNorm:
-    """A sublayer's float32 output ``y`` that is still to be added to the stream through an RMS norm:
-    x += multiplier * y / sqrt(mean(y^2) + eps).  A block may hand this on as its pending value so that the
+    """A sublayer's float32 output ``y`` (or a ``NormedSum`` / ``ExpertSum`` that is still to be formed) that is to be added
+    to the stream through an RMS norm: x += multiplier * y / sqrt(mean(y^2) + eps).  A block may hand this on as its pending value so that the
     reader of the stream applies it in the same kernel as its own opening norm."""
     __slots__ = ("y", "multiplier", "eps")
 
     def __init__(self, y: torch.Tensor, multiplier: torch.Tensor, eps: float) -> None:
         self.y, self.multiplier, self.eps = y, multiplier, float(eps)
+
+
+class NormedSum:
+    """A mixer's output made of two branches before its sum: sum of multiplier * y / sqrt(mean(y^2) + eps) over
+    ``branches``, two (float32 [rows, width], float32 multiplier [width]) pairs.  The kernel that applies the norm behind
+    the mixer forms the sum in the same pass; ``formed`` forms it by itself."""
+    __slots__ = ("branches", "eps")
+
+    def __init__(self, branches, eps: float) -> None:
+        self.branches, self.eps = tuple(branches), float(eps)
+
+    def formed(self) -> torch.Tensor:
+        from ..kernels import library as K
+        out = torch.zeros_like(self.branches[0][0])
+        for y, multiplier in self.branches:
+            K.norm_post_pre(out, y, multiplier, None, None, self.eps)
+        return out
 
 
 class ExpertSum:
@@ -268,6 +326,10 @@ class ExpertSum:
 
     def __init__(self, y: torch.Tensor, work: torch.Tensor, wt: torch.Tensor, experts: int) -> None:
         self.y, self.work, self.wt, self.experts = y, work, wt, int(experts)
+
+    def place(self) -> ctypes.c_void_p:
+        """Where every (row, choice) pair's row of ``y`` is listed, as the experts' sort leaves it."""
+        return ctypes.c_void_p(self.work.data_ptr() + 4 * (self.experts + 2 + self.wt.numel()))
 
     def combined(self) -> torch.Tensor:
         from ..kernels import library as K

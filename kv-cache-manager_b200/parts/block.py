@@ -10,7 +10,7 @@ from typing import Optional
 import torch
 
 from ..kernels import library as K
-from .base import (BLOCKS, Block, ClosingNorm, ExpertSum, FeedForward, Mixer, Norm, SiteCache, StateSpec, StepContext, settle,
+from .base import (BLOCKS, Block, ClosingNorm, ExpertSum, FeedForward, Mixer, Norm, NormedSum, SiteCache, StateSpec, StepContext, settle,
                    split_pending)
 
 
@@ -149,11 +149,13 @@ class ParallelNormsBlock(Block):
 @BLOCKS.register("sandwich")
 class SandwichBlock(Block):
     """Every sublayer normalised on both sides: x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))).  The four
-    norms expose ``multiplier`` (float32 [hidden]) and ``eps`` ("rmsnorm_offset").  The sublayers return float32; the
+    norms expose ``multiplier`` (float32 [hidden]) and ``eps`` ("rmsnorm_offset", "rmsnorm_f32").  The sublayers return float32; the
     norm that closes one sublayer and the norm that opens the next are one kernel, also across layers: the
     closing norm of a layer's last sublayer is handed on as a ``ClosingNorm`` and applied by whatever reads the
     stream next (the next sandwich block's opening norm, the final norm, or a part between layers through
-    ``settle``).  ``fuse`` off: every norm is a launch of its own and the stream is complete when the layer ends.
+    ``settle``).  A mixer may return its branches unsummed (``NormedSum``) and a routed feed-forward its experts
+    (``ExpertSum``): the closing norm's kernel forms those too.  ``fuse`` off: every norm is a launch of its own, sums are
+    formed where they arise, and the stream is complete when the layer ends.
     ``ffn`` may be None: a layer of a mixer only."""
 
     def __init__(self, norm1: Norm, mixer: Mixer, norm1b: Norm, norm2: Optional[Norm] = None,
@@ -177,6 +179,8 @@ class SandwichBlock(Block):
             settle(x, pending)
             K.norm_post_pre(x, None, None, self.norm1.multiplier, h, self.norm1.eps)
         y = self.mixer.forward(h, ctx, site)
+        if isinstance(y, NormedSum) and not fuse:
+            y = y.formed()
         if self.ffn is None:
             return self._close(x, y, self.norm1b, fuse)
         if fuse and self.norm1b.eps == self.norm2.eps:
@@ -184,7 +188,8 @@ class SandwichBlock(Block):
         else:
             K.norm_post_pre(x, y, self.norm1b.multiplier, None, None, self.norm1b.eps)
             K.norm_post_pre(x, None, None, self.norm2.multiplier, h, self.norm2.eps)
-        y = self.ffn.forward(h, ctx, out_dtype=torch.float32)
+        deferred = getattr(self.ffn, "forward_unsummed", None) if fuse else None
+        y = deferred(h, ctx) if deferred is not None else self.ffn.forward(h, ctx, out_dtype=torch.float32)
         return self._close(x, y, self.norm2b, fuse)
 
     @staticmethod

@@ -155,33 +155,3 @@ class ChannelDecayDeltaMixer(Mixer):
         gated = torch.empty((T, H * self.dv), dtype=h.dtype, device=h.device)
         K.group_rms_gate(o, gate, self._f32["norm"], gated, self.dv, self.norm_eps, False, "sigmoid")
         return self.o.forward(gated, ctx, out_dtype=torch.float32)
-
-
-@MIXERS.register("side_by_side")
-class SideBySideMixer(Mixer):
-    """Two mixers that read the same input; the result is left_scale * left + right_scale * right.  At most
-    one of them may keep paged keys and values and at most one fixed-size state (they share the call site).
-    The sum is not formed here: the two float32 outputs are returned as (tensor, scale) pairs for the
-    block to hand to the next norm kernel, which adds them into the stream."""
-
-    def __init__(self, left: Mixer, right: Mixer, left_scale: float = 1.0, right_scale: float = 1.0) -> None:
-        super().__init__()
-        self.left, self.right = self.add_child("left", left), self.add_child("right", right)
-        self.left_scale, self.right_scale = float(left_scale), float(right_scale)
-        specs = [m.cache_spec() for m in (left, right)]
-        states = [m.state_spec() for m in (left, right)]
-        if all(s is not None for s in specs) or all(s is not None for s in states):
-            raise ValueError("side_by_side: both mixers want the call site's cache (or its state)")
-
-    def cache_spec(self):
-        return self.left.cache_spec() or self.right.cache_spec()
-
-    def state_spec(self):
-        return self.left.state_spec() or self.right.state_spec()
-
-    def forward(self, h: torch.Tensor, ctx: StepContext, site: SiteCache):
-        out = []
-        for m, s in ((self.left, self.left_scale), (self.right, self.right_scale)):
-            y = m.forward(h, ctx, site)
-            out += [(t, c * s) for t, c in y] if isinstance(y, (list, tuple)) else [(y, s)]
-        return out

@@ -29,6 +29,22 @@ from .linear import Linear
 CHUNKED_MIN_TOKENS = 32       # portions at least this long take the chunked form
 
 
+def constant_decay_recurrence(proj: torch.Tensor, bases, decay: torch.Tensor, state: torch.Tensor, ctx: StepContext, o: torch.Tensor,
+                              heads: int, dk: int, dv: int, storage: torch.dtype, silu: bool = False, exact: bool = False) -> None:
+    """S <- decay_h S + k v^T; o = S^T q over the step's rows, from and into ``state``; ``decay`` float32 [1, heads], q, k and v at
+    ``bases`` of the float32 rows ``proj``.  16-bit storage: portions of CHUNKED_MIN_TOKENS and more in chunks on the tensor
+    cores (``exact``: with queries and keys in two parts each)."""
+    rows = decay.expand(proj.shape[0], heads)
+    mode = ctx.options.get("scan", "auto")
+    if (mode == "chunks" or (mode == "auto" and storage == torch.bfloat16 and ctx.max_q_len >= CHUNKED_MIN_TOKENS)) \
+            and ctx.prefill_tiles > 0 and K.linear_chunk_supported(dk):
+        if ctx.decode_seqs:                                                          # the single-row entries come first
+            K.state_scan(K.SCAN_LINEAR, proj, bases, None, rows, None, state, ctx, o, heads, heads, dk, dv, silu=silu, seqs=ctx.decode_seqs)
+        K.linear_chunk(proj, bases, decay, state, ctx, o, heads, heads, dk, dv, silu=silu, exact=exact)
+    else:
+        K.state_scan(K.SCAN_LINEAR, proj, bases, None, rows, None, state, ctx, o, heads, heads, dk, dv, silu=silu)
+
+
 @MIXERS.register("lightning")
 class LightningAttention(Mixer):
     def __init__(self, hidden: int, heads: int, dk: int, dv: int, decay: Sequence[float], norm_eps: float) -> None:
@@ -58,15 +74,7 @@ class LightningAttention(Mixer):
         n, v0 = H * dv, 2 * H * dk
         proj = self.qkvg.forward(h, ctx, out_dtype=torch.float32)
         o = torch.empty((T, n), dtype=torch.float32, device=h.device)                # (the scan zeroes padding rows)
-        bases, decay = (0, H * dk, v0), self._decay.expand(T, H)
-        mode = ctx.options.get("scan", "auto")
-        if (mode == "chunks" or (mode == "auto" and h.dtype == torch.bfloat16 and ctx.max_q_len >= CHUNKED_MIN_TOKENS)) \
-                and ctx.prefill_tiles > 0 and K.linear_chunk_supported(dk):
-            if ctx.decode_seqs:                                                      # the single-row entries come first
-                K.state_scan(K.SCAN_LINEAR, proj, bases, None, decay, None, site.state, ctx, o, H, H, dk, dv, silu=True, seqs=ctx.decode_seqs)
-            K.linear_chunk(proj, bases, self._decay, site.state, ctx, o, H, H, dk, dv, silu=True)
-        else:
-            K.state_scan(K.SCAN_LINEAR, proj, bases, None, decay, None, site.state, ctx, o, H, H, dk, dv, silu=True)
+        constant_decay_recurrence(proj, (0, H * dk, v0), self._decay, site.state, ctx, o, H, dk, dv, h.dtype, silu=True)
         gated = torch.empty((T, n), dtype=h.dtype, device=h.device)
         K.group_rms_gate(o, proj[:, v0 + n:], self._norm, gated, n, self.norm_eps, False, "sigmoid")
         return self.o.forward(gated, ctx, out_dtype=torch.float32)

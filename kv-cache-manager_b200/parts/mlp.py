@@ -66,15 +66,15 @@ class GatedMLP(FeedForward):
 
 @FEED_FORWARDS.register("dense_mlp")
 class DenseMLP(FeedForward):
-    """Ungated feed-forward: down( act(x Wu^T) ); act "relu2" = max(z, 0)^2, or "polynorm":
+    """Ungated feed-forward: down( act(x Wu^T) ); act "relu2" = max(z, 0)^2, "gelu_tanh" = the tanh form of gelu, or "polynorm":
     a N(z) + b N(z^2) + c N(z^3) + e with the four learned numbers ``act`` = (a, b, c, e), powers taken
     element by element and N(v) = v / sqrt(mean(v^2) + norm_eps) over a row's ``intermediate`` values (the up
     product's float32 result goes in; sums and roots are float32)."""
 
     def __init__(self, hidden: int, intermediate: int, activation: str = "relu2", norm_eps: float = 1e-6) -> None:
         super().__init__()
-        if activation not in ("relu2", "polynorm"):
-            raise ValueError(f"dense_mlp: activation '{activation}' has no kernel (only 'relu2', 'polynorm')")
+        if activation not in (*K.UNARY_KINDS, "polynorm"):
+            raise ValueError(f"dense_mlp: activation '{activation}' has no kernel (only {', '.join(K.UNARY_KINDS)}, polynorm)")
         self.hidden, self.intermediate, self.activation, self.norm_eps = hidden, intermediate, activation, float(norm_eps)
         self.up = self.add_child("up", Linear(hidden, intermediate, hidden ** -0.5))
         self.down = self.add_child("down", Linear(intermediate, hidden, intermediate ** -0.5))
@@ -101,8 +101,16 @@ class DenseMLP(FeedForward):
                 and ctx.options.get("fuse", True) and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0
                 and (M <= 8 or w.numel() * 2 <= STREAM_MAX_BYTES) and K.stream_gemm_supported(M, self.intermediate, h.shape[1])):
             z = torch.empty((M, self.intermediate), dtype=h.dtype, device=h.device)
-            K.gemm_stream_relu_sq(h, w, z)
+            K.gemm_stream_act(h, w, z, self.activation)
+        elif (h.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and ctx.options.get("fuse", True) and M >= TCGEN05_MIN_ROWS
+              and ctx.options.get("gemm", "auto") in ("auto", "native", "tcgen05")
+              and (ctx.options.get("gemm", "auto") != "auto"
+                   or (tiles_fill_well(M, self.intermediate, h.device) and h.shape[1] <= TCGEN05_GATED_MAX_HIDDEN))
+              and K.tcgen05_gemm_supported(h, w)):
+            # Many rows (prefill), as for the gated feed-forward above: the activation in the tcgen05 product's epilogue.
+            z = torch.empty((M, self.intermediate), dtype=h.dtype, device=h.device)
+            K.gemm_tcgen05_act(h, w, z, self.activation)
         else:
             z = self.up.forward(h, ctx)
-            K.relu_sq(z, z)
+            K.unary_act(z, z, self.activation)
         return self.down.forward(z, ctx, out_dtype)

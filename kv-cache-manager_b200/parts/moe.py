@@ -10,7 +10,8 @@ Options (constructor parameters): ``scores`` "sigmoid" takes s = sigmoid(z) inst
 declares a learned number per expert that is added to s for the CHOICE only (choice scores may be negative, the
 weights use s itself); ``group_top`` = 2 scores a group by the sum of its two largest choice scores;
 ``shared_gate`` False runs the shared expert ungated (the router matrix then has no extra row); ``renorm`` divides the
-chosen scores by their sum (+ 1e-20) before the scale.
+chosen scores by their sum (+ 1e-20) before the scale; ``scores`` "softmax_chosen" chooses by the logits and takes the softmax
+over the chosen ones only as weights; ``router_bias`` declares a learned number per expert that joins the logits.
 
 The experts' matrices are stacked ([E, 2F, D] gate rows before up rows, [E, D, F]); the optional
 shared expert is the engine's gated feed-forward and runs for every row; its per-row gate is one
@@ -32,7 +33,7 @@ from .mlp import GatedMLP
 class RoutedExperts(FeedForward):
     def __init__(self, hidden: int, experts: int, expert_ff: int, top: int, scale: float = 1.0, groups: int = 1,
                  keep: int = 1, shared_ff: int = 0, scores: str = "softmax", correction: bool = False, group_top: int = 1,
-                 shared_gate: bool = True, renorm: bool = False) -> None:
+                 shared_gate: bool = True, renorm: bool = False, router_bias: bool = False) -> None:
         super().__init__()
         if experts < 1 or groups < 1 or experts % groups or not (1 <= keep <= groups):
             raise ValueError(f"routed_experts: {experts} experts do not form {groups} equal groups of which {keep} are kept")
@@ -40,8 +41,8 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"routed_experts: top {top} exceeds the {(experts // groups) * keep} experts a row may choose from")
         self.hidden, self.experts, self.expert_ff, self.top = hidden, experts, expert_ff, top
         self.scale, self.groups, self.keep = float(scale), groups, keep
-        if scores not in ("softmax", "sigmoid") or group_top not in (1, 2):
-            raise ValueError("routed_experts: scores 'softmax' | 'sigmoid', group_top 1 | 2")
+        if scores not in K.ROUTE_SCORES or group_top not in (1, 2):
+            raise ValueError("routed_experts: scores 'softmax' | 'sigmoid' | 'softmax_chosen', group_top 1 | 2")
         self.scores, self.group_top = scores, int(group_top)
         self.shared_gate = bool(shared_gate) and bool(shared_ff)
         self.renorm = bool(renorm)
@@ -52,7 +53,9 @@ class RoutedExperts(FeedForward):
         self.declare("router", (experts + (1 if self.shared_gate else 0), hidden), ("normal", hidden ** -0.5), "matrix")
         if correction:
             self.declare("correction", (experts,), ("normal", 0.1), "vector")
-        self._correction = None
+        if router_bias:
+            self.declare("router_bias", (experts,), ("normal", 0.1), "vector")
+        self._correction = self._bias = None
         self.declare("gate_up", (experts * 2 * expert_ff, hidden), ("normal", hidden ** -0.5), "matrix")
         self.declare("down", (experts * hidden, expert_ff), ("normal", expert_ff ** -0.5), "matrix")
         self._wgu = self._wd = self._router = None
@@ -66,6 +69,8 @@ class RoutedExperts(FeedForward):
         self._router = r if r.dtype in (torch.float32, dtype) else r.to(dtype)
         if "correction" in self.param_specs():
             self._correction = self.param("correction").to(device=device, dtype=torch.float32).contiguous()
+        if "router_bias" in self.param_specs():
+            self._bias = self.param("router_bias").to(device=device, dtype=torch.float32).contiguous()
 
     def forward(self, h: torch.Tensor, ctx: StepContext, out_dtype=None) -> torch.Tensor:
         """Returns float32 rows (``out_dtype`` is accepted for the feed-forward interface and must allow that)."""
@@ -92,7 +97,7 @@ class RoutedExperts(FeedForward):
         wt = torch.empty((M, top), dtype=torch.float32, device=dev)
         gate = torch.empty((M,), dtype=torch.float32, device=dev) if self.shared_gate else None
         K.moe_route(h, self._router, self.experts, self.groups, self.keep, top, self.scale, idx, wt, gate, self.scores,
-                    self._correction, self.group_top, self.renorm)
+                    self._correction, self.group_top, self.renorm, self._bias)
         work = torch.empty((K.moe_work_ints(M, top, self.experts),), dtype=torch.int32, device=dev)
         act = torch.empty((M * top, self.expert_ff), dtype=h.dtype, device=dev)
         y = torch.empty((M * top, D), dtype=torch.float32, device=dev)

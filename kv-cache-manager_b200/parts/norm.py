@@ -79,7 +79,7 @@ class Float32RMSNorm(Norm):
     """RMS norm all in float32 up to the one rounding of its result: out = w * x / sqrt(mean(x^2) + eps).  ``pending`` may
     be a list of (float32 tensor, scale) pairs and one ``ExpertSum`` (a block whose sublayers' outputs are summed hands
     them on unsummed); ``forward`` reads the stream with them and leaves x as it is: the final norm, with its row gather.
-    The "parallel_norms" block uses two of these (``multiplier``, ``eps``) in one kernel."""
+    The "parallel_norms" block uses two of these (``multiplier``, ``eps``) in one kernel, the "sandwich" block four."""
 
     def __init__(self, hidden: int, eps: float, init=("ones",)) -> None:
         super().__init__()
@@ -92,6 +92,12 @@ class Float32RMSNorm(Norm):
         self.multiplier = self.param("weight").to(device=device, dtype=torch.float32).contiguous()
 
     def forward(self, x: torch.Tensor, pending, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        if isinstance(pending, ClosingNorm):
+            if pending.eps != self.eps:
+                settle(x, pending)
+                pending = ClosingNorm(None, None, self.eps)
+            K.norm_post_pre(x, pending.y, pending.multiplier, self.multiplier, out, self.eps, rows)
+            return
         dense, experts = split_pending(pending)
         K.norm_pair(x, dense, experts, self.multiplier, self.eps, out, rows=rows)
 

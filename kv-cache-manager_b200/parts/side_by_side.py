@@ -1,0 +1,100 @@
+"""Two mixers that read the same rows, side by side in one layer.
+
+    y = left_scale * left(h) + right_scale * right(h)                                          (``out_norm`` off)
+    y = left_scale * w_l * left(h) / rms(left(h)) + right_scale * w_r * right(h) / rms(right(h))        (``out_norm`` on)
+
+rms(v) = sqrt(mean(v^2) + norm_eps) over the model's width, w_l and w_r plain learned vectors [hidden].
+
+At most one of the two keeps paged keys and values.  Each may keep fixed-size state: the call site's state row is then theirs
+one behind the other, each part starting at a multiple of four floats.  The sum is not formed here: without ``out_norm`` the two
+float32 outputs are returned as (tensor, scale) pairs for the block to hand to the next norm kernel, which adds
+them into the stream; with it they are returned as a ``NormedSum``, which the closing norm's kernel forms.
+
+Two staged mixers (see ``parts.base.Mixer``) share launches: their input projections are one product (the matrices are joined
+row-wise once, after loading, and the mixers' own parameters become views of the joint one), their heads are prepared by one
+launch and gated by one.  ``fuse`` off: each mixer runs by itself.
+"""
+from __future__ import annotations
+
+import dataclasses
+
+import torch
+
+from ..kernels import library as K
+from .base import MIXERS, Mixer, NormedSum, SiteCache, StateSpec, StepContext, run_prepare
+from .linear import matmul_nt
+
+
+def _up4(n: int) -> int:
+    return (n + 3) // 4 * 4
+
+
+@MIXERS.register("side_by_side")
+class SideBySideMixer(Mixer):
+    def __init__(self, left: Mixer, right: Mixer, left_scale: float = 1.0, right_scale: float = 1.0, out_norm: bool = False,
+                 hidden: int = 0, norm_eps: float = 1e-6, init=("ones_jitter", 0.1)) -> None:
+        super().__init__()
+        self.left, self.right = self.add_child("left", left), self.add_child("right", right)
+        self.left_scale, self.right_scale, self.norm_eps = float(left_scale), float(right_scale), float(norm_eps)
+        if left.cache_spec() is not None and right.cache_spec() is not None:
+            raise ValueError("side_by_side: both mixers want the call site's cache")
+        sizes = []
+        for m in (left, right):
+            s = m.state_spec()
+            if s is not None and (len(s.shape) != 1 or s.dtype != torch.float32):
+                raise ValueError("side_by_side: the mixers' states are float32 rows")
+            sizes.append(s.shape[0] if s is not None else 0)
+        self._state_sizes = tuple(sizes)
+        self._state_starts = (0, _up4(sizes[0]))
+        self._sub_sites = {}
+        self.out_norm = bool(out_norm)
+        if self.out_norm:
+            self.declare("left_out", (hidden,), init, "vector")
+            self.declare("right_out", (hidden,), init, "vector")
+        self._multipliers = self._joint = None
+
+    def cache_spec(self):
+        return self.left.cache_spec() or self.right.cache_spec()
+
+    def state_spec(self):
+        n, (_, at) = self._state_sizes, self._state_starts
+        return StateSpec((_up4(at + n[1]),), torch.float32) if any(n) else None
+
+    def prepare(self, device, dtype) -> None:
+        left, right = self.left, self.right
+        if left.staged and right.staged:
+            a, b = left.projection.param("weight"), right.projection.param("weight")
+            self._joint = torch.cat([a, b])
+            left.projection.set_param("weight", self._joint[:a.shape[0]])
+            right.projection.set_param("weight", self._joint[a.shape[0]:])
+        super().prepare(device, dtype)
+        if self.out_norm:
+            self._multipliers = tuple((self.param(n).to(device=device, dtype=torch.float32) * s).contiguous()
+                                      for n, s in (("left_out", self.left_scale), ("right_out", self.right_scale)))
+
+    def _sites(self, site: SiteCache):
+        """The call site as each mixer sees it: its own part of the state rows."""
+        if site.state is None:
+            return site, site
+        key = (site.state.data_ptr(), site.group, site.k.data_ptr() if site.k is not None else 0)
+        if key not in self._sub_sites:
+            self._sub_sites[key] = tuple(dataclasses.replace(site, state=site.state[:, at:at + n] if n else None)
+                                         for at, n in zip(self._state_starts, self._state_sizes))
+        return self._sub_sites[key]
+
+    def forward(self, h: torch.Tensor, ctx: StepContext, site: SiteCache):
+        sites, mixers = self._sites(site), (self.left, self.right)
+        if self._joint is not None and ctx.options.get("fuse", True):
+            proj = matmul_nt(h, self._joint, torch.float32, ctx.options)
+            works = [m.begin(proj, at, h.dtype, ctx, s) for m, at, s in zip(mixers, (0, self.left.projection.out_features), sites)]
+            run_prepare(proj, works, h.dtype, ctx)
+            K.gate_heads(proj, [m.mix(w) for m, w in zip(mixers, works)])
+            outs = [m.finish(w) for m, w in zip(mixers, works)]
+        else:
+            outs = [m.forward(h, ctx, s) for m, s in zip(mixers, sites)]
+        if self.out_norm:
+            return NormedSum(list(zip(outs, self._multipliers)), self.norm_eps)
+        pairs = []
+        for y, s in zip(outs, (self.left_scale, self.right_scale)):
+            pairs += [(t, c * s) for t, c in y] if isinstance(y, (list, tuple)) else [(y, s)]
+        return pairs

@@ -360,9 +360,9 @@ def test_squared_relu_in_the_streaming_product():
             continue
         y = torch.empty(M, N, dtype=torch.bfloat16, device="cuda")
         K.gemm_stream(x, w, y)
-        K.relu_sq(y, y)
+        K.unary_act(y, y, "relu2")
         z = torch.empty_like(y)
-        K.gemm_stream_relu_sq(x, w, z)
+        K.gemm_stream_act(x, w, z, "relu2")
         assert torch.equal(y, z)
         ref = torch.relu(x.double() @ w.double().T) ** 2
         assert (z.double() - ref).abs().max().item() < 0.05 * max(1.0, ref.abs().max().item())
