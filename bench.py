@@ -583,6 +583,56 @@ def bimepel_work(z, T, ctx, decode):
     }
 
 
+# --compare pemorax: the Pemorax design (windowed attention with short convolutions, kept first tokens, a unit sink and a gate
+# beside retention in EVERY layer; dense gelu or routed experts) beside Bimepel (whose attention, recurrence and expert kernels
+# are the like ones, an attention or a recurrence per layer) and the Llama decoder, at equal width, number of layers, head
+# counts and active feed-forward size.
+PEMORAX_SIZES = {
+    "p2048": dict(BIMEPEL_SIZES["p2048"], window=1024, keep=4, taps=4, dense_ff=6144),
+    "p4096": dict(BIMEPEL_SIZES["p4096"], window=1024, keep=4, taps=4, dense_ff=12288),
+}
+
+
+def pemorax_configs(z):
+    """(Pemorax config, Bimepel config, Llama config) of one size: the layers that are Bimepel's attention layers carry the
+    dense feed-forward, its lightning layers the experts."""
+    from kvcm.config import config_from_dict
+    D, H, G, d = z["width"], z["heads"], z["kv_heads"], z["dim"]
+    rot = {"base": 500000.0, "dims": d, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}
+    mixer = {"left": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "conv": z["taps"], "rot": rot, "softcap": 50.0,
+                      "mask": {"size": z["window"], "keep_first": z["keep"]}},
+             "right": {"heads": H, "dim": d, "vdim": d, "decay": [1.0 - 2.0 ** (-1 - 8.0 * h / H) for h in range(H)], "rot": {"base": 10000.0, "dims": d}}}
+    dense = {"kind": "dense", "ff": z["dense_ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["moe_top"]}}
+    layers = [{"type": "parallel", "mixer": mixer, "mlp": dense if kind == "attention" else moe} for kind in rivetar_runs(z)]
+    pem = {"architecture": "Pemorax", "vocab": COMPARE_VOCAB, "width": D, "norm": {"eps": 1e-6}, "layers": layers}
+    bim, lla = bimepel_configs(z)
+    return config_from_dict(pem), bim, lla
+
+
+def pemorax_work(z, T, ctx, decode):
+    """What the families of one Pemorax step have to do at least: flops, or bytes they must move."""
+    D, H, G, d, W = z["width"], z["heads"], z["kv_heads"], z["dim"], z["window"]
+    runs = rivetar_runs(z)
+    n_den, n_moe, L = runs.count("attention"), runs.count("lightning"), len(runs)
+    own = min(ctx, W + z["keep"])                                 # keys of the last position
+    seen = T * own if decode else sum(min(i + 1, W + z["keep"]) for i in range(T))
+    hit = min(z["experts"], T * z["moe_top"])
+    q, kv, r = H * d, G * d, H * d
+    return {
+        "attention": dict(flops=4.0 * H * d * seen * L, bytes=2.0 * 2 * G * d * T * own * L if decode else None),
+        "state_scan": dict(flops=T * 4.0 * H * d * d * L, bytes=8.0 * T * H * d * d * L if decode else None),
+        "moe_experts_tcgen05": dict(flops=2.0 * T * z["moe_top"] * 3 * z["expert_ff"] * D * n_moe,
+                                    bytes=2.0 * hit * 3 * z["expert_ff"] * D * n_moe if decode else None),
+        "feed_forward": dict(flops=2.0 * T * 2 * z["dense_ff"] * D * n_den, bytes=2.0 * 2 * z["dense_ff"] * D * n_den if decode else None),
+        # the projections' q, k, v of the attention and q, k of the recurrence read, written as 16 and 32 bits
+        "head_prepare": dict(flops=None, bytes=T * ((q + 2 * kv) * (4.0 + 2.0) + 2 * r * (4.0 + 4.0)) * L),
+        "head_gate": dict(flops=None, bytes=T * ((q * (2.0 + 4.0 + 2.0)) + r * (4.0 + 4.0 + 2.0)) * L),
+        # two norm launches a layer: the stream read and written, one output; two branches, or the sublayer's result(s)
+        "norm_post_pre": dict(flops=None, bytes=T * D * (2 * (4.0 + 4.0 + 2.0) * L + 2 * 4.0 * L + 4.0 * n_den + 4.0 * z["moe_top"] * n_moe)),
+    }
+
+
 def compare_main(args) -> int:
     import torch
     from kvcm.config import EngineConfig, KVManagerConfig, SchedulerConfig
@@ -594,8 +644,11 @@ def compare_main(args) -> int:
                                   "rivetar": (RIVETAR_SIZES, rivetar_configs, rivetar_work),
                                   "lobutar": (LOBUTAR_SIZES, lobutar_configs, lobutar_work),
                                   "bimepel": (BIMEPEL_SIZES, bimepel_configs, bimepel_work),
+                                  "pemorax": (PEMORAX_SIZES, pemorax_configs, pemorax_work),
                                   "tolanex": (COMPARE_SIZES, compare_configs, tolanex_work)}[first]
-    out = {"compare": f"{first} beside llama at equal width, depth and (active) feed-forward size", "dtype": "bf16",
+    names = (first, "bimepel", "llama") if first == "pemorax" else (first, "llama")
+    work_of = {first: first_work, "llama": llama_work, **({"bimepel": bimepel_work} if first == "pemorax" else {})}
+    out = {"compare": f"{first} beside {' and '.join(names[1:])} at equal width, depth and (active) feed-forward size", "dtype": "bf16",
            "data": "synthetic: random weights, uniform random token ids", "peaks": pk, "sizes": {}}
     steps, warmup = min(args.steps, 200), max(args.warmup, 3)
     for name, z in sizes.items():
@@ -603,12 +656,12 @@ def compare_main(args) -> int:
             continue
         if first == "bifatar":
             z = dict(z, layers=len(z["order"]), top=1, ff=z["llama_ff"], shared=0)      # the keys llama_work reads
-        elif first in ("rivetar", "bimepel"):
+        elif first in ("rivetar", "bimepel", "pemorax"):
             z = dict(z, layers=len(rivetar_runs(z)), top=1, ff=z["llama_ff"], shared=0)
         elif first == "lobutar":
             z = dict(z, layers=len(z["order"]), top=1, ff=z["llama_ff"], shared=0)
         res = {}
-        for arch, cfg in zip((first, "llama"), configs(z)):
+        for arch, cfg in zip(names, configs(z)):
             tensors = dict(random_tensors(cfg, 0, torch.bfloat16, device="cuda:0"))
             spec = model_from_tensors(cfg, tensors, "bfloat16", "cuda:0")
             del tensors
@@ -620,8 +673,7 @@ def compare_main(args) -> int:
             pre = prefill_times(spec, ec, COMPARE_VOCAB)
             fam = {k: {kk: {"calls": c, "ms": round(ms, 4)} for kk, (c, ms) in family_profile(spec, COMPARE_VOCAB, k).items()}
                    for k in ("prefill", "decode")}
-            work = {"prefill": (first_work if arch == first else llama_work)(z, PREFILL_TOKENS, PREFILL_TOKENS, False),
-                    "decode": (first_work if arch == first else llama_work)(z, 8, 1024, True)}
+            work = {"prefill": work_of[arch](z, PREFILL_TOKENS, PREFILL_TOKENS, False), "decode": work_of[arch](z, 8, 1024, True)}
             res[arch] = {"decode_tokens_per_s": round(8 * steps * 1e3 / dec["dev_ms"], 1),
                          "decode_ms_per_step": round(dec["dev_ms"] / steps, 4),
                          "decode_e2e_tokens_per_s": round(8 * steps * 1e3 / dec["wall_ms"], 1),
@@ -761,8 +813,8 @@ def main() -> int:
                          "'native' this engine's kernels only, 'library' the library wherever it can stand")
     ap.add_argument("--only", default="all", choices=["all", "prefill"],
                     help="'prefill': run only the 2,048-token prefill step and print its numbers (for profiling)")
-    ap.add_argument("--compare", default="", choices=["", "tolanex", "bifatar", "rivetar", "lobutar", "bimepel"],
-                    help="'tolanex' | 'bifatar' | 'rivetar' | 'lobutar' | 'bimepel': instead of the default workload, prefill and decode of that design beside "
+    ap.add_argument("--compare", default="", choices=["", "tolanex", "bifatar", "rivetar", "lobutar", "bimepel", "pemorax"],
+                    help="'tolanex' | 'bifatar' | 'rivetar' | 'lobutar' | 'bimepel' | 'pemorax': instead of the default workload, prefill and decode of that design beside "
                          "the Llama decoder at equal sizes, with device time per kernel family")
     ap.add_argument("--size", default="all", choices=["all"] + sorted(COMPARE_SIZES) + sorted(BIFATAR_SIZES) + sorted(RIVETAR_SIZES) + sorted(LOBUTAR_SIZES) + sorted(BIMEPEL_SIZES),
                     help="with --compare: one size only")

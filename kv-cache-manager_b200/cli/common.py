@@ -112,6 +112,21 @@ def _bimepel_mini():
             ]}
 
 
+def _pemorax_mini():
+    """A small Pemorax: windowed attention that keeps the first tokens, with a scaled rotation, beside retention in every
+    layer; routed experts, a layer without a feed-forward, a dense one."""
+    rot = {"base": 10000.0, "dims": 32, "scaling": {"factor": 4.0, "original": 256, "fast": 32.0, "slow": 1.0}}
+    left = {"heads": 6, "kv_heads": 2, "dim": 64, "vdim": 32, "scale": 0.125, "conv": 4, "rot": rot, "softcap": 30.0}
+    right = {"heads": 4, "dim": 32, "vdim": 96, "decay": [0.75, 0.95, 0.99, 0.999], "rot": {"base": 10000.0, "dims": 16}}
+    windowed = {"left": dict(left, mask={"size": 90, "keep_first": 3}), "right": right}
+    return {"architecture": "Pemorax", "vocab": 1000, "width": 384, "norm": {"eps": 1e-5},
+            "layers": [
+                {"type": "parallel", "mixer": windowed, "mlp": {"kind": "moe", "expert": {"ff": 128}, "router": {"experts": 16, "top": 3}}},
+                {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": None},
+                {"type": "parallel", "mixer": windowed, "mlp": {"kind": "dense", "ff": 640}},
+            ]}
+
+
 PRESETS = {
     # name: (config.json keys, seed, norm jitter); keys with "architecture" go through the registry,
     # the others are those of a Llama dense decoder
@@ -120,6 +135,7 @@ PRESETS = {
     "rivetar-mini": (_rivetar_mini(), 7, 0.1),
     "lobutar-mini": (_lobutar_mini(), 8, 0.1),
     "bimepel-mini": (_bimepel_mini(), 9, 0.1),
+    "pemorax-mini": (_pemorax_mini(), 10, 0.1),
     "tiny-a": (dict(vocab_size=256, hidden_size=64, intermediate_size=172, num_hidden_layers=2,
                     num_attention_heads=4, num_key_value_heads=2, head_dim=16, max_position_embeddings=128,
                     rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=False), 0, 0.0),

@@ -136,3 +136,16 @@ def test_kvbench_and_kvcorrect_on_the_bimepel_preset():
     rc, out, err = run("kvcorrect", "--preset", "bimepel-mini", "--steps", "8", "--prompts", "3", "--prompt-len", "40")
     assert rc in (0, 2), out[-2000:] + err[-2000:]
     assert "[PASS] alone (scattered pages) = batch" in out and "[PASS] paged = contiguous" in out
+
+
+def test_kvbench_and_kvcorrect_on_the_pemorax_preset():
+    """A seventh architecture through the same flags: windowed attention with short convolutions beside retention in every
+    layer (pages and state of one call site), dense and routed feed-forwards, served by the scheduler, and kvcorrect's checks."""
+    rc, out, err = run("kvbench", "--preset", "pemorax-mini", "--requests", "10", "--rate", "0", "--prompt-len", "60",
+                       "--output-len", "12", "--max-seq-len", "128", "--num-blocks", "48", "--max-num-seqs", "4",
+                       "--max-batched-tokens", "96", "--warmup", "1")
+    assert rc == 0, err[-2000:]
+    assert "completed 10/10" in out
+    rc, out, err = run("kvcorrect", "--preset", "pemorax-mini", "--steps", "8", "--prompts", "3", "--prompt-len", "40")
+    assert rc in (0, 2), out[-2000:] + err[-2000:]
+    assert "[PASS] alone (scattered pages) = batch" in out and "[PASS] paged = contiguous" in out
