@@ -76,7 +76,7 @@ unary_act_kernel(const T* in, T* out, long long n, int kind) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    stf(out + i, unary_act(kind, ldf(in + i)));
+    stf(out + i, sizeof(T) == 2 ? unary_act_16(kind, ldf(in + i)) : unary_act(kind, ldf(in + i)));
   }
 }
 
@@ -91,7 +91,7 @@ unary_act_vec_kernel(const uint4* in, uint4* out, long long n8, int kind) {
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       float2 f = __bfloat1622float2(h[k]);
-      h[k] = __floats2bfloat162_rn(unary_act(kind, f.x), unary_act(kind, f.y));
+      h[k] = __floats2bfloat162_rn(unary_act_16(kind, f.x), unary_act_16(kind, f.y));
     }
     out[i] = v;
   }

@@ -27,6 +27,12 @@ __device__ __forceinline__ float unary_act(int kind, float z) {
   if (kind == kUnaryGeluTanh) return z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));
   return z;
 }
+// The same where the result is rounded to bfloat16: CUDA's fast exponential and division (a few units in float's last place;
+// a denominator beyond 2^126 gives zero, which is the limit).  Every kernel that stores bfloat16 takes this one.
+__device__ __forceinline__ float unary_act_16(int kind, float z) {
+  if (kind == kUnaryGeluTanh) return __fdividef(z, 1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));
+  return unary_act(kind, z);
+}
 
 template <int KIND, typename T>
 __device__ __forceinline__ float gated_act(float g, float u, const GatedAct& a) {

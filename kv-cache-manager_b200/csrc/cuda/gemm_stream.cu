@@ -493,7 +493,7 @@ gemm_stream_kernel(StreamParams p) {
         const int n = row_in(base, r);
         if (n < p.N && m < p.M) {
           float v = total_of(r, m);
-          if (p.unary) v = unary_act(p.unary, Store<OutT>::round(v));   // as the separate kernel: of the rounded sum
+          if (p.unary) v = unary_act_16(p.unary, Store<OutT>::round(v));   // as the separate kernel: of the rounded sum
           stf(Y + size_t(m) * p.ldy + n, v);
         }
       }

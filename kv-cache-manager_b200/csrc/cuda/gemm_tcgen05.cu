@@ -213,7 +213,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
                   const float2 f = __bfloat1622float2(h2[i]);
-                  h2[i] = __floats2bfloat162_rn(unary_act(act.unary, f.x), unary_act(act.unary, f.y));
+                  h2[i] = __floats2bfloat162_rn(unary_act_16(act.unary, f.x), unary_act_16(act.unary, f.y));
                 }
               }
 #pragma unroll
@@ -228,7 +228,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
             for (int i = 0; i < 32; ++i)
               if (col0 + i < N) {
                   const float f = __uint_as_float(v[i]);
-                  stf(dst + i, act.unary ? unary_act(act.unary, Store<OutT>::round(f)) : f);
+                  stf(dst + i, act.unary ? unary_act_16(act.unary, Store<OutT>::round(f)) : f);
                 }
           }
         }

@@ -32,12 +32,13 @@ struct HeadSegment {                       // (mirrored by kernels/library.py)
   int src, conv;                           // first column of the projection; first convolved channel or -1
   int table, interleaved, dest;            // rotation table or -1
   float scale;
+  int rows;                                // rows of the step that the segment covers, from the first on
   int items;                               // work items of a head (filled in by the launcher)
 };
 struct HeadPrepareParams {
   const float* proj; long long ldp;
   const int* positions;
-  const float* inv_freq[2]; int half[2]; float amplitude[2];
+  const float* inv_freq[2]; const float* cs[2]; int half[2]; float amplitude[2];      // cs: [rows][half cosines | half sines] (used for many rows) or null
   const float* conv_w; float* state; long long state_stride;
   int taps, channels, conv_col, write_state;
   const int* row_seq; const int* seq_q_start; const int* seq_q_len; const int* seq_state_slot;
@@ -61,10 +62,11 @@ __device__ __forceinline__ void hp_load4(float (&v)[4], const float* p) {
 
 // What a block's rows need besides the projection.
 template <int R> struct HeadRowInfo {
-  int local[R], state_slot[R], cache_slot[R];     // row of its portion, the request's state slot, the row's page slot
+  int local[R], state_slot[R], page[R], off[R];   // row of its portion, the request's state slot, the row's page (or -1) and place
+  int whole;                                      // all rows are there and none reaches ahead of its portion
 };
 
-// Cosines and sines of R rows: [row][table 0: half cosines, half sines | table 1: ..]
+// Cosines and sines of R rows: [row][table 0: half cosines, half sines | table 1: ..], amplitude included
 template <int R>
 __device__ __forceinline__ void hp_tables(const HeadPrepareParams& p, int r0, float* cs) {
   const int n0 = p.half[0], n = n0 + p.half[1];
@@ -104,17 +106,34 @@ __device__ __forceinline__ void hp_quads(const HeadPrepareParams& p, const HeadS
   }
   if constexpr (TAPS > 1) {
   float raw[R + TAPS - 1][4], w[4 * TAPS];
+  if (R > 1 && info.whole) {
+    const float* from = src + (r0 - (TAPS - 1)) * p.ldp;
 #pragma unroll
-  for (int k = 0; k < R + TAPS - 1; ++k) {
-    const int row = r0 + k - (TAPS - 1);
-    raw[k][0] = raw[k][1] = raw[k][2] = raw[k][3] = 0.f;
-    if (row >= 0 && row < p.rows) hp_load4(raw[k], src + row * p.ldp);
+    for (int k = 0; k < R + TAPS - 1; ++k, from += p.ldp) hp_load4(raw[k], from);
+  } else {
+#pragma unroll
+    for (int k = 0; k < R + TAPS - 1; ++k) {
+      const int row = r0 + k - (TAPS - 1);
+      raw[k][0] = raw[k][1] = raw[k][2] = raw[k][3] = 0.f;
+      if (row >= 0 && row < p.rows) hp_load4(raw[k], src + row * p.ldp);
+    }
   }
   const float* wp = p.conv_w + size_t(g.conv + at) * TAPS;
 #pragma unroll
   for (int k = 0; k < TAPS; ++k) {
     float4 f = *reinterpret_cast<const float4*>(wp + 4 * k);
     w[4 * k] = f.x; w[4 * k + 1] = f.y; w[4 * k + 2] = f.z; w[4 * k + 3] = f.w;
+  }
+  if (R > 1 && info.whole) {
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[i][e] = w[e * TAPS] * raw[i][e];
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) v[i][e] = fmaf(w[e * TAPS + j], raw[i + j][e], v[i][e]);
+      }
+    return;
   }
 #pragma unroll
   for (int i = 0; i < R; ++i) {
@@ -144,19 +163,52 @@ template <typename T, int R>
 __device__ __forceinline__ void hp_put(const HeadPrepareParams& p, const HeadSegment& g, const HeadRowInfo<R>& info, int r0, int i, int u, int c,
                                        const float (&v)[4]) {
   const int row = r0 + i;
-  if (row >= p.rows) return;
+  if (row >= g.rows) return;
   if (g.dest == kHeadFloatRows) {
     hp_store4(reinterpret_cast<float*>(g.out) + row * g.ld + u * g.dim + c, v);
   } else if (g.dest == kHeadRows) {
     hp_store4(reinterpret_cast<T*>(g.out) + row * g.ld + size_t(u) * g.HD + c, v);
-  } else if (info.cache_slot[i] >= 0) {
-    const int page = info.cache_slot[i] / p.block_size, off = info.cache_slot[i] - page * p.block_size;
-    hp_store4(reinterpret_cast<T*>(g.out) + ((size_t(page) * g.units + u) * p.block_size + off) * g.HD + c, v);
+  } else if (info.page[i] >= 0) {
+    hp_store4(reinterpret_cast<T*>(g.out) + ((size_t(info.page[i]) * g.units + u) * p.block_size + info.off[i]) * g.HD + c, v);
   }
 }
 
-template <typename T, int TAPS, int R>
-__global__ void __launch_bounds__(kHeadPrepareThreads)
+// The angles of N neighbouring pairs from j on, for the block's row i: from shared memory, or (TAB) from the step's table.
+template <int N, bool TAB>
+__device__ __forceinline__ void hp_angles(const HeadPrepareParams& p, const HeadSegment& g, const float* cs, int n_cs, int r0, int i, int j,
+                                          float (&c)[N], float (&s)[N]) {
+  const int t = g.table, half = p.half[t];
+  if constexpr (TAB) {
+    const float* at = p.cs[t] + size_t(min(r0 + i, p.rows - 1)) * 2 * half + j;
+    if constexpr (N == 4) {
+      hp_load4(c, at);
+      hp_load4(s, at + half);
+    } else {
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        const bool in = j + e < half;
+        c[e] = in ? at[e] : 1.f;
+        s[e] = in ? at[half + e] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      c[e] *= p.amplitude[t];
+      s[e] *= p.amplitude[t];
+    }
+  } else {
+    const float* at = cs + i * n_cs + (t ? 2 * p.half[0] : 0) + j;
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      const bool in = j + e < half;
+      c[e] = in ? at[e] : 1.f;
+      s[e] = in ? at[half + e] : 0.f;
+    }
+  }
+}
+
+template <typename T, int TAPS, int R, bool TAB>
+__global__ void __launch_bounds__(kHeadPrepareThreads, R > 1 ? 3 : 1)
 head_prepare_kernel(const __grid_constant__ HeadPrepareParams p) {
   extern __shared__ __align__(16) float cs[];
   __shared__ HeadRowInfo<R> info;
@@ -171,11 +223,19 @@ head_prepare_kernel(const __grid_constant__ HeadPrepareParams p) {
       local = row - p.seq_q_start[s];
       slot = p.seq_state_slot[s];
     }
+    const int cache = in && p.slot_mapping ? p.slot_mapping[row] : -1;
+    const int page = cache >= 0 ? cache / p.block_size : -1;
     info.local[threadIdx.x] = local;
     info.state_slot[threadIdx.x] = slot;
-    info.cache_slot[threadIdx.x] = in && p.slot_mapping ? p.slot_mapping[row] : -1;
+    info.page[threadIdx.x] = page;
+    info.off[threadIdx.x] = cache - page * p.block_size;
+    if constexpr (R > 1) {
+      const unsigned mask = (1u << R) - 1;
+      const bool all = __all_sync(mask, in && local >= TAPS - 1);
+      if (threadIdx.x == 0) info.whole = all;
+    }
   }
-  hp_tables<R>(p, r0, cs);
+  if constexpr (!TAB) hp_tables<R>(p, r0, cs);
   __syncthreads();
   pdl_wait();
   const int n_cs = 2 * (p.half[0] + p.half[1]);
@@ -183,9 +243,9 @@ head_prepare_kernel(const __grid_constant__ HeadPrepareParams p) {
     int s = 0, it = item;
     while (it >= p.seg[s].units * p.seg[s].items) { it -= p.seg[s].units * p.seg[s].items; ++s; }
     const HeadSegment& g = p.seg[s];
+    if (r0 >= g.rows) continue;
     const int u = it / g.items, k = it - u * g.items;
     const int half = g.table >= 0 ? p.half[g.table] : 0;
-    const float* table = cs + (g.table == 1 ? 2 * p.half[0] : 0);
     if (half > 0 && !g.interleaved && k < half / 4) {                   // four pairs (c, c + half)
       const int c = 4 * k;
       float a[R][4], b[R][4];
@@ -193,10 +253,11 @@ head_prepare_kernel(const __grid_constant__ HeadPrepareParams p) {
       hp_quads<TAPS, R>(p, g, info, r0, u, c + half, b);
 #pragma unroll
       for (int i = 0; i < R; ++i) {
-        float x[4], y[4];
+        float x[4], y[4], co[4], si[4];
+        hp_angles<4, TAB>(p, g, cs, n_cs, r0, i, c, co, si);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          rotate_pair(a[i][e], b[i][e], table[i * n_cs + c + e], table[i * n_cs + half + c + e], x[e], y[e]);
+          rotate_pair(a[i][e], b[i][e], co[e], si[e], x[e], y[e]);
           x[e] *= g.scale;
           y[e] *= g.scale;
         }
@@ -215,16 +276,16 @@ head_prepare_kernel(const __grid_constant__ HeadPrepareParams p) {
     }
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-      if (g.interleaved) {
+      if (half > 0 && g.interleaved && c < 2 * half) {
+        float co[2], si[2];
+        hp_angles<2, TAB>(p, g, cs, n_cs, r0, i, c / 2, co, si);
 #pragma unroll
         for (int e = 0; e < 4; e += 2) {
-          const int j = (c + e) / 2;
-          if (j < half) {
-            float x, y;
-            rotate_pair(a[i][e], a[i][e + 1], table[i * n_cs + j], table[i * n_cs + half + j], x, y);
-            a[i][e] = x;
-            a[i][e + 1] = y;
-          }
+          if (c / 2 + e / 2 >= half) break;
+          float x, y;
+          rotate_pair(a[i][e], a[i][e + 1], co[e / 2], si[e / 2], x, y);
+          a[i][e] = x;
+          a[i][e + 1] = y;
         }
       }
 #pragma unroll
@@ -275,6 +336,7 @@ head_prepare_any_kernel(const __grid_constant__ HeadPrepareParams p) {
     int s = 0, u = h;
     while (u >= p.seg[s].units) { u -= p.seg[s].units; ++s; }
     const HeadSegment& g = p.seg[s];
+    if (row >= g.rows) continue;
     const int half = g.table >= 0 ? p.half[g.table] : 0;
     const float* table = cs + (g.table == 1 ? 2 * p.half[0] : 0);
     for (int c = lane; c < g.dim; c += 32) mine[c] = hp_element(p, g, row, local, slot, u * g.dim + c);
@@ -321,14 +383,18 @@ head_conv_state_kernel(const float* __restrict__ cols, long long ldp, int taps, 
 }
 
 template <typename T, int TAPS>
-static int launch_head_prepare_quads(const HeadPrepareParams& p, cudaStream_t s) {
+static int launch_head_prepare_quads(HeadPrepareParams p, cudaStream_t s) {
   const bool run = p.rows >= 1024;                             // many rows: several of them a thread
   const int R = run ? kHeadRunRows : 1;
   const int bx = (p.rows + R - 1) / R, most = (p.items + kHeadPrepareThreads - 1) / kHeadPrepareThreads;
-  const int by = max(1, min(most, 592 / bx));
-  const size_t smem = size_t(R) * 2 * (p.half[0] + p.half[1]) * sizeof(float);
-  if (run) return pdl_launch(head_prepare_kernel<T, TAPS, kHeadRunRows>, dim3(bx, by), dim3(kHeadPrepareThreads), smem, s, p);
-  return pdl_launch(head_prepare_kernel<T, TAPS, 1>, dim3(bx, by), dim3(kHeadPrepareThreads), smem, s, p);
+  auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  bool tab = run;                                              // (every rotation of the launch has a table)
+  for (int t = 0; t < 2; ++t) tab = tab && (p.half[t] == 0 || (p.cs[t] && (p.half[t] % 4) == 0 && aligned(p.cs[t])));
+  const int by = tab ? most : max(1, min(most, 592 / bx));
+  const size_t smem = tab ? 0 : size_t(R) * 2 * (p.half[0] + p.half[1]) * sizeof(float);
+  if (tab) return pdl_launch(head_prepare_kernel<T, TAPS, kHeadRunRows, true>, dim3(bx, by), dim3(kHeadPrepareThreads), smem, s, p);
+  if (run) return pdl_launch(head_prepare_kernel<T, TAPS, kHeadRunRows, false>, dim3(bx, by), dim3(kHeadPrepareThreads), smem, s, p);
+  return pdl_launch(head_prepare_kernel<T, TAPS, 1, false>, dim3(bx, by), dim3(kHeadPrepareThreads), smem, s, p);
 }
 
 template <typename T>
@@ -344,7 +410,7 @@ static int launch_head_prepare(HeadPrepareParams p, cudaStream_t s) {
   p.items = 0;
   for (int i = 0; i < p.segments; ++i) {
     HeadSegment& g = p.seg[i];
-    if (g.units < 1 || g.dim < 1 || g.HD < g.dim || g.table > 1 || (g.table >= 0 && 2 * p.half[g.table] > g.dim) ||
+    if (g.units < 1 || g.dim < 1 || g.rows < 0 || g.rows > p.rows || g.HD < g.dim || g.table > 1 || (g.table >= 0 && 2 * p.half[g.table] > g.dim) ||
         (g.dest == kHeadFloatRows && g.HD != g.dim) || (g.conv >= 0 && !p.conv_w) || g.dest < 0 || g.dest > 2)
       return KVCM_ERR_UNSUPPORTED;
     const int half = g.table >= 0 ? p.half[g.table] : 0;
@@ -427,7 +493,11 @@ head_gate_kernel(const __grid_constant__ HeadGateParams p) {
     const size_t at = size_t(row) * g.ldx + size_t(u) * g.HD;
     const float* gate = p.gates + row * p.ldg + g.gate + u * g.dv;
     T* out = reinterpret_cast<T*>(g.out) + size_t(row) * g.ldo + size_t(u) * g.dv;
-    auto act = [&](float z) { const float sg = 1.f / (1.f + expf(-z)); return g.silu ? z * sg : sg; };
+    // (bfloat16 results: CUDA's fast exponential and division, a few units in float's last place)
+    auto act = [&](float z) {
+      const float sg = sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : 1.f / (1.f + expf(-z));
+      return g.silu ? z * sg : sg;
+    };
     if (p.vec && g.dv <= 256) {                       // up to two quads a lane, kept in registers between the two passes
       float x[2][4], z[2][4];
 #pragma unroll

@@ -43,6 +43,7 @@ struct LinearChunkParams {
   const int* tile_seq; const int* tile_q0; const int* seq_q_start; const int* seq_q_len; const int* seq_state_slot;
   float* out;                              // [rows, heads * dv]
   int tiles, heads, qk_heads, dk, dv, dvp, silu, vec;
+  const float* cs; int half; float amplitude, k_scale;      // cs [rows][half cosines | half sines]: q and k turn in pairs (i, i + half); or null
 };
 
 __device__ __forceinline__ float lc_act(float z) { return z / (1.f + expf(-z)); }
@@ -89,6 +90,54 @@ __device__ __forceinline__ void lc_rows(const float* src, int ld, int n, int wid
   }
 }
 
+// The same with the row's pairs (i, i + half), i < half, turned by the step's angles and everything multiplied by `scale`
+// (vec, half % 4 == 0).  An item is four pairs or four elements behind them.
+template <int W, typename Put>
+__device__ __forceinline__ void lc_rows_turned(const LinearChunkParams& p, const float* src, int row0, int n, float scale, Put put) {
+  const int pairs = p.half / 4, per = W / 4 - pairs, total = kLcRows * per;
+  constexpr int kBatch = 4;
+#pragma unroll 1
+  for (int i0 = threadIdx.x; i0 < total; i0 += kBatch * kLcOuterThreads) {
+    float a[kBatch][4], b[kBatch][4], c[kBatch][4], s[kBatch][4];
+#pragma unroll
+    for (int t = 0; t < kBatch; ++t) {
+      const int i = i0 + t * kLcOuterThreads, r = i / per, k = i - r * per;
+      const bool turn = k < pairs;
+      const int at = turn ? 4 * k : 2 * p.half + 4 * (k - pairs);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { a[t][e] = b[t][e] = s[t][e] = 0.f; c[t][e] = 1.f; }
+      if (i >= total || r >= n || at >= p.dk) continue;
+      const float4 f = *reinterpret_cast<const float4*>(src + size_t(r) * p.ld + at);
+      a[t][0] = f.x; a[t][1] = f.y; a[t][2] = f.z; a[t][3] = f.w;
+      if (turn) {
+        const float4 g = *reinterpret_cast<const float4*>(src + size_t(r) * p.ld + at + p.half);
+        const float* cs = p.cs + size_t(row0 + r) * 2 * p.half + at;
+        const float4 co = *reinterpret_cast<const float4*>(cs), si = *reinterpret_cast<const float4*>(cs + p.half);
+        b[t][0] = g.x; b[t][1] = g.y; b[t][2] = g.z; b[t][3] = g.w;
+        c[t][0] = co.x; c[t][1] = co.y; c[t][2] = co.z; c[t][3] = co.w;
+        s[t][0] = si.x; s[t][1] = si.y; s[t][2] = si.z; s[t][3] = si.w;
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < kBatch; ++t) {
+      const int i = i0 + t * kLcOuterThreads, r = i / per, k = i - r * per;
+      if (i >= total) break;
+      const bool turn = k < pairs;
+      const int at = turn ? 4 * k : 2 * p.half + 4 * (k - pairs);
+      float x[4], y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (turn) rotate_pair(a[t][e], b[t][e], c[t][e] * p.amplitude, s[t][e] * p.amplitude, x[e], y[e]);
+        else x[e] = a[t][e];
+        x[e] *= scale;
+        y[e] *= scale;
+      }
+      put(r, at, x);
+      if (turn) put(r, at + p.half, y);
+    }
+  }
+}
+
 // Four neighbouring bfloat16 values as one 8-byte store (tile rows are an even number of elements wide).
 __device__ __forceinline__ void lc_store4(bf16* dst, float a, float b, float c, float d) {
   uint2 raw;
@@ -115,7 +164,7 @@ __device__ __forceinline__ void lc_pv_64(float (&o)[8][4], const uint32_t (&a)[4
   }
 }
 
-template <int DK, int DVB>                     // DVB: columns of S a block forms
+template <int DK, int DVB, bool TURN>          // DVB: columns of S a block forms; TURN: q and k are turned and scaled on their way in
 __global__ void __launch_bounds__(kLcOuterThreads, 2)
 linear_chunk_outer_kernel(LinearChunkParams p) {
   constexpr int LDK = DK + 8, LDV = DVB + 8;
@@ -139,7 +188,7 @@ linear_chunk_outer_kernel(LinearChunkParams p) {
   bf16* qg = p.q + th * kLcRows * DK;
   bf16* kg = p.k + th * kLcRows * DK;
   bf16* vg = p.v + th * kLcRows * p.dvp + c0;
-  lc_rows<DK>(src + p.k_base + qk, p.ld, n, p.dk, p.silu, p.vec, [&](int r, int c, const float (&x)[4]) {
+  auto put_k = [&](int r, int c, const float (&x)[4]) {
     // the key as a bfloat16 operand, then times its power of the decay in two parts
     const float f = r < n ? pw[n - 1 - r] : 0.f;
     float y[4], hi[4];
@@ -154,17 +203,21 @@ linear_chunk_outer_kernel(LinearChunkParams p) {
       lc_store4(kg + r * DK + c, x[0], x[1], x[2], x[3]);
       if (p.k_lo) lc_store4(p.k_lo + th * kLcRows * DK + r * DK + c, x[0] - lc_round(x[0]), x[1] - lc_round(x[1]), x[2] - lc_round(x[2]), x[3] - lc_round(x[3]));
     }
-  });
+  };
+  if constexpr (TURN) lc_rows_turned<DK>(p, src + p.k_base + qk, row0, n, p.k_scale, put_k);
+  else lc_rows<DK>(src + p.k_base + qk, p.ld, n, p.dk, p.silu, p.vec, put_k);
   lc_rows<DVB>(src + p.v_base + head * p.dv + c0, p.ld, n, p.dv - c0, p.silu, p.vec, [&](int r, int c, const float (&x)[4]) {
     lc_store4(vs + r * LDV + c, x[0], x[1], x[2], x[3]);
     lc_store4(vg + r * p.dvp + c, x[0], x[1], x[2], x[3]);
   });
-  if (first)
-    lc_rows<DK>(src + p.q_base + qk, p.ld, n, p.dk, p.silu, p.vec,
-                [&](int r, int c, const float (&x)[4]) {
-                  lc_store4(qg + r * DK + c, x[0], x[1], x[2], x[3]);
-                  if (p.q_lo) lc_store4(p.q_lo + th * kLcRows * DK + r * DK + c, x[0] - lc_round(x[0]), x[1] - lc_round(x[1]), x[2] - lc_round(x[2]), x[3] - lc_round(x[3]));
-                });
+  if (first) {
+    auto put_q = [&](int r, int c, const float (&x)[4]) {
+      lc_store4(qg + r * DK + c, x[0], x[1], x[2], x[3]);
+      if (p.q_lo) lc_store4(p.q_lo + th * kLcRows * DK + r * DK + c, x[0] - lc_round(x[0]), x[1] - lc_round(x[1]), x[2] - lc_round(x[2]), x[3] - lc_round(x[3]));
+    };
+    if constexpr (TURN) lc_rows_turned<DK>(p, src + p.q_base + qk, row0, n, 1.f, put_q);
+    else lc_rows<DK>(src + p.q_base + qk, p.ld, n, p.dk, p.silu, p.vec, put_q);
+  }
   __syncthreads();
   float* dst = p.outer + th * DK * p.dvp + c0;
   const int g = lane >> 2, t4 = lane & 3;
@@ -370,16 +423,20 @@ static LinearChunkScratch linear_chunk_scratch(int tiles, int heads, int DK, int
 static int linear_chunk_dk(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : 128; }
 static int linear_chunk_dvp(int dv) { return (dv + 63) / 64 * 64; }
 
-template <int DK, int DVB>
-static int launch_linear_outer(const LinearChunkParams& p, cudaStream_t s) {
+template <int DK, int DVB, bool TURN>
+static int launch_linear_outer_as(const LinearChunkParams& p, cudaStream_t s) {
   constexpr size_t smem = size_t(2 * kLcRows * (DK + 8) + kLcRows * (DVB + 8)) * sizeof(bf16);
   static bool configured = false;
   if (!configured && smem > 40 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(linear_chunk_outer_kernel<DK, DVB>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    const cudaError_t e = cudaFuncSetAttribute(linear_chunk_outer_kernel<DK, DVB, TURN>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     if (e != cudaSuccess) return int(e);
     configured = true;
   }
-  return pdl_launch(linear_chunk_outer_kernel<DK, DVB>, dim3(p.tiles, p.heads, p.dvp / DVB), dim3(kLcOuterThreads), smem, s, p);
+  return pdl_launch(linear_chunk_outer_kernel<DK, DVB, TURN>, dim3(p.tiles, p.heads, p.dvp / DVB), dim3(kLcOuterThreads), smem, s, p);
+}
+template <int DK, int DVB>
+static int launch_linear_outer(const LinearChunkParams& p, cudaStream_t s) {
+  return p.cs ? launch_linear_outer_as<DK, DVB, true>(p, s) : launch_linear_outer_as<DK, DVB, false>(p, s);
 }
 
 template <int DK, bool EXACT>
@@ -417,11 +474,12 @@ KVCM_API long long kvcm_linear_chunk_scratch_bytes(int tiles, int heads, int dk,
 
 // Runs the recurrence over the rows of every portion of more than one token (the step's tiles of 64 rows); single-row
 // entries are not touched.  proj: float rows of `ld` elements with q, k, v at the given bases; decay [heads]; scratch:
-// kvcm_linear_chunk_scratch_bytes(), 16-byte aligned; out: float [rows, heads * dv].
+// kvcm_linear_chunk_scratch_bytes(), 16-byte aligned; cs (optional): q and k are turned on their way in, k times k_scale; out: float [rows, heads * dv].
 KVCM_API int kvcm_linear_chunk(const float* proj, int ld, int q_base, int k_base, int v_base, const float* decay, void* scratch,
                                float* state, long long state_stride, const int* tile_seq, const int* tile_q0,
                                const int* seq_q_start, const int* seq_q_len, const int* seq_state_slot, float* out, int tiles,
-                               int heads, int qk_heads, int dk, int dv, int silu, int exact, void* stream) {
+                               int heads, int qk_heads, int dk, int dv, int silu, int exact, const float* cs, int half, float amplitude,
+                               float k_scale, void* stream) {
   if (tiles == 0) return 0;
   if (dk < 1 || dk > 128 || dv < 1 || qk_heads < 1 || heads % qk_heads || tiles > 65535 || heads > 65535 ||
       (reinterpret_cast<uintptr_t>(scratch) & 15))
@@ -438,6 +496,8 @@ KVCM_API int kvcm_linear_chunk(const float* proj, int ld, int q_base, int k_base
   p.q_lo = exact ? reinterpret_cast<bf16*>(base + at.q_lo) : nullptr; p.k_lo = exact ? reinterpret_cast<bf16*>(base + at.k_lo) : nullptr;
   p.vec = (dk % 4) == 0 && (dv % 4) == 0 && (ld % 4) == 0 && (q_base % 4) == 0 && (k_base % 4) == 0 && (v_base % 4) == 0 &&
           (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
+  p.cs = cs; p.half = half; p.amplitude = amplitude; p.k_scale = k_scale;
+  if (cs && (!p.vec || silu || half < 4 || half % 4 || 2 * half > dk || (reinterpret_cast<uintptr_t>(cs) & 15))) return KVCM_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
   if (dk <= 32) return launch_linear_chunk<32>(p, s);
   if (dk <= 64) return launch_linear_chunk<64>(p, s);

@@ -70,7 +70,7 @@ __device__ __forceinline__ void load_cols(float (&v)[1], const float* p) { v[0] 
 template <typename T> __device__ __forceinline__ void store_cols(T* p, const float (&v)[4]) { st4(p, v[0], v[1], v[2], v[3]); }
 template <typename T> __device__ __forceinline__ void store_cols(T* p, const float (&v)[1]) { stf(p, v[0]); }
 
-// Two block-wide sums at once.
+// Two block-wide sums at once, with one barrier (`scratch`, 32 pairs, is not used again by the launch).
 __device__ __forceinline__ float2 block_sum2(float a, float b, float2* scratch) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   a = warp_sum(a);
@@ -178,6 +178,104 @@ norm_post_pre_kernel(NormPostPreParams p) {
 #pragma unroll
     for (int e = 0; e < V; ++e) x[e] = w[e] * (x[e] * inv2);
     store_cols(o + i, x);
+  }
+}
+
+// The same for rows whose float4s fit NQ a thread: the row stays in registers, the weights (which no launch of the step
+// writes) are asked for before the wait, and every sum costs one barrier.
+template <typename T, int NQ, int MODE>
+__global__ void __launch_bounds__(512)
+norm_post_pre_regs_kernel(NormPostPreParams p) {
+  __shared__ float2 scratch[3][32];
+  pdl_launch_dependents();
+  const int H = p.H;
+  const int r = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+  float* xr = p.x + size_t(r) * H;
+  float x[NQ][4], y[NQ][4], wb[NQ][4], wn[NQ][4];
+  float z[MODE == kYJoined ? NQ : 1][4], w0[MODE == kYJoined ? NQ : 1][4], w1[MODE == kYJoined ? NQ : 1][4];
+  auto at = [&](int q) { return 4 * int(threadIdx.x + q * blockDim.x); };
+#pragma unroll
+  for (int q = 0; q < NQ; ++q) {
+    if (at(q) >= H) continue;
+    if constexpr (MODE != kYNone) load_cols(wb[q], p.wb + at(q));
+    if (p.out) load_cols(wn[q], p.wn + at(q));
+    if constexpr (MODE == kYJoined) {
+      load_cols(w0[q], p.w0 + at(q));
+      load_cols(w1[q], p.w1 + at(q));
+    }
+  }
+  pdl_wait();
+#pragma unroll
+  for (int q = 0; q < NQ; ++q) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[q][e] = y[q][e] = 0.f;
+    if constexpr (MODE == kYJoined) z[q][0] = z[q][1] = z[q][2] = z[q][3] = 0.f;
+    if (at(q) >= H) continue;
+    load_cols(x[q], xr + at(q));
+    if constexpr (MODE == kYDense || MODE == kYJoined) load_cols(y[q], p.y + size_t(r) * H + at(q));
+    if constexpr (MODE == kYJoined) load_cols(z[q], p.y1 + size_t(r) * H + at(q));
+  }
+  if constexpr (MODE == kYExperts) {
+#pragma unroll 4
+    for (int k = 0; k < p.top; ++k) {
+      const float* src = p.y + size_t(p.place[size_t(r) * p.top + k]) * H;
+      const float w = p.wt[size_t(r) * p.top + k];
+#pragma unroll
+      for (int q = 0; q < NQ; ++q) {
+        if (at(q) >= H) continue;
+        float a[4];
+        load_cols(a, src + at(q));
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[q][e] = fmaf(w, a[e], y[q][e]);
+      }
+    }
+  }
+  float s2 = 0.f;
+  if constexpr (MODE != kYNone) {
+    float sa = 0.f, sb = 0.f;
+    if constexpr (MODE == kYJoined) {
+#pragma unroll
+      for (int q = 0; q < NQ; ++q)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sa = fmaf(y[q][e], y[q][e], sa);
+          sb = fmaf(z[q][e], z[q][e], sb);
+        }
+      const float2 t = block_sum2(sa, sb, scratch[0]);
+      const float i0 = 1.f / sqrtf(t.x / float(H) + p.eps_join), i1 = 1.f / sqrtf(t.y / float(H) + p.eps_join);
+#pragma unroll
+      for (int q = 0; q < NQ; ++q)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (at(q) < H) y[q][e] = w0[q][e] * (y[q][e] * i0) + w1[q][e] * (z[q][e] * i1);
+      sa = 0.f;
+    }
+#pragma unroll
+    for (int q = 0; q < NQ; ++q)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sa = fmaf(y[q][e], y[q][e], sa);
+    const float inv = 1.f / sqrtf(block_sum2(sa, 0.f, scratch[1]).x / float(H) + p.eps);
+#pragma unroll
+    for (int q = 0; q < NQ; ++q) {
+      if (at(q) >= H) continue;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[q][e] = x[q][e] + wb[q][e] * (y[q][e] * inv);
+      if (!p.rows) store_cols(xr + at(q), x[q]);
+    }
+    if (!p.out) return;
+  }
+#pragma unroll
+  for (int q = 0; q < NQ; ++q)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s2 = fmaf(x[q][e], x[q][e], s2);
+  const float inv2 = 1.f / sqrtf(block_sum2(s2, 0.f, scratch[2]).x / float(H) + p.eps);
+  T* o = reinterpret_cast<T*>(p.out) + size_t(blockIdx.x) * H;
+#pragma unroll
+  for (int q = 0; q < NQ; ++q) {
+    if (at(q) >= H) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[q][e] = wn[q][e] * (x[q][e] * inv2);
+    store_cols(o + at(q), x[q]);
   }
 }
 
@@ -348,6 +446,13 @@ KVCM_API int kvcm_embed_scaled_bf16(KVCM_EMBED_SCALED_ARGS) {
 
 template <typename T, int V, int MODE>
 static int launch_norm_post_pre_as(const NormPostPreParams& p, int rows, cudaStream_t s) {
+  if constexpr (V == 4) {
+    const int quads = p.H / 4;
+    if (quads <= 512 && (rows < 256 || quads < 128))     // (many rows: fewer, longer threads and more rows at a time)
+      return pdl_launch(norm_post_pre_regs_kernel<T, 1, MODE>, dim3(rows), dim3((quads + 31) / 32 * 32), 0, s, p);
+    if (quads <= 1024)
+      return pdl_launch(norm_post_pre_regs_kernel<T, 2, MODE>, dim3(rows), dim3((quads + 63) / 64 * 32), 0, s, p);
+  }
   const size_t smem = size_t(p.H) * (MODE == kYJoined ? 3 : 2) * sizeof(float);
   if (smem > 200 * 1024) return KVCM_ERR_UNSUPPORTED;
   static size_t configured = 0;

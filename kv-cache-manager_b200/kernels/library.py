@@ -1226,12 +1226,20 @@ def linear_chunk_supported(dk: int) -> bool:
     return int(dk) <= int(_lib().kvcm_linear_chunk_max_dk())
 
 
+def linear_chunk_turns(columns: int, bases, dk: int, dv: int, pairs: int) -> bool:
+    """True when ``linear_chunk`` can turn q and k of this row layout itself."""
+    return pairs >= 4 and pairs % 4 == 0 and all(n % 4 == 0 for n in (columns, dk, dv, *bases))
+
+
 def linear_chunk(qkv: torch.Tensor, bases, decay: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int,
-                 qk_heads: int, dk: int, dv: int, silu: bool = False, exact: bool = False) -> None:
+                 qk_heads: int, dk: int, dv: int, silu: bool = False, exact: bool = False, table: Optional[torch.Tensor] = None,
+                 amplitude: float = 1.0, k_scale: float = 1.0) -> None:
     """``state_scan``'s linear form with one constant decay per head (``decay`` float32 [heads]), in chunks of 64 tokens on the
     tensor cores, for the step's portions of more than one token (csrc/cuda/linear_chunk.cu); rows of single-row
     entries are left alone.  For a 16-bit model: v, and without ``exact`` q and k too, are bfloat16 operands there; with it
-    q and k keep 16 leading bits (they are no plain projections: rotated, scaled)."""
+    q and k keep 16 leading bits (they are no plain projections: rotated, scaled).  ``table`` (float32 [T, 2 * pairs],
+    ``rope_table``): q and k are turned as they are read, in pairs (i, i + pairs), by the step's angles times ``amplitude``,
+    and k is multiplied by ``k_scale`` (see ``linear_chunk_turns``)."""
     _cuda(qkv, decay, state, out)
     _need(all(t.dtype == torch.float32 for t in (qkv, decay, state, out)), "linear_chunk: float32")
     _need(qkv.is_contiguous() and out.is_contiguous() and state.dim() == 2 and state.stride(1) == 1 and decay.is_contiguous() and decay.numel() == heads,
@@ -1240,12 +1248,15 @@ def linear_chunk(qkv: torch.Tensor, bases, decay: torch.Tensor, state: torch.Ten
     C = qkv.shape[1]
     _need(max(qb, kb) + qk_heads * dk <= C and vb + heads * dv <= C and out.shape == (qkv.shape[0], heads * dv)
           and state.shape[1] >= heads * dk * dv and ctx.tile_rows == 64, "linear_chunk: shapes")
+    _need(table is None or (table.dtype == torch.float32 and table.is_contiguous() and table.is_cuda and table.shape[0] == qkv.shape[0] and not silu),
+          "linear_chunk: table float32 [T, 2 * pairs]")
     tiles = ctx.prefill_tiles
     _lib().kvcm_linear_chunk_scratch_bytes.restype = ctypes.c_longlong
     scratch = torch.empty((int(_lib().kvcm_linear_chunk_scratch_bytes(tiles, heads, dk, dv, int(bool(exact)))),), dtype=torch.uint8, device=qkv.device)
     _check(_lib().kvcm_linear_chunk(_p(qkv), C, qb, kb, vb, _p(decay), _p(scratch), _p(state), _ll(state.stride(0)), _p(ctx.tile_seq),
                                     _p(ctx.tile_q0), _p(ctx.seq_q_start), _p(ctx.seq_q_len), _p(ctx.seq_state_slot), _p(out), tiles,
-                                    heads, qk_heads, dk, dv, int(bool(silu)), int(bool(exact)), _stream()), "linear_chunk", f"(dk={dk}, dv={dv})")
+                                    heads, qk_heads, dk, dv, int(bool(silu)), int(bool(exact)), _p(table), table.shape[1] // 2 if table is not None else 0,
+                                    ctypes.c_float(amplitude), ctypes.c_float(k_scale), _stream()), "linear_chunk", f"(dk={dk}, dv={dv})")
     global _launches
     _launches += 2                          # outer, carry, read
 
@@ -1661,7 +1672,7 @@ def norm_pair(x: torch.Tensor, pending, experts, w1: torch.Tensor, eps1: float, 
 class _HeadSegment(ctypes.Structure):
     _fields_ = [("out", ctypes.c_void_p), ("ld", ctypes.c_longlong), ("units", ctypes.c_int), ("dim", ctypes.c_int), ("HD", ctypes.c_int),
                 ("src", ctypes.c_int), ("conv", ctypes.c_int), ("table", ctypes.c_int), ("interleaved", ctypes.c_int),
-                ("dest", ctypes.c_int), ("scale", ctypes.c_float), ("items", ctypes.c_int)]
+                ("dest", ctypes.c_int), ("scale", ctypes.c_float), ("rows", ctypes.c_int), ("items", ctypes.c_int)]
 
 
 _HEAD_SEGMENTS, _GATE_SEGMENTS = 6, 4
@@ -1669,7 +1680,7 @@ _HEAD_SEGMENTS, _GATE_SEGMENTS = 6, 4
 
 class _HeadPrepareParams(ctypes.Structure):
     _fields_ = [("proj", ctypes.c_void_p), ("ldp", ctypes.c_longlong), ("positions", ctypes.c_void_p), ("inv_freq", ctypes.c_void_p * 2),
-                ("half", ctypes.c_int * 2), ("amplitude", ctypes.c_float * 2), ("conv_w", ctypes.c_void_p), ("state", ctypes.c_void_p),
+                ("cs", ctypes.c_void_p * 2), ("half", ctypes.c_int * 2), ("amplitude", ctypes.c_float * 2), ("conv_w", ctypes.c_void_p), ("state", ctypes.c_void_p),
                 ("state_stride", ctypes.c_longlong), ("taps", ctypes.c_int), ("channels", ctypes.c_int), ("conv_col", ctypes.c_int),
                 ("write_state", ctypes.c_int), ("row_seq", ctypes.c_void_p), ("seq_q_start", ctypes.c_void_p), ("seq_q_len", ctypes.c_void_p),
                 ("seq_state_slot", ctypes.c_void_p), ("slot_mapping", ctypes.c_void_p), ("block_size", ctypes.c_int), ("rows", ctypes.c_int),
@@ -1699,12 +1710,14 @@ class HeadSegment:
     them: ``conv`` (first channel of the step's short convolution), rotation by ``inv_freq`` (float32 [pairs]; None: none) with
     ``amplitude`` and the pairing, ``scale``, and where they go: ``dest`` "rows" (out [T, units * HD] in the storage dtype,
     padded with zeros), "pages" (out [pages, units, page, HD]) or "float" (out float32 rows, column of the first head
-    ``out_col``; may be the projection itself)."""
-    __slots__ = ("units", "dim", "src", "conv", "inv_freq", "amplitude", "interleaved", "scale", "dest", "out", "out_col")
+    ``out_col``; may be the projection itself).  ``table`` (float32 [T, 2 * pairs], ``rope_table``): the step's cosines and
+    sines, where they have been formed; ``rows``: only the step's first rows."""
+    __slots__ = ("units", "dim", "src", "conv", "inv_freq", "amplitude", "interleaved", "scale", "dest", "out", "out_col", "table", "rows")
 
     def __init__(self, units: int, dim: int, src: int, dest: str, out: torch.Tensor, conv: Optional[int] = None,
                  inv_freq: Optional[torch.Tensor] = None, amplitude: float = 1.0, interleaved: bool = False, scale: float = 1.0,
-                 out_col: int = 0) -> None:
+                 out_col: int = 0, table: Optional[torch.Tensor] = None, rows: Optional[int] = None) -> None:
+        self.table, self.rows = table, rows
         self.units, self.dim, self.src, self.dest, self.out, self.conv = units, dim, src, dest, out, conv
         self.inv_freq, self.amplitude, self.interleaved, self.scale, self.out_col = inv_freq, amplitude, interleaved, scale, out_col
 
@@ -1750,6 +1763,7 @@ def prepare_heads(proj: torch.Tensor, segments, ctx, dtype: torch.dtype, conv: O
         s = p.seg[i]
         s.units, s.dim, s.src, s.scale, s.interleaved = g.units, g.dim, g.src, g.scale, int(bool(g.interleaved))
         s.conv = -1 if g.conv is None else g.conv
+        s.rows = T if g.rows is None else min(int(g.rows), T)
         _need(g.src >= 0 and g.src + g.units * g.dim <= W and g.out.is_cuda, "prepare_heads: columns of a segment")
         _need(g.conv is None or (conv is not None and 0 <= g.conv and g.conv + g.units * g.dim <= channels and g.src == conv.col + g.conv),
               "prepare_heads: convolved columns and channels go together")
@@ -1763,6 +1777,10 @@ def prepare_heads(proj: torch.Tensor, segments, ctx, dtype: torch.dtype, conv: O
                 _need(len(tables) <= 2, "prepare_heads: at most two rotations")
                 t = len(tables) - 1
                 p.inv_freq[t], p.half[t], p.amplitude[t] = key
+                if g.table is not None:
+                    _need(g.table.dtype == torch.float32 and g.table.is_contiguous() and g.table.is_cuda and g.table.shape == (T, 2 * g.inv_freq.numel()),
+                          "prepare_heads: table float32 [T, 2 * pairs]")
+                    p.cs[t] = g.table.data_ptr()
             s.table = tables.index(key)
         if g.dest == "pages":
             _need(slot_mapping is not None and g.out.dtype == dtype and g.out.is_contiguous() and g.out.dim() == 4 and g.out.shape[1] == g.units

@@ -17,6 +17,7 @@ import torch
 from ..kernels import library as K
 from .base import CacheSpec, MIXERS, Mixer, PositionEncoding, SiteCache, StagedWork, StateSpec, StepContext
 from .linear import Linear, matmul_nt
+from .rope import STEP_TABLE_ROWS
 
 
 def plain_amplitude(position: PositionEncoding) -> None:
@@ -213,7 +214,8 @@ class GeneralAttention(Mixer):
         nq, nk = self.nh * self.dk, self.nkv * self.dk
         work.q = torch.empty((proj.shape[0], self.nh * self.hd), dtype=dtype, device=proj.device)
         at = (0, nq, nq + nk) if self.taps else (None, None, None)
-        turn = dict(inv_freq=pos.inv_freq, amplitude=pos.amplitude, interleaved=pos.interleaved)
+        table = pos.step_table(ctx) if pos.inv_freq is not None and ctx.prefill_rows >= STEP_TABLE_ROWS else None
+        turn = dict(inv_freq=pos.inv_freq, amplitude=pos.amplitude, interleaved=pos.interleaved, table=table)
         work.segments.append(K.HeadSegment(self.nh, self.dk, base, "rows", work.q, conv=at[0], **turn))
         if site.writes:
             work.slot_mapping, work.block_size = g.slot_mapping, g.block_size

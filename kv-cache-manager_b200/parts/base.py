@@ -270,9 +270,12 @@ class StagedWork:
 def run_prepare(proj: torch.Tensor, works, dtype: torch.dtype, ctx: StepContext) -> None:
     """One ``prepare_heads`` launch for the given mixers (at most one of them convolves, at most one writes pages)."""
     from ..kernels import library as K
+    segments = [s for w in works for s in w.segments]
+    if not segments:
+        return
     conv = next((w.conv for w in works if w.conv is not None), None)
     paged = next((w for w in works if w.slot_mapping is not None), None)
-    K.prepare_heads(proj, [s for w in works for s in w.segments], ctx, dtype, conv, paged.slot_mapping if paged else None,
+    K.prepare_heads(proj, segments, ctx, dtype, conv, paged.slot_mapping if paged else None,
                     paged.block_size if paged else 1)
 
 

@@ -29,18 +29,23 @@ from .linear import Linear
 CHUNKED_MIN_TOKENS = 32       # portions at least this long take the chunked form
 
 
+def takes_chunks(ctx: StepContext, storage: torch.dtype, dk: int) -> bool:
+    """Whether a step's portions take the chunked form (its single rows never do)."""
+    mode = ctx.options.get("scan", "auto")
+    return (mode == "chunks" or (mode == "auto" and storage == torch.bfloat16 and ctx.max_q_len >= CHUNKED_MIN_TOKENS)) \
+        and ctx.prefill_tiles > 0 and K.linear_chunk_supported(dk)
+
+
 def constant_decay_recurrence(proj: torch.Tensor, bases, decay: torch.Tensor, state: torch.Tensor, ctx: StepContext, o: torch.Tensor,
-                              heads: int, dk: int, dv: int, storage: torch.dtype, silu: bool = False, exact: bool = False) -> None:
+                              heads: int, dk: int, dv: int, storage: torch.dtype, silu: bool = False, exact: bool = False, **turn) -> None:
     """S <- decay_h S + k v^T; o = S^T q over the step's rows, from and into ``state``; ``decay`` float32 [1, heads], q, k and v at
     ``bases`` of the float32 rows ``proj``.  16-bit storage: portions of CHUNKED_MIN_TOKENS and more in chunks on the tensor
-    cores (``exact``: with queries and keys in two parts each)."""
+    cores (``exact``: with queries and keys in two parts each; ``turn``: the chunked kernel's own rotation of their rows)."""
     rows = decay.expand(proj.shape[0], heads)
-    mode = ctx.options.get("scan", "auto")
-    if (mode == "chunks" or (mode == "auto" and storage == torch.bfloat16 and ctx.max_q_len >= CHUNKED_MIN_TOKENS)) \
-            and ctx.prefill_tiles > 0 and K.linear_chunk_supported(dk):
+    if takes_chunks(ctx, storage, dk):
         if ctx.decode_seqs:                                                          # the single-row entries come first
             K.state_scan(K.SCAN_LINEAR, proj, bases, None, rows, None, state, ctx, o, heads, heads, dk, dv, silu=silu, seqs=ctx.decode_seqs)
-        K.linear_chunk(proj, bases, decay, state, ctx, o, heads, heads, dk, dv, silu=silu, exact=exact)
+        K.linear_chunk(proj, bases, decay, state, ctx, o, heads, heads, dk, dv, silu=silu, exact=exact, **turn)
     else:
         K.state_scan(K.SCAN_LINEAR, proj, bases, None, rows, None, state, ctx, o, heads, heads, dk, dv, silu=silu)
 

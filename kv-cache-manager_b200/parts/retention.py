@@ -9,8 +9,8 @@ Each head's o is divided by its root mean square over dv (no weight), the heads 
 and go through the output projection.
 
 State of a request: one float32 row per call site, S of every head.  A staged mixer (see ``parts.base.Mixer``): one product gives
-q | k | v | g (float32), one launch turns and scales q and k in place, the recurrence is that of ``parts.lightning``, one
-launch normalises and gates.  Everything between the two products is float32 in both storage dtypes; in the chunked form
+q | k | v | g (float32), one launch turns and scales q and k in place (the chunked recurrence turns its rows itself, as it
+reads them), the recurrence is that of ``parts.lightning``, one launch normalises and gates.  Everything between the two products is float32 in both storage dtypes; in the chunked form
 of the recurrence v is a bfloat16 operand (a plain projection), q and k are split in two bfloat16 parts.
 """
 from __future__ import annotations
@@ -21,8 +21,9 @@ import torch
 
 from ..kernels import library as K
 from .base import MIXERS, Mixer, PositionEncoding, SiteCache, StagedWork, StateSpec, StepContext
-from .lightning import constant_decay_recurrence
+from .lightning import constant_decay_recurrence, takes_chunks
 from .linear import Linear
+from .rope import STEP_TABLE_ROWS
 
 
 @MIXERS.register("retention")
@@ -57,17 +58,25 @@ class Retention(Mixer):
 
     def begin(self, proj: torch.Tensor, base: int, dtype: torch.dtype, ctx: StepContext, site: SiteCache) -> StagedWork:
         work, pos, n = StagedWork(proj, base, dtype, ctx, site), self.position, self.heads * self.dk
-        turn = dict(inv_freq=pos.inv_freq, amplitude=pos.amplitude, interleaved=pos.interleaved)
-        if pos.inv_freq is not None:
+        rows, table, work.turn = ctx.rows, None, {}
+        if pos.inv_freq is not None and ctx.prefill_rows >= STEP_TABLE_ROWS:
+            table = pos.step_table(ctx)
+            if takes_chunks(ctx, dtype, self.dk) and not pos.interleaved and ctx.options.get("fuse", True) \
+                    and K.linear_chunk_turns(proj.shape[1], (base, base + n, base + 2 * n), self.dk, self.dv, pos.rotary_dim // 2):
+                work.turn = dict(table=table, amplitude=pos.amplitude, k_scale=self.dk ** -0.5)
+                rows = ctx.decode_seqs                      # the portions' rows are turned where they are read
+        turn = dict(inv_freq=pos.inv_freq, amplitude=pos.amplitude, interleaved=pos.interleaved, table=table, rows=rows)
+        if pos.inv_freq is not None and rows:
             work.segments.append(K.HeadSegment(self.heads, self.dk, base, "float", proj, out_col=base, **turn))
-        work.segments.append(K.HeadSegment(self.heads, self.dk, base + n, "float", proj, out_col=base + n, scale=self.dk ** -0.5, **turn))
+        if rows:
+            work.segments.append(K.HeadSegment(self.heads, self.dk, base + n, "float", proj, out_col=base + n, scale=self.dk ** -0.5, **turn))
         return work
 
     def mix(self, work: StagedWork) -> K.GateSegment:
         T, n, nk, base = work.proj.shape[0], self.heads * self.dv, self.heads * self.dk, work.base
         o = torch.empty((T, n), dtype=torch.float32, device=work.proj.device)        # (the recurrence zeroes padding rows)
         constant_decay_recurrence(work.proj, (base, base + nk, base + 2 * nk), self._decay, work.site.state, work.ctx, o, self.heads,
-                                  self.dk, self.dv, work.dtype, exact=True)
+                                  self.dk, self.dv, work.dtype, exact=True, **work.turn)
         work.out = torch.empty((T, n), dtype=work.dtype, device=work.proj.device)
         return K.GateSegment(o, work.out, self.heads, self.dv, base + 2 * nk + n, self.norm_eps, "silu")
 

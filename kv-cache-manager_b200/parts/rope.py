@@ -19,7 +19,11 @@ from typing import Optional
 
 import torch
 
+from ..kernels import library as K
 from .base import POSITION_ENCODINGS, PositionEncoding
+
+
+STEP_TABLE_ROWS = 256        # steps with that many rows of portions form their cosines and sines once for all layers
 
 
 @POSITION_ENCODINGS.register("rope")
@@ -53,6 +57,16 @@ class RotaryEmbedding(PositionEncoding):
 
     def prepare(self, device, dtype) -> None:
         self.inv_freq = self.frequency_table().to(device)
+
+    def step_table(self, ctx) -> torch.Tensor:
+        """The step's cosines and sines (float32 [rows, rotary_dim], without the amplitude), formed once per step for all layers
+        with these frequencies."""
+        key = ("rope_table", self.theta, self.rotary_dim, repr(self.scaling))
+        table = ctx.shared.get(key)
+        if table is None:
+            table = ctx.shared[key] = torch.empty((ctx.rows, self.rotary_dim), dtype=torch.float32, device=self.inv_freq.device)
+            K.rope_table(ctx.positions, self.inv_freq, table)
+        return table
 
 
 @POSITION_ENCODINGS.register("none")

@@ -12,7 +12,9 @@ them into the stream; with it they are returned as a ``NormedSum``, which the cl
 
 Two staged mixers (see ``parts.base.Mixer``) share launches: their input projections are one product (the matrices are joined
 row-wise once, after loading, and the mixers' own parameters become views of the joint one), their heads are prepared by one
-launch and gated by one.  ``fuse`` off: each mixer runs by itself.
+launch and gated by one.  In a step of single rows, whose kernels leave most of the device idle, the right mixer's launches
+behind the preparation go to a second stream that joins again before the mixers' results are read (``options['branches']``:
+'one' keeps to one stream).  ``fuse`` off: each mixer runs by itself.
 """
 from __future__ import annotations
 
@@ -23,6 +25,9 @@ import torch
 from ..kernels import library as K
 from .base import MIXERS, Mixer, NormedSum, SiteCache, StateSpec, StepContext, run_prepare
 from .linear import matmul_nt
+
+
+_SIDE_STREAMS = {}            # one per device, for all layers
 
 
 def _up4(n: int) -> int:
@@ -82,14 +87,34 @@ class SideBySideMixer(Mixer):
                                          for at, n in zip(self._state_starts, self._state_sizes))
         return self._sub_sites[key]
 
+    def _two_streams(self, proj: torch.Tensor, mixers, works):
+        """Each branch on a stream of its own.  What the side stream's launches read and write is allocated on either stream
+        and lives until the join is enqueued; a block freed later is used again on its own stream behind the next fork."""
+        main, device = torch.cuda.current_stream(), proj.device
+        side = _SIDE_STREAMS.get(device)
+        if side is None:
+            side = _SIDE_STREAMS[device] = torch.cuda.Stream(device=device)
+        outs = [None, None]
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            K.gate_heads(proj, [mixers[1].mix(works[1])])
+            outs[1] = mixers[1].finish(works[1])
+        K.gate_heads(proj, [mixers[0].mix(works[0])])
+        outs[0] = mixers[0].finish(works[0])
+        main.wait_stream(side)
+        return outs
+
     def forward(self, h: torch.Tensor, ctx: StepContext, site: SiteCache):
         sites, mixers = self._sites(site), (self.left, self.right)
         if self._joint is not None and ctx.options.get("fuse", True):
             proj = matmul_nt(h, self._joint, torch.float32, ctx.options)
             works = [m.begin(proj, at, h.dtype, ctx, s) for m, at, s in zip(mixers, (0, self.left.projection.out_features), sites)]
             run_prepare(proj, works, h.dtype, ctx)
-            K.gate_heads(proj, [m.mix(w) for m, w in zip(mixers, works)])
-            outs = [m.finish(w) for m, w in zip(mixers, works)]
+            if ctx.prefill_rows == 0 and ctx.options.get("branches", "two") == "two" and not K.profiling():
+                outs = self._two_streams(proj, mixers, works)
+            else:
+                K.gate_heads(proj, [m.mix(w) for m, w in zip(mixers, works)])
+                outs = [m.finish(w) for m, w in zip(mixers, works)]
         else:
             outs = [m.forward(h, ctx, s) for m, s in zip(mixers, sites)]
         if self.out_norm:
