@@ -1035,7 +1035,7 @@ def delta_conv(proj: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, co
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == C), "delta_conv: bias float32 [channels]")
     _need(conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape[0] == C, "delta_conv: taps [channels, taps] float32")
     _need(out.dtype == torch.float32 and out.is_contiguous() and proj.stride(1) == 1 and proj.shape[1] >= C, "delta_conv: layout")
-    _need(state.dtype == torch.float32 and state.is_contiguous() and state.dim() == 2
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
           and state.shape[1] >= conv_off + (taps - 1) * C, "delta_conv: state rows too short")
     fn = getattr(_lib(), "kvcm_delta_conv_" + _suffix(proj))
     _check(fn(_p(proj), proj.stride(0), _p(conv_w), taps, _p(state), _ll(state.stride(0)), _ll(conv_off), _p(ctx.row_seq),
