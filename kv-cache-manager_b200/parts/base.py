@@ -155,6 +155,7 @@ class SiteCache:
     writes: bool = True
     state: Optional[torch.Tensor] = None    # [slots, *shape], the mixer's
     block_state: Optional[torch.Tensor] = None   # [slots, *shape], the block's own (see Block.state_spec)
+    shares: Optional[tuple] = None          # the site as the parts of a composed mixer see it (made by that mixer, once)
 
 
 @dataclass

@@ -51,7 +51,6 @@ class SideBySideMixer(Mixer):
             sizes.append(s.shape[0] if s is not None else 0)
         self._state_sizes = tuple(sizes)
         self._state_starts = (0, _up4(sizes[0]))
-        self._sub_sites = {}
         self.out_norm = bool(out_norm)
         if self.out_norm:
             self.declare("left_out", (hidden,), init, "vector")
@@ -81,11 +80,10 @@ class SideBySideMixer(Mixer):
         """The call site as each mixer sees it: its own part of the state rows."""
         if site.state is None:
             return site, site
-        key = (site.state.data_ptr(), site.group, site.k.data_ptr() if site.k is not None else 0)
-        if key not in self._sub_sites:
-            self._sub_sites[key] = tuple(dataclasses.replace(site, state=site.state[:, at:at + n] if n else None)
-                                         for at, n in zip(self._state_starts, self._state_sizes))
-        return self._sub_sites[key]
+        if site.shares is None:
+            site.shares = tuple(dataclasses.replace(site, state=site.state[:, at:at + n] if n else None)
+                                for at, n in zip(self._state_starts, self._state_sizes))
+        return site.shares
 
     def _two_streams(self, proj: torch.Tensor, mixers, works):
         """Each branch on a stream of its own.  What the side stream's launches read and write is allocated on either stream
